@@ -4,9 +4,10 @@ from .vemedra import VemedraConfig
 from .pidutar import PidutarConfig
 from .ledudra import LedudraConfig
 from .tamovik import TamovikConfig
+from .zekalorn import ZekalornConfig
 from .registry import (ArchitectureEntry, load_config, register_architecture,
                        registered_architectures, resolve_architecture)
 
-__all__ = ["ConfigError", "ModelConfig", "Qwen3Config", "VemedraConfig", "PidutarConfig", "LedudraConfig", "TamovikConfig", "read_config_json", "take",
+__all__ = ["ConfigError", "ModelConfig", "Qwen3Config", "VemedraConfig", "PidutarConfig", "LedudraConfig", "TamovikConfig", "ZekalornConfig", "read_config_json", "take",
            "ArchitectureEntry", "load_config", "register_architecture",
            "registered_architectures", "resolve_architecture"]

@@ -11,7 +11,8 @@
 //
 // heads_prepare_kernel makes q, k, v out of a float32 projection row [q heads | k heads | v heads | gates]: bias,
 // optional RMS norm of every q and k head with a gain shared by the heads, optional rotation of NEIGHBOURING pairs
-// (2i, 2i + 1) of the first rot_dims elements by position * inv_freq[i] with cos and sin times `mag`, optional blend of
+// (2i, 2i + 1) of the first rot_dims elements by position * inv_freq[i] with cos and sin times `mag`, optional temperature
+// of the queries (q times 1 + coef * ln(floor((position + 1) / every) + 1), see temp_every), optional blend of
 // the values with those another layer made for the same token (v <- (1 - lam) v + lam v_first), cache write, and
 // sigmoid of the gate columns.
 #include "common.cuh"
@@ -30,6 +31,7 @@ struct PrepArgs {
   const float* inv_freq; int rot_dims; float mag;
   const float* v_first_in; float* v_first_out; const float* lam;
   float* gate_out; int n_gate;
+  int temp_every; float temp_coef;   // temp_every > 0: the queries' temperature
   int vec;        // every head is a multiple of four elements and every pointer 16-byte aligned: four elements a lane
 };
 
@@ -61,6 +63,7 @@ __global__ void __launch_bounds__(128) heads_prepare_kernel(const PrepArgs a) {
   const int H = a.H, G = a.G, dim = a.dim, vdim = a.vdim;
   const int half = a.inv_freq ? a.rot_dims / 2 : 0;
   const float lam = (a.v_first_in && a.lam) ? *a.lam : 0.f;
+  const float q_mul = a.temp_every > 0 ? 1.f + a.temp_coef * logf((float)((pos + 1) / a.temp_every + 1)) : 1.f;
 
   for (int head = blockIdx.y * 4 + warp; head < H + 2 * G; head += 4 * gridDim.y) {
     const bool is_q = head < H, is_k = !is_q && head < H + G;
@@ -77,6 +80,7 @@ __global__ void __launch_bounds__(128) heads_prepare_kernel(const PrepArgs a) {
         dst = (T*)a.k_pages + (((size_t)page * G + (head - H)) * SX_PAGE + (pos & 63)) * dim;
       }
       float inv = 1.f;
+      const float mul = is_q ? q_mul : 1.f;
       if (a.vec) {
         // four elements a lane (two pairs of the rotation): 16-byte loads, 8- or 16-byte stores
         if (gain) {
@@ -100,7 +104,7 @@ __global__ void __launch_bounds__(128) heads_prepare_kernel(const PrepArgs a) {
             s0 *= a.mag; c0 *= a.mag; s1 *= a.mag; c1 *= a.mag;
             x = make_float4(x.x * c0 - x.y * s0, x.y * c0 + x.x * s0, x.z * c1 - x.w * s1, x.w * c1 + x.z * s1);
           }
-          prep_st4(dst + d, x.x, x.y, x.z, x.w);
+          prep_st4(dst + d, x.x * mul, x.y * mul, x.z * mul, x.w * mul);
         }
         continue;
       }
@@ -115,13 +119,13 @@ __global__ void __launch_bounds__(128) heads_prepare_kernel(const PrepArgs a) {
         float sn, cs;
         sincosf((float)pos * a.inv_freq[i], &sn, &cs);
         sn *= a.mag; cs *= a.mag;
-        dst[2 * i] = from_f32<T>(u * cs - v * sn);
-        dst[2 * i + 1] = from_f32<T>(v * cs + u * sn);
+        dst[2 * i] = from_f32<T>((u * cs - v * sn) * mul);
+        dst[2 * i + 1] = from_f32<T>((v * cs + u * sn) * mul);
       }
       for (int d = 2 * half + lane; d < dim; d += 32) {
         float x = src[d] + (bs ? bs[d] : 0.f);
         if (gain) x *= inv * gain[d];
-        dst[d] = from_f32<T>(x);
+        dst[d] = from_f32<T>(x * mul);
       }
     } else {
       const int c = head - H - G;
@@ -162,7 +166,7 @@ extern "C" int sx_heads_prepare(const float* proj, int row, const float* bias, v
                                 const int* positions, const int* seq_of_token, const int* block_table, int maxp, int n_pages,
                                 int n_tokens, int H, int G, int dim, int vdim, const float* qn, const float* kn, float eps,
                                 const float* inv_freq, int rot_dims, float mag, const float* v_first_in, float* v_first_out,
-                                const float* lam, float* gate_out, int n_gate, int dt, cudaStream_t stream) {
+                                const float* lam, float* gate_out, int n_gate, int temp_every, float temp_coef, int dt, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || rot_dims < 0 || rot_dims % 2 || rot_dims > dim ||
       row < (H + G) * dim + G * vdim + n_gate)
@@ -173,6 +177,7 @@ extern "C" int sx_heads_prepare(const float* proj, int row, const float* bias, v
   a.H = H; a.G = G; a.dim = dim; a.vdim = vdim; a.qn = qn; a.kn = kn; a.eps = eps; a.inv_freq = inv_freq;
   a.rot_dims = rot_dims; a.mag = mag; a.v_first_in = v_first_in; a.v_first_out = v_first_out; a.lam = lam;
   a.gate_out = gate_out; a.n_gate = n_gate;
+  a.temp_every = temp_every; a.temp_coef = temp_coef;
   a.vec = dim % 4 == 0 && vdim % 4 == 0 && rot_dims % 4 == 0 && row % 4 == 0 &&
           (((uintptr_t)proj | (uintptr_t)bias | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)qn |
             (uintptr_t)kn | (uintptr_t)v_first_in | (uintptr_t)v_first_out) & 15) == 0;

@@ -46,6 +46,7 @@ LIBRARIES: Dict[str, tuple] = {
     "layernorm": ("layernorm.cu", []),
     "attn_scored": ("attn_scored.cu", []),
     "mlstm": ("mlstm.cu", []),
+    "delta": ("delta.cu", []),
     "latent": ("latent.cu", []),
     "moe": ("moe.cu", []),
     "moe_tc": ("moe_tc.cu", []),

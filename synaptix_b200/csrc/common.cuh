@@ -177,7 +177,14 @@ __device__ __forceinline__ float cluster_load_f32(const float* local, uint32_t r
 // ---------------------------------------------------------------------------------------
 #define SX_GATE_SIGMOID 0
 #define SX_GATE_GELU_TANH 1
+#define SX_UNARY_RELU2 2
 struct GateAct { float alpha, limit; int form; };
+// products of ONE matrix with an activation in their epilogue: form 2 is relu(z)^2, any other form is none
+__device__ __forceinline__ float unary_act(float z, const GateAct a) {
+  if (a.form != SX_UNARY_RELU2) return z;
+  const float r = fmaxf(z, 0.f);
+  return r * r;
+}
 __device__ __forceinline__ float gelu_tanh_f32(float z) {
   // 1 + tanh(y) = 2 / (1 + exp(-2 y)): one exponential, no cancellation for large |y|
   const float y = 0.7978845608028654f * (z + 0.044715f * z * z * z);

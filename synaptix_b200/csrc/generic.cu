@@ -17,11 +17,13 @@
 #include "common.cuh"
 
 // ---------------------------------------------------------------------------------------
-// embedding gather: out[t, :] = float(table[ids[t], :]) * scale; an id outside the table gives zeros
+// embedding gather: out[t, :] = float(table[ids[t], :]) * scale [+ float(pos_table[positions[t], :])]; an id outside its
+// table gives zeros for that part, a position beyond the last row reads the last row (the engine refuses such steps)
 // ---------------------------------------------------------------------------------------
 template <typename T>
 __global__ void embed_gather_kernel(const T* __restrict__ table, const int* __restrict__ ids,
-                                    float* __restrict__ out, int H, int V, float scale) {
+                                    float* __restrict__ out, int H, int V, float scale, const T* __restrict__ pos_table,
+                                    const int* __restrict__ positions, int P) {
   pdl_wait();
   pdl_trigger();
   const int t = blockIdx.x;
@@ -29,16 +31,25 @@ __global__ void embed_gather_kernel(const T* __restrict__ table, const int* __re
   const bool ok = id >= 0 && id < V;
   const T* row = table + (size_t)(ok ? id : 0) * H;
   float* o = out + (size_t)t * H;
+  if (pos_table) {
+    const T* pr = pos_table + (size_t)min(max(positions[t], 0), P - 1) * H;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = fmaf(ok ? to_f32(row[i]) : 0.f, scale, to_f32(pr[i]));
+    return;
+  }
   for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = ok ? to_f32(row[i]) * scale : 0.f;
 }
 
-extern "C" int sx_embed_gather(const void* table, int dt, const int* ids, float* out,
-                               int n_tokens, int H, int V, float scale, cudaStream_t stream) {
+// pos_table null: no positions
+extern "C" int sx_embed_gather(const void* table, int dt, const int* ids, float* out, int n_tokens, int H, int V, float scale,
+                               const void* pos_table, const int* positions, int P, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
+  if (pos_table != nullptr && (positions == nullptr || P <= 0)) return SX_ERR_SIZE;
   if (dt == SX_F32)
-    return sx_launch(embed_gather_kernel<float>, dim3(n_tokens), dim3(256), 0, stream, (const float*)table, ids, out, H, V, scale);
+    return sx_launch(embed_gather_kernel<float>, dim3(n_tokens), dim3(256), 0, stream, (const float*)table, ids, out, H, V, scale,
+                     (const float*)pos_table, positions, P);
   if (dt == SX_BF16)
-    return sx_launch(embed_gather_kernel<bf16>, dim3(n_tokens), dim3(256), 0, stream, (const bf16*)table, ids, out, H, V, scale);
+    return sx_launch(embed_gather_kernel<bf16>, dim3(n_tokens), dim3(256), 0, stream, (const bf16*)table, ids, out, H, V, scale,
+                     (const bf16*)pos_table, positions, P);
   return SX_ERR_DTYPE;
 }
 

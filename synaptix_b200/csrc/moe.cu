@@ -13,6 +13,8 @@
 //                      silu(gate) * up  [T * top, ff] in sorted order; else rows are read in sorted order and the
 //                      result is the plain product [T * top, N].  64x64x16 tiles, 4x4 results a thread, 32-bit FFMA
 //                      (float32, and bfloat16 with K % 8 != 0).
+//                      MODE MOE_UP (experts without a gate): rows gathered as for GATE_UP, one matrix [ff, K] an expert
+//                      and an activation of one operand (see unary_act).
 //   moe_mma_kernel     the same product for bfloat16 on the tensor cores (see there).
 //   moe_combine_kernel out[t] = sum_j weights[t, j] * y[place[t * top + j]], the choices in their order.
 #include "common.cuh"
@@ -223,11 +225,18 @@ __device__ __forceinline__ float moe_gate(float g, float u, const GateAct a) {
   return g / (1.f + expf(-g)) * u;
 }
 
-template <typename TA, typename TW, typename TC, bool GATE_UP>
+// what a grouped product does: rows in sorted order and the plain result; rows gathered, [gate; up] and the gated
+// activation; rows gathered, one matrix and an activation of its own
+#define MOE_PLAIN 0
+#define MOE_GATE_UP 1
+#define MOE_UP 2
+
+template <typename TA, typename TW, typename TC, int MODE>
 __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A, const TW* __restrict__ Wt, TC* __restrict__ C,
                                                        const int* __restrict__ offsets, const int* __restrict__ order,
                                                        int E, int N, int K, int top, const GateAct act) {
   constexpr int BM = 64, BN = 64, BK = 16;
+  constexpr bool GATE_UP = MODE == MOE_GATE_UP, GATHER = MODE != MOE_PLAIN;
   __shared__ float As[BK][BM + 4];
   __shared__ float Ws[BK][BN + 4];
   __shared__ float Us[GATE_UP ? BK : 1][BN + 4];
@@ -250,7 +259,7 @@ __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A,
   __syncthreads();
   const int e = which[0], r0 = which[1], nr = which[2];
   if (r0 < 0) return;
-  if (tid < BM) src[tid] = tid < nr ? (GATE_UP ? order[r0 + tid] / top : r0 + tid) : -1;
+  if (tid < BM) src[tid] = tid < nr ? (GATHER ? order[r0 + tid] / top : r0 + tid) : -1;
   __syncthreads();
   const int tx = tid & 15, ty = tid >> 4;
   const int n0 = blockIdx.x * BN;
@@ -297,7 +306,10 @@ __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A,
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < N) C[(size_t)(r0 + r) * N + n] = from_f32<TC>(GATE_UP ? moe_gate(acc[i][j], acu[i][j], act) : acc[i][j]);
+      if (n < N) {
+        const float z = GATE_UP ? moe_gate(acc[i][j], acu[i][j], act) : (MODE == MOE_UP ? unary_act(acc[i][j], act) : acc[i][j]);
+        C[(size_t)(r0 + r) * N + n] = from_f32<TC>(z);
+      }
     }
   }
 }
@@ -343,12 +355,13 @@ __device__ __forceinline__ void mm_mma(float* c, const uint32_t* a, uint32_t b0,
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-template <typename TC, bool GATE_UP, int BM>
+template <typename TC, int MODE, int BM>
 __global__ void __launch_bounds__(256) moe_mma_kernel(const bf16* __restrict__ A, const bf16* __restrict__ Wt, TC* __restrict__ C,
                                                       const int* __restrict__ offsets, const int* __restrict__ order,
                                                       int E, int N, int K, int top, const GateAct act) {
   using Sh = MmShape<BM>;
   constexpr int STAGES = Sh::STAGES, MI = Sh::MI, NT = Sh::NT;
+  constexpr bool GATE_UP = MODE == MOE_GATE_UP, GATHER = MODE != MOE_PLAIN;
   extern __shared__ __align__(16) unsigned char mm_smem[];
   bf16* As = (bf16*)mm_smem;                                        // STAGES * BM * MM_LD
   bf16* Ws = As + STAGES * BM * MM_LD;                              // STAGES * MM_BN * MM_LD
@@ -370,7 +383,7 @@ __global__ void __launch_bounds__(256) moe_mma_kernel(const bf16* __restrict__ A
   __syncthreads();
   const int e = which[0], r0 = which[1], nr = which[2];
   if (r0 < 0) return;
-  if (tid < BM) src[tid] = tid < nr ? (GATE_UP ? order[r0 + tid] / top : r0 + tid) : -1;
+  if (tid < BM) src[tid] = tid < nr ? (GATHER ? order[r0 + tid] / top : r0 + tid) : -1;
   __syncthreads();
   constexpr int NOUT = GATE_UP ? MM_BN / 2 : MM_BN;                 // output columns of a block
   const int n0 = blockIdx.x * NOUT;
@@ -480,58 +493,62 @@ __global__ void __launch_bounds__(256) moe_mma_kernel(const bf16* __restrict__ A
 #pragma unroll
           for (int x = 0; x < 2; ++x) {
             const int n = n0 + wn * NT * 8 + j * 8 + col_in + x;
-            if (n < N) crow[n] = from_f32<TC>(acc[mi][j][half * 2 + x]);
+            if (n < N) crow[n] = from_f32<TC>(MODE == MOE_UP ? unary_act(acc[mi][j][half * 2 + x], act) : acc[mi][j][half * 2 + x]);
           }
       }
     }
 }
 
-template <typename TC, bool GATE_UP, int BM>
+template <typename TC, int MODE, int BM>
 static int moe_mma_launch(const void* A, const void* Wt, void* C, const int* offsets, const int* order, int rows, int E, int N,
                           int K, int top, cudaStream_t stream) {
   const size_t smem = MmShape<BM>::SMEM;
   static bool set = false;
   if (!set) {
-    cudaError_t err = cudaFuncSetAttribute(moe_mma_kernel<TC, GATE_UP, BM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t err = cudaFuncSetAttribute(moe_mma_kernel<TC, MODE, BM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (err != cudaSuccess) return (int)err;
     set = true;
   }
   const int tiles = (rows + BM - 1) / BM + (E < rows ? E : rows);
   if (tiles > 65535) return SX_ERR_SIZE;
-  const int nout = GATE_UP ? MM_BN / 2 : MM_BN;
+  const int nout = MODE == MOE_GATE_UP ? MM_BN / 2 : MM_BN;
   dim3 grid((N + nout - 1) / nout, tiles);
-  return sx_launch(moe_mma_kernel<TC, GATE_UP, BM>, grid, dim3(256), smem, stream, (const bf16*)A, (const bf16*)Wt, (TC*)C, offsets,
+  return sx_launch(moe_mma_kernel<TC, MODE, BM>, grid, dim3(256), smem, stream, (const bf16*)A, (const bf16*)Wt, (TC*)C, offsets,
                    order, E, N, K, top, g_sx_gate);
 }
 
 // up to this many (token, choice) rows a step, blocks of 16 rows with the deeper ring
 #define MM_FEW_ROWS 64
 
-// rows: T * top; the grid's y axis has room for every expert's last, partly filled tile
+// rows: T * top; the grid's y axis has room for every expert's last, partly filled tile; mode: MOE_PLAIN, MOE_GATE_UP, MOE_UP
 extern "C" int sx_moe_gemm(const void* A, const void* Wt, void* C, const int* offsets, const int* order, int rows, int E, int N,
-                           int K, int top, int gate_up, int a_dt, int c_dt, cudaStream_t stream) {
+                           int K, int top, int mode, int a_dt, int c_dt, cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (E <= 0 || N <= 0 || K <= 0) return SX_ERR_SIZE;
+  if (E <= 0 || N <= 0 || K <= 0 || mode < MOE_PLAIN || mode > MOE_UP) return SX_ERR_SIZE;
   const int tiles = (rows + 63) / 64 + (E < rows ? E : rows);
   if (tiles > 65535) return SX_ERR_SIZE;
   if (a_dt == SX_BF16 && K % 8 == 0 && ((uintptr_t)A | (uintptr_t)Wt) % 16 == 0) {       // the tensor cores
-#define MM_GO(TC, GU)                                                                                               \
-  return rows <= MM_FEW_ROWS ? moe_mma_launch<TC, GU, 16>(A, Wt, C, offsets, order, rows, E, N, K, top, stream)    \
-                             : moe_mma_launch<TC, GU, 64>(A, Wt, C, offsets, order, rows, E, N, K, top, stream)
-    if (gate_up && c_dt == SX_BF16) MM_GO(bf16, true);
-    if (!gate_up && c_dt == SX_F32) MM_GO(float, false);
-    if (!gate_up && c_dt == SX_BF16) MM_GO(bf16, false);
+#define MM_GO(TC, M)                                                                                              \
+  return rows <= MM_FEW_ROWS ? moe_mma_launch<TC, M, 16>(A, Wt, C, offsets, order, rows, E, N, K, top, stream)    \
+                             : moe_mma_launch<TC, M, 64>(A, Wt, C, offsets, order, rows, E, N, K, top, stream)
+    if (mode == MOE_GATE_UP && c_dt == SX_BF16) MM_GO(bf16, MOE_GATE_UP);
+    if (mode == MOE_UP && c_dt == SX_BF16) MM_GO(bf16, MOE_UP);
+    if (mode == MOE_PLAIN && c_dt == SX_F32) MM_GO(float, MOE_PLAIN);
+    if (mode == MOE_PLAIN && c_dt == SX_BF16) MM_GO(bf16, MOE_PLAIN);
 #undef MM_GO
   }
   dim3 grid((N + 63) / 64, tiles);
-#define MOE_GO(TA, TC, GU) return sx_launch(moe_gemm_kernel<TA, TA, TC, GU>, grid, dim3(256), 0, stream, (const TA*)A, (const TA*)Wt, (TC*)C, offsets, order, E, N, K, top, g_sx_gate)
-  if (gate_up) {
-    if (a_dt == SX_F32 && c_dt == SX_F32) MOE_GO(float, float, true);
-    if (a_dt == SX_BF16 && c_dt == SX_BF16) MOE_GO(bf16, bf16, true);
+#define MOE_GO(TA, TC, M) return sx_launch(moe_gemm_kernel<TA, TA, TC, M>, grid, dim3(256), 0, stream, (const TA*)A, (const TA*)Wt, (TC*)C, offsets, order, E, N, K, top, g_sx_gate)
+  if (mode == MOE_GATE_UP) {
+    if (a_dt == SX_F32 && c_dt == SX_F32) MOE_GO(float, float, MOE_GATE_UP);
+    if (a_dt == SX_BF16 && c_dt == SX_BF16) MOE_GO(bf16, bf16, MOE_GATE_UP);
+  } else if (mode == MOE_UP) {
+    if (a_dt == SX_F32 && c_dt == SX_F32) MOE_GO(float, float, MOE_UP);
+    if (a_dt == SX_BF16 && c_dt == SX_BF16) MOE_GO(bf16, bf16, MOE_UP);
   } else {
-    if (a_dt == SX_F32 && c_dt == SX_F32) MOE_GO(float, float, false);
-    if (a_dt == SX_BF16 && c_dt == SX_F32) MOE_GO(bf16, float, false);
-    if (a_dt == SX_BF16 && c_dt == SX_BF16) MOE_GO(bf16, bf16, false);
+    if (a_dt == SX_F32 && c_dt == SX_F32) MOE_GO(float, float, MOE_PLAIN);
+    if (a_dt == SX_BF16 && c_dt == SX_F32) MOE_GO(bf16, float, MOE_PLAIN);
+    if (a_dt == SX_BF16 && c_dt == SX_BF16) MOE_GO(bf16, bf16, MOE_PLAIN);
   }
 #undef MOE_GO
   return SX_ERR_DTYPE;

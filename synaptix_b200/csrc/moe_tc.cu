@@ -9,7 +9,8 @@
 // by one lane -> accumulator in tensor memory -> tcgen05.ld epilogue of four warps:
 //   GATE_UP: the tile's 256 matrix rows are 128 gate rows and the 128 up rows of the same outputs; the epilogue
 //            writes silu(gate) * up as bfloat16 [rows, N];
-//   else:    the plain product as float32 [rows, N].
+//   UP:      one matrix an expert (256 rows a tile); the epilogue writes an activation of the product as bfloat16;
+//   PLAIN:   the plain product as float32 [rows, N].
 // Every wait on an mbarrier is bounded; a wait that runs out sets the status word, and the block still frees its
 // tensor memory.  K % 8 == 0 (TMA strides); a tail of K is zero-filled by TMA.
 #include "tcgen05.cuh"
@@ -23,11 +24,16 @@
 #define MT_STAGES 4
 #define MT_THREADS 192
 
-template <bool GATE_UP>
+#define MT_PLAIN 0
+#define MT_GATE_UP 1
+#define MT_UP 2
+
+template <int MODE>
 __global__ void __launch_bounds__(MT_THREADS, 1) moe_tc_kernel(const __grid_constant__ CUtensorMap map_a,
                                                                const __grid_constant__ CUtensorMap map_w,
                                                                void* __restrict__ out, const int* __restrict__ offsets,
                                                                int E, int N, int K, int* __restrict__ status, const GateAct act) {
+  constexpr bool GATE_UP = MODE == MT_GATE_UP;
   extern __shared__ unsigned char mt_smem_raw[];
   unsigned char* tiles = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(mt_smem_raw) + 1023) & ~(uintptr_t)1023);
   uint64_t* bars = reinterpret_cast<uint64_t*>(tiles + MT_STAGES * MT_STAGE_BYTES);   // full[S], empty[S], accum
@@ -120,13 +126,13 @@ __global__ void __launch_bounds__(MT_THREADS, 1) moe_tc_kernel(const __grid_cons
         asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
         if (r >= nr || n0 + c0 >= N) continue;
         const int ncol = min(32, N - (n0 + c0));
-        if (GATE_UP) {
+        if (MODE != MT_PLAIN) {
           bf16* dst = reinterpret_cast<bf16*>(out) + (size_t)(m0 + r) * N + n0 + c0;
           float f[32];
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const float g = __uint_as_float(v[i]);
-            f[i] = gate_mul(g, __uint_as_float(u[i]), act);
+            f[i] = GATE_UP ? gate_mul(g, __uint_as_float(u[i]), act) : unary_act(g, act);
           }
           if (ncol == 32 && (N % 8) == 0) {
 #pragma unroll
@@ -197,13 +203,13 @@ extern "C" int sx_moe_tc_status(int* host_value, int reset) {
 }
 
 extern "C" int sx_moe_tc(const void* A, const void* Wt, void* out, const int* offsets, int rows, int E, int N, int K,
-                         int gate_up, cudaStream_t stream) {
+                         int mode, cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (E <= 0 || N <= 0 || K <= 0 || K % 8) return SX_ERR_SIZE;
+  if (E <= 0 || N <= 0 || K <= 0 || K % 8 || mode < MT_PLAIN || mode > MT_UP) return SX_ERR_SIZE;
   if (((uintptr_t)A | (uintptr_t)Wt | (uintptr_t)out) % 16) return SX_ERR_ALIGN;
   int* status = mt_status_word();
   if (!status) return SX_ERR_SIZE;
-  const int NW = gate_up ? 2 * N : N;
+  const int NW = mode == MT_GATE_UP ? 2 * N : N;
   CUtensorMap ma, mw;
   int rc = tc_make_map_rows(&ma, A, rows, K, MT_BM);
   if (rc) return rc;
@@ -212,22 +218,19 @@ extern "C" int sx_moe_tc(const void* A, const void* Wt, void* out, const int* of
   const int tiles = (rows + MT_BM - 1) / MT_BM + (E < rows ? E : rows);
   if (tiles > 65535) return SX_ERR_SIZE;
   const size_t smem = (size_t)MT_STAGES * MT_STAGE_BYTES + 1024 + (2 * MT_STAGES + 1) * 8 + 32;
-  if (gate_up) {
-    static bool set = false;
-    if (!set) {
-      cudaError_t err = cudaFuncSetAttribute(moe_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-      if (err != cudaSuccess) return (int)err;
-      set = true;
-    }
-    return sx_launch(moe_tc_kernel<true>, dim3((N + MT_BN / 2 - 1) / (MT_BN / 2), tiles), dim3(MT_THREADS), smem, stream, ma, mw, out,
-                     offsets, E, N, K, status, g_sx_gate);
-  }
-  static bool set2 = false;
-  if (!set2) {
-    cudaError_t err = cudaFuncSetAttribute(moe_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (err != cudaSuccess) return (int)err;
-    set2 = true;
-  }
-  return sx_launch(moe_tc_kernel<false>, dim3((N + MT_BN - 1) / MT_BN, tiles), dim3(MT_THREADS), smem, stream, ma, mw, out, offsets, E,
-                   N, K, status, g_sx_gate);
+#define MT_GO(M, COLS)                                                                                                             \
+  do {                                                                                                                            \
+    static bool set = false;                                                                                                      \
+    if (!set) {                                                                                                                   \
+      cudaError_t err = cudaFuncSetAttribute(moe_tc_kernel<M>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
+      if (err != cudaSuccess) return (int)err;                                                                                    \
+      set = true;                                                                                                                 \
+    }                                                                                                                             \
+    return sx_launch(moe_tc_kernel<M>, dim3((N + COLS - 1) / COLS, tiles), dim3(MT_THREADS), smem, stream, ma, mw, out, offsets,  \
+                     E, N, K, status, g_sx_gate);                                                                                 \
+  } while (0)
+  if (mode == MT_GATE_UP) MT_GO(MT_GATE_UP, (MT_BN / 2));
+  if (mode == MT_UP) MT_GO(MT_UP, MT_BN);
+  MT_GO(MT_PLAIN, MT_BN);
+#undef MT_GO
 }

@@ -29,6 +29,7 @@ import torch
 
 from .. import ops
 from ..cache import PAGE_TOKENS, Cache, pages_for
+from ..cache.pages import CacheFull
 from ..csrc.build import KernelsUnavailable
 from ..parts.base import StepContext
 
@@ -273,6 +274,11 @@ class Engine:
         return self.cache.max_seqs
 
     @property
+    def max_positions(self) -> Optional[int]:
+        """How many tokens one sequence can have at most (a model with learned positions; ``None``: no such limit)."""
+        return getattr(self.model, "max_positions", None)
+
+    @property
     def free_tokens(self) -> int:
         """Tokens the pages hold that no open sequence has: what new sequences can still take."""
         return min(pool.n_free for pool in self.cache.slots.pools) * PAGE_TOKENS
@@ -335,6 +341,11 @@ class Engine:
                 if not (0 <= w < n):
                     raise StepError(f"slot {e.slot}: wanted place {w} is outside its {n} tokens")
         new = [len(e.tokens) for e in entries]
+        limit = self.max_positions
+        if limit is not None:
+            for e, n in zip(entries, new):
+                if slots.length(e.slot) + n > limit:
+                    raise StepError(f"slot {e.slot}: {slots.length(e.slot)} + {n} tokens, but the model has {limit} positions")
         slots.reserve_many([e.slot for e in entries], new)
         past = [slots.length(e.slot) for e in entries]
         return past, new
@@ -617,6 +628,9 @@ class DecodeSession:
         for r, ln in zip(self.rows, self.lens):
             if slots.length(r.slot) != ln:
                 raise StepError(f"slot {r.slot} was stepped outside its decode session")
+        limit = eng.max_positions
+        if limit is not None and max(self.lens) >= limit:
+            raise CacheFull(f"a sequence has reached the model's {limit} positions")       # as with the pages: nothing has changed
         slots.reserve_many([r.slot for r in self.rows], [1] * n)          # CacheFull: nothing has changed
         need_p = max(pages_for(ln + 1) for ln in self.lens)
         # a captured step has dummy rows up to a bucket; an eager one runs the live rows alone, since

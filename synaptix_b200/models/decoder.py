@@ -101,6 +101,11 @@ class DecoderModel(Part):
     def vocab_size(self) -> int:
         return self.head.vocab
 
+    @property
+    def max_positions(self) -> Optional[int]:
+        """How many tokens a sequence can have at most (``None``: as many as the cache holds)."""
+        return getattr(self.embedding, "max_positions", None)
+
     def children(self) -> List[Part]:
         extra = [self.stream_vectors] if self.stream_vectors is not None else []
         return [self.embedding] + extra + self.layers + [self.final_norm, self.head]
@@ -125,11 +130,8 @@ class DecoderModel(Part):
     # -- one step ------------------------------------------------------------
     def forward(self, ctx: StepContext, cache) -> torch.Tensor:
         """Logits float32 ``[n_want, vocab]`` for ``ctx.want_rows``."""
-        if self._embedding_entry is not None:
-            h = self.embedding.forward_step(ctx, cache.view(self._embedding_entry))
-        else:
-            h = self.embedding.forward(ctx.token_ids)
-        h0 = self.embedding.forward(ctx.token_ids) if self._keeps_embedding else None     # h is summed into in place
+        h = self.embedding.forward_step(ctx, cache.view(self._embedding_entry) if self._embedding_entry is not None else None)
+        h0 = self.embedding.forward_step(ctx) if self._keeps_embedding else None     # h is summed into in place
         pending = None
         observe = getattr(ctx, "observe", None)
         n_run = 0

@@ -23,7 +23,8 @@ from .options import OPTIONS, KernelOptions, options, set_options
 from .generic import (add_rmsnorm, attn_generic, decode_advance, decode_begin, embed_gather, gemm_generic, qkv_prepare,
                       residual_add, rope_table, silu_mul)
 from .sequence import add_rmsnorm_conv, capped_glu, mingru, retention, stream_add
-from .block import add_scaled, add_scaled_rmsnorm, scale_rows
+from .block import add_scaled, add_scaled_rmsnorm, scale_rows, side_gate
+from .delta import DeltaWeights, delta_rule, delta_step_fits
 from .layernorm import add_layernorm
 from .normed import WeightedRows, add_normed, embed_bigram
 from .convqk import convqk_prepare, sigmoid_gate
@@ -31,7 +32,7 @@ from .scored import attn_scored as attn_scored_all_heads, heads_prepare
 from .latent import (head_gate, latent_attention, latent_expand, latent_gather, latent_output, latent_prepare, latent_query,
                      latent_rotate_q)
 from .mlstm import mlstm
-from .moe import ExpertPlan, moe_combine, moe_down, moe_gate_up, moe_route, moe_sort
+from .moe import ExpertPlan, moe_combine, moe_down, moe_gate_up, moe_route, moe_sort, moe_up
 
 __all__ = ["OPTIONS", "KernelOptions", "options", "set_options", "KernelsUnavailable", "KernelError", "set_launch_counter", "decode_advance", "decode_begin", "check_status", "add_rmsnorm", "attn_generic", "embed_gather",
            "gemm_generic", "qkv_prepare", "residual_add", "silu_mul", "linear", "linear_normed", "norm_fusable", "attention",
@@ -39,7 +40,8 @@ __all__ = ["OPTIONS", "KernelOptions", "options", "set_options", "KernelsUnavail
            "linear_into_residual", "linear_scaled", "projection_prepares_heads", "project_and_prepare", "rope_table",
            "add_rmsnorm_conv", "capped_glu", "mingru", "retention", "stream_add", "gate_activation",
            "add_normed", "WeightedRows", "embed_bigram", "convqk_prepare", "sigmoid_gate", "add_scaled", "add_scaled_rmsnorm", "scale_rows", "add_layernorm", "attn_scored", "heads_prepare", "latent_attention", "latent_output", "latent_prepare",
-           "latent_query", "latent_gather", "latent_expand", "latent_rotate_q", "head_gate", "mlstm", "ExpertPlan", "moe_combine", "moe_down", "moe_gate_up", "moe_route", "moe_sort"]
+           "latent_query", "latent_gather", "latent_expand", "latent_rotate_q", "head_gate", "mlstm", "ExpertPlan", "moe_combine", "moe_down", "moe_gate_up", "moe_route", "moe_sort", "moe_up",
+           "side_gate", "DeltaWeights", "delta_rule", "delta_step_fits"]
 
 
 _STATUS_READERS = {"gemm_tc": ("the tcgen05 matrix product (gemm_tc)", "gemm_tc_status"),

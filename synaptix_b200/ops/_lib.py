@@ -130,9 +130,10 @@ c_ulonglong = ctypes.c_ulonglong
 # g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit); ``form="gelu_tanh"`` is
 # gelu_tanh(g) * u (the tanh form of GELU; alpha and limit unused).  A feed-forward that wants another form than the
 # first runs its gate/up product inside ``gate_activation(...)``; the faces of the products call ``use_gate`` before a
-# launch with that epilogue, which tells the library if its last value was another one.
+# launch with that epilogue, which tells the library if its last value was another one.  ``form="relu2"`` is for the
+# experts' products of ONE matrix (``moe_up``): relu(z)^2.
 # ---------------------------------------------------------------------------------------------------------------
-GATE_FORMS = {"sigmoid": 0, "gelu_tanh": 1}
+GATE_FORMS = {"sigmoid": 0, "gelu_tanh": 1, "relu2": 2}
 _GATE = [(0.0, 0.0, 0)]
 _LIB_GATE = {}
 

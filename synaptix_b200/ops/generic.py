@@ -10,9 +10,14 @@ from ._lib import (KernelError, c_float, c_int, c_longlong, check, dt_code, fn, 
 
 
 def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: Optional[torch.Tensor] = None,
-                 scale: float = 1.0) -> torch.Tensor:
-    """``out[t] = float32(table[ids[t]]) * scale``; ``ids`` int32 ``[T]``; result float32 ``[T, H]``."""
-    require_cuda(table, ids, out)
+                 scale: float = 1.0, pos_table: Optional[torch.Tensor] = None,
+                 positions: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out[t] = float32(table[ids[t]]) * scale``; ``ids`` int32 ``[T]``; result float32 ``[T, H]``.  ``pos_table`` (of
+    ``table``'s dtype and width) with ``positions`` int32 ``[T]``: ``+ float32(pos_table[positions[t]])``."""
+    require_cuda(table, ids, out, pos_table, positions)
+    if pos_table is not None and (positions is None or positions.dtype != torch.int32 or pos_table.dtype != table.dtype
+                                  or pos_table.shape[1] != table.shape[1]):
+        raise KernelError("embed_gather: the position table shares the table's dtype and width and comes with int32 positions")
     V, H = table.shape
     T = ids.numel()
     if ids.dtype != torch.int32:
@@ -20,7 +25,8 @@ def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: Optional[torch.Ten
     if out is None:
         out = torch.empty((T, H), dtype=torch.float32, device=table.device)
     check(fn("generic", "sx_embed_gather")(ptr(table), c_int(dt_code(table.dtype)), ptr(ids), ptr(out),
-                                           c_int(T), c_int(H), c_int(V), c_float(scale), stream()), "embed_gather")
+                                           c_int(T), c_int(H), c_int(V), c_float(scale), ptr(pos_table), ptr(positions),
+                                           c_int(0 if pos_table is None else pos_table.shape[0]), stream()), "embed_gather")
     return out
 
 

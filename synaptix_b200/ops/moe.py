@@ -13,6 +13,9 @@ from ._lib import KernelError, c_float, c_int, check, dt_code, fn, ptr, require_
 # sorted order first); fewer rows (single-token steps, short prompts) run the mma.sync kernel, which gathers as it loads.
 TC_MIN_ROWS = 512
 
+# what a grouped product does (see csrc/moe.cu)
+MODE_PLAIN, MODE_GATE_UP, MODE_UP = 0, 1, 2
+
 
 def _tc_fits(rows: int, K: int, dtype) -> bool:
     return dtype == torch.bfloat16 and rows >= TC_MIN_ROWS and K % 8 == 0
@@ -89,12 +92,37 @@ def moe_gate_up(x: torch.Tensor, gate_up: torch.Tensor, plan: ExpertPlan, top: i
         use_gate("moe_tc")
         check(fn("moe_tc", "sx_moe_gather")(ptr(x), ptr(plan.order), ptr(xs), c_int(rows), c_int(W), c_int(top), stream()), "moe_gather")
         check(fn("moe_tc", "sx_moe_tc")(ptr(xs), ptr(gate_up), ptr(z), ptr(plan.offsets), c_int(rows), c_int(E), c_int(ff2 // 2),
-                                        c_int(W), c_int(1), stream()), "moe_gate_up")
+                                        c_int(W), c_int(MODE_GATE_UP), stream()), "moe_gate_up")
         return z
     use_gate("moe")
     check(fn("moe", "sx_moe_gemm")(ptr(x), ptr(gate_up), ptr(z), ptr(plan.offsets), ptr(plan.order), c_int(rows), c_int(E),
-                                   c_int(ff2 // 2), c_int(W), c_int(top), c_int(1), c_int(dt_code(x.dtype)),
+                                   c_int(ff2 // 2), c_int(W), c_int(top), c_int(MODE_GATE_UP), c_int(dt_code(x.dtype)),
                                    c_int(dt_code(z.dtype)), stream()), "moe_gate_up")
+    return z
+
+
+def moe_up(x: torch.Tensor, up: torch.Tensor, plan: ExpertPlan, top: int) -> torch.Tensor:
+    """Experts without a gate: ``act(x_t Wu_e^T)`` for every pair in sorted order, ``act`` the activation in force
+    (``gate_activation(form="relu2")``: ``relu(z)^2``); ``up [experts, ff, width]``; returns ``[pairs, ff]`` in ``x``'s
+    dtype."""
+    require_cuda(x, up)
+    T, W = x.shape
+    E, ff, W2 = up.shape
+    if W2 != W or E != plan.experts or up.dtype != x.dtype:
+        raise KernelError("moe_up: sizes or dtypes do not fit")
+    rows = plan.order.numel()
+    z = torch.empty((rows, ff), dtype=x.dtype, device=x.device)
+    if _tc_fits(rows, W, x.dtype):
+        xs = torch.empty((rows, W), dtype=x.dtype, device=x.device)
+        use_gate("moe_tc")
+        check(fn("moe_tc", "sx_moe_gather")(ptr(x), ptr(plan.order), ptr(xs), c_int(rows), c_int(W), c_int(top), stream()), "moe_gather")
+        check(fn("moe_tc", "sx_moe_tc")(ptr(xs), ptr(up), ptr(z), ptr(plan.offsets), c_int(rows), c_int(E), c_int(ff), c_int(W),
+                                        c_int(MODE_UP), stream()), "moe_up")
+        return z
+    use_gate("moe")
+    check(fn("moe", "sx_moe_gemm")(ptr(x), ptr(up), ptr(z), ptr(plan.offsets), ptr(plan.order), c_int(rows), c_int(E), c_int(ff),
+                                   c_int(W), c_int(top), c_int(MODE_UP), c_int(dt_code(x.dtype)), c_int(dt_code(z.dtype)),
+                                   stream()), "moe_up")
     return z
 
 
@@ -108,10 +136,10 @@ def moe_down(z: torch.Tensor, down: torch.Tensor, plan: ExpertPlan) -> torch.Ten
     y = torch.empty((rows, W), dtype=torch.float32, device=z.device)
     if _tc_fits(rows, ff, z.dtype):
         check(fn("moe_tc", "sx_moe_tc")(ptr(z), ptr(down), ptr(y), ptr(plan.offsets), c_int(rows), c_int(E), c_int(W), c_int(ff),
-                                        c_int(0), stream()), "moe_down")
+                                        c_int(MODE_PLAIN), stream()), "moe_down")
         return y
     check(fn("moe", "sx_moe_gemm")(ptr(z), ptr(down), ptr(y), ptr(plan.offsets), ptr(plan.order), c_int(rows), c_int(E),
-                                   c_int(W), c_int(ff), c_int(1), c_int(0), c_int(dt_code(z.dtype)), c_int(dt_code(y.dtype)),
+                                   c_int(W), c_int(ff), c_int(1), c_int(MODE_PLAIN), c_int(dt_code(z.dtype)), c_int(dt_code(y.dtype)),
                                    stream()), "moe_down")
     return y
 

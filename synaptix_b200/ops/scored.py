@@ -16,9 +16,10 @@ def heads_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], q_out: torch
                   v_pages: Optional[torch.Tensor], positions: torch.Tensor, seq_of_token: torch.Tensor,
                   block_table: torch.Tensor, H: int, G: int, dim: int, vdim: int, *, q_gain=None, k_gain=None,
                   eps: float = 0.0, inv_freq=None, rot_dims: int = 0, magnitude: float = 1.0, v_first_in=None,
-                  v_first_out=None, lam=None, gate_out=None) -> None:
+                  v_first_out=None, lam=None, gate_out=None, q_temp=None) -> None:
     """``proj`` float32 ``[T, >= (H + G) dim + G vdim + gates]``: q heads, k heads, v heads, then one gate column per
-    entry of ``gate_out``'s row.  See the kernel's comment for what is done to each."""
+    entry of ``gate_out``'s row.  ``q_temp = (coef, every)``: the queries of position ``p`` are multiplied by
+    ``1 + coef ln(floor((p + 1) / every) + 1)``.  See the kernel's comment for what is done to each."""
     require_cuda(proj, bias, q_out, k_pages, v_pages, positions, seq_of_token, block_table, q_gain, k_gain, inv_freq,
                  v_first_in, v_first_out, lam, gate_out)
     if proj.dtype != torch.float32:
@@ -42,6 +43,7 @@ def heads_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], q_out: torch
         ptr(seq_of_token), ptr(block_table), c_int(block_table.shape[1]), c_int(n_pages), c_int(T), c_int(H), c_int(G),
         c_int(dim), c_int(vdim), ptr(q_gain), ptr(k_gain), c_float(eps), ptr(inv_freq), c_int(rot_dims if inv_freq is not None else 0),
         c_float(magnitude), ptr(v_first_in), ptr(v_first_out), ptr(lam), ptr(gate_out), c_int(n_gate),
+        c_int(0 if q_temp is None else int(q_temp[1])), c_float(0.0 if q_temp is None else float(q_temp[0])),
         c_int(dt_code(q_out.dtype)), stream()), "heads_prepare")
 
 

@@ -17,6 +17,9 @@ norm of its own and times a learned vector over the width (a layer scale):
 row's root mean square, so one kernel makes both; the sum is handed on as a
 ``ScaledSum`` and added by the next norm's kernel.  The feed-forward half may be absent.
 
+A ``ParallelBlock`` may also have ONE norm that both sublayers read (``norm2=None`` with a feed-forward), no layer scales
+(``scale_names=None``), and an input of the token of its own behind the sum (``side``, a ``TokenSide``).
+
 ``SandwichBlock``: every sublayer between two norms, ``h += mult * post(sublayer(pre(h)))``,
 with an optional ``TokenShift`` of what the mixer reads.
 
@@ -134,7 +137,10 @@ def _side_stream(device) -> "torch.cuda.Stream":
 class ParallelBlock(Part):
     """``h += mult * (ls1 * mixer(norm1(h)) + ls2 * ffn(norm2(h)))``, both branches of the same ``h``.  ``norm1`` and
     ``norm2`` are RMS norms (their gains may differ, their eps not); ``scale_names`` are the tensors ``ls1`` and
-    ``ls2`` (vectors over the width).  ``norm2`` and ``ffn`` may both be ``None``.
+    ``ls2`` (vectors over the width; ``None``: no layer scales).  ``ffn`` may be ``None``, and then ``norm2`` is; with
+    ``norm2=None`` and a feed-forward both sublayers read ``norm1(h)``.  ``side``: a layer's own input of the token
+    (``TokenSide``), formed from the stream behind the sum; its branch, which has a norm of its own, is then what the
+    block hands on.
 
     The branches do not depend on each other.  In single-token steps, where a layer is a chain of small kernels, the
     feed-forward runs on a second stream (option ``branch_streams``): it begins behind the norm kernel (an event) and the
@@ -146,28 +152,35 @@ class ParallelBlock(Part):
     takes_pending_product = False
 
     def __init__(self, norm1: Norm, mixer: Mixer, norm2: Optional[Norm], ffn: Optional[FeedForward], *,
-                 scale_names: Tuple[str, str], mult: float = 1.0):
-        if (norm2 is None) != (ffn is None):
-            raise ValueError("norm2 and ffn come together or not at all")
+                 scale_names: Optional[Tuple[str, str]] = None, mult: float = 1.0, side: Optional[Part] = None):
+        if norm2 is not None and ffn is None:
+            raise ValueError("norm2 comes with a feed-forward")
         if norm2 is not None and norm2.eps != norm1.eps:
             raise ValueError("the two norms of a parallel block share their eps")
         self.norm1, self.mixer, self.norm2, self.ffn = norm1, mixer, norm2, ffn
-        self.scale_names = tuple(scale_names)
+        self.scale_names = None if scale_names is None else tuple(scale_names)
         self.mult = float(mult)
+        if self.scale_names is None and self.mult != 1.0:
+            raise ValueError("a factor on the sum is folded into the layer scales")
+        self.side = side
         self.width = norm1.width
         self.s1: Optional[torch.Tensor] = None
         self.s2: Optional[torch.Tensor] = None
 
     def children(self) -> List[Part]:
-        return [p for p in (self.norm1, self.mixer, self.norm2, self.ffn) if p is not None]
+        return [p for p in (self.norm1, self.mixer, self.norm2, self.ffn, self.side) if p is not None]
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
+        if self.scale_names is None:
+            return {}
         specs = {self.scale_names[0]: TensorSpec((self.width,), "gain")}
         if self.ffn is not None:
             specs[self.scale_names[1]] = TensorSpec((self.width,), "gain")
         return specs
 
     def bind(self, tensors: Mapping[str, torch.Tensor], rt: Runtime) -> None:
+        if self.scale_names is None:
+            return
         # mult * (ls1 * a + ls2 * b) as (mult ls1) * a + (mult ls2) * b, the factors formed once in 32-bit
         self.s1 = to_device_f32(tensors[self.scale_names[0]].to(torch.float32) * self.mult, rt)
         if self.ffn is not None:
@@ -176,31 +189,51 @@ class ParallelBlock(Part):
     def cache_request(self):
         return self.mixer.cache_request()
 
-    def forward(self, h: torch.Tensor, pending, ctx: StepContext, cache_view, write_cache: bool = True):
+    def _read(self, h: torch.Tensor, pending, dtype):
+        """``h += pending`` and what the two sublayers read of it (the same rows where they share a norm)."""
+        gains = [self.norm1.weight] + ([self.norm2.weight] if self.norm2 is not None else [])
+        if isinstance(pending, NormedDelta) and pending.is_rms and pending.norm.eps == self.norm1.eps and len(gains) == 1:
+            # a branch with a norm of its own: its norm, the sum and this block's norm in one kernel
+            terms, factor = pending.rms_terms()
+            x = ops.add_normed(h, terms, pending.norm.weight, self.norm1.eps, dtype, factor=factor, out_gain=gains[0])
+            return x, x
         if isinstance(pending, ScaledSum):
             terms = pending.terms
         else:
             pending = plain(pending)
             terms = [] if pending is None else [(pending, None)]
-        gains = [self.norm1.weight] + ([self.norm2.weight] if self.ffn is not None else [])
-        xs = ops.add_scaled_rmsnorm(h, terms, gains, self.norm1.eps, ctx.runtime.dtype)
+        xs = ops.add_scaled_rmsnorm(h, terms, gains, self.norm1.eps, dtype)
+        return xs[0], xs[-1]
+
+    def _ffn(self, x: torch.Tensor, ctx: StepContext):
+        # the sum behind a block with a side input can form a mixture's weighted sum on its way
+        if self.side is not None and getattr(self.ffn, "can_defer_combine", False):
+            return self.ffn.forward(x, ctx, defer_combine=True)
+        return self.ffn.forward(x, ctx)
+
+    def forward(self, h: torch.Tensor, pending, ctx: StepContext, cache_view, write_cache: bool = True):
+        x1, x2 = self._read(h, pending, ctx.runtime.dtype)
         if self.ffn is None:
-            return h, ScaledSum([(self.mixer.forward(xs[0], ctx, cache_view, write_cache), self.s1)])
-        if ctx.all_single and ops.OPTIONS.branch_streams and h.is_cuda:
-            main, side = torch.cuda.current_stream(h.device), _side_stream(h.device)
-            fork = torch.cuda.Event()
-            fork.record(main)
-            side.wait_event(fork)
-            with torch.cuda.stream(side):
-                b = self.ffn.forward(xs[1], ctx)
-                join = torch.cuda.Event()
-                join.record(side)
-            a = self.mixer.forward(xs[0], ctx, cache_view, write_cache)
-            main.wait_event(join)
+            terms = [(self.mixer.forward(x1, ctx, cache_view, write_cache), self.s1)]
         else:
-            a = self.mixer.forward(xs[0], ctx, cache_view, write_cache)
-            b = self.ffn.forward(xs[1], ctx)
-        return h, ScaledSum([(a, self.s1), (b, self.s2)])
+            if ctx.all_single and ops.OPTIONS.branch_streams and h.is_cuda:
+                main, side = torch.cuda.current_stream(h.device), _side_stream(h.device)
+                fork = torch.cuda.Event()
+                fork.record(main)
+                side.wait_event(fork)
+                with torch.cuda.stream(side):
+                    b = self._ffn(x2, ctx)
+                    join = torch.cuda.Event()
+                    join.record(side)
+                a = self.mixer.forward(x1, ctx, cache_view, write_cache)
+                main.wait_event(join)
+            else:
+                a = self.mixer.forward(x1, ctx, cache_view, write_cache)
+                b = self._ffn(x2, ctx)
+            terms = [(a, self.s1), (b, self.s2)]
+        if self.side is not None:
+            return h, self.side.forward(h, terms, ctx)
+        return h, ScaledSum(terms)
 
 
 class TokenShift(Part):

@@ -7,7 +7,7 @@ the rows asked for and returned in float32.
 """
 from __future__ import annotations
 
-from typing import Dict, Mapping, Optional
+from typing import Dict, Mapping, Optional, Tuple
 
 import torch
 
@@ -18,22 +18,43 @@ from .linear import Linear
 
 
 class Embedding(Part):
-    """``scale``: the gathered rows are multiplied by it (in 32-bit, on their way into the stream)."""
+    """``scale``: the gathered rows are multiplied by it (in 32-bit, on their way into the stream).  ``positions=(name,
+    rows)``: a learned vector per position, ``E[id_t] * scale + P[t]`` (not scaled), is added in the same kernel; a
+    sequence can then be no longer than the table (``max_positions``, which the engine asks of every step)."""
 
-    def __init__(self, weight_name: str, vocab: int, width: int, scale: float = 1.0):
+    def __init__(self, weight_name: str, vocab: int, width: int, scale: float = 1.0,
+                 positions: Optional[Tuple[str, int]] = None):
         self.weight_name, self.vocab, self.width = weight_name, vocab, width
         self.scale = float(scale)
+        self.position_name, self.position_rows = positions if positions is not None else (None, 0)
         self.weight: Optional[torch.Tensor] = None
+        self.position_table: Optional[torch.Tensor] = None
+
+    @property
+    def max_positions(self) -> Optional[int]:
+        """How many tokens a sequence can have (``None``: no limit)."""
+        return self.position_rows if self.position_name is not None else None
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
-        return {self.weight_name: TensorSpec((self.vocab, self.width), "embedding")}
+        specs = {self.weight_name: TensorSpec((self.vocab, self.width), "embedding")}
+        if self.position_name is not None:
+            specs[self.position_name] = TensorSpec((self.position_rows, self.width), "embedding")
+        return specs
 
     def bind(self, tensors: Mapping[str, torch.Tensor], rt: Runtime) -> None:
         self.weight = to_device_matrix(tensors[self.weight_name], rt)
+        if self.position_name is not None:
+            self.position_table = to_device_matrix(tensors[self.position_name], rt)
 
-    def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
-        """float32 residual stream ``[T, width]``."""
-        return ops.embed_gather(self.weight, token_ids, scale=self.scale)
+    def forward(self, token_ids: torch.Tensor, positions: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """float32 residual stream ``[T, width]``; ``positions`` (int32 ``[T]``) only where there is a position table."""
+        if self.position_table is None:
+            return ops.embed_gather(self.weight, token_ids, scale=self.scale)
+        return ops.embed_gather(self.weight, token_ids, scale=self.scale, pos_table=self.position_table, positions=positions)
+
+    def forward_step(self, ctx, state: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """The step's residual stream; ``state`` is the cache entry of an embedding that has one."""
+        return self.forward(ctx.token_ids, ctx.positions)
 
 
 class BigramEmbedding(Embedding):
@@ -61,7 +82,7 @@ class BigramEmbedding(Embedding):
         from ..cache.store import StateRequest
         return StateRequest((), torch.int32)
 
-    def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
+    def forward(self, token_ids: torch.Tensor, positions: Optional[torch.Tensor] = None) -> torch.Tensor:
         raise TypeError("an embedding with a state is called with the step: forward_step(ctx, state)")
 
     def forward_step(self, ctx, state: torch.Tensor) -> torch.Tensor:

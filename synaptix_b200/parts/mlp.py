@@ -13,7 +13,8 @@ are) and multiplied by ``scale``; the result is the weighted sum of the chosen e
 choice: ``correction`` (a tensor of one number per expert, added to the scores for the choice only; the weights use
 the scores without it) and ``groups=(count, keep)`` (the experts form ``count`` equal groups of neighbours, a group's
 value is the sum of its two largest choice values, only experts of the ``keep`` best groups can be chosen).
-``activation=(alpha, limit)`` makes the experts ``CappedGLU``s instead of SwiGLUs.
+``activation=(alpha, limit)`` makes the experts ``CappedGLU``s instead of SwiGLUs; ``gated=False`` makes them
+``down( relu(x Wu^T)^2 )``, two matrices and no gate.
 The tokens are sorted by expert on the device and each expert's rows run as one group of a grouped product.
 """
 from __future__ import annotations
@@ -93,11 +94,13 @@ class MixtureOfExperts(FeedForward):
     def __init__(self, prefix: str, width: int, intermediate: int, experts: int, top: int, *, scale: float = 1.0,
                  scoring: str = "softmax", renormalize: bool = True, correction: bool = False,
                  groups: Optional[Tuple[int, int]] = None, activation: Optional[Tuple[float, float]] = None,
-                 names: Optional[Mapping[str, str]] = None):
+                 gated: bool = True, names: Optional[Mapping[str, str]] = None):
         if not 0 < top <= experts:
             raise ValueError("0 < top <= experts")
         if scoring not in ("softmax", "sigmoid"):
             raise ValueError("scoring is softmax or sigmoid")
+        if activation is not None and not gated:
+            raise ValueError("the capped activation is a gated one")
         if groups is not None:
             count, keep = groups
             if count <= 0 or experts % count or not 0 < keep <= count or top > keep * (experts // count):
@@ -107,10 +110,11 @@ class MixtureOfExperts(FeedForward):
         self.scoring, self.renormalize, self.has_correction = scoring, bool(renormalize), bool(correction)
         self.groups = None if groups is None else (int(groups[0]), int(groups[1]))
         self.activation = None if activation is None else (float(activation[0]), float(activation[1]))
+        self.gated = bool(gated)
         self.correction: Optional[torch.Tensor] = None  # float32 [experts]
         self.names = dict(self.NAMES, **(names or {}))
         self.router: Optional[torch.Tensor] = None      # float32 [experts, width]
-        self.gate_up: Optional[torch.Tensor] = None     # [experts, 2 * intermediate, width]: gate rows, then up rows
+        self.gate_up: Optional[torch.Tensor] = None     # [experts, 2 * intermediate, width]: gate rows, then up rows (no gate rows without a gate)
         self.down: Optional[torch.Tensor] = None        # [experts, width, intermediate]
 
     def _name(self, e: int, which: str) -> str:
@@ -121,7 +125,8 @@ class MixtureOfExperts(FeedForward):
         if self.has_correction:
             specs[self.prefix + self.names["correction"]] = TensorSpec((self.experts,), "bias")
         for e in range(self.experts):
-            specs[self._name(e, "gate")] = TensorSpec((self.intermediate, self.width), "matrix")
+            if self.gated:
+                specs[self._name(e, "gate")] = TensorSpec((self.intermediate, self.width), "matrix")
             specs[self._name(e, "up")] = TensorSpec((self.intermediate, self.width), "matrix")
             specs[self._name(e, "down")] = TensorSpec((self.width, self.intermediate), "matrix")
         return specs
@@ -130,7 +135,8 @@ class MixtureOfExperts(FeedForward):
         self.router = to_device_f32(tensors[self.prefix + self.names["router"]], rt)
         if self.has_correction:
             self.correction = to_device_f32(tensors[self.prefix + self.names["correction"]], rt)
-        gu = [torch.cat([tensors[self._name(e, "gate")], tensors[self._name(e, "up")]], dim=0) for e in range(self.experts)]
+        parts = ("gate", "up") if self.gated else ("up",)
+        gu = [torch.cat([tensors[self._name(e, n)] for n in parts], dim=0) for e in range(self.experts)]
         self.gate_up = to_device_matrix(torch.stack(gu), rt)
         self.down = to_device_matrix(torch.stack([tensors[self._name(e, "down")] for e in range(self.experts)]), rt)
 
@@ -140,7 +146,10 @@ class MixtureOfExperts(FeedForward):
         ids, weights = ops.moe_route(x, self.router, self.top, self.scale, self.SUM_EPS, scoring=self.scoring,
                                      correction=self.correction, groups=self.groups, renormalize=self.renormalize)
         plan = ops.moe_sort(ids, self.experts)
-        if self.activation is not None:
+        if not self.gated:
+            with ops.gate_activation(form="relu2"):              # the grouped up product's epilogue applies it
+                z = ops.moe_up(x, self.gate_up, plan, self.top)
+        elif self.activation is not None:
             with ops.gate_activation(*self.activation):          # the grouped gate/up product's epilogue applies it
                 z = ops.moe_gate_up(x, self.gate_up, plan, self.top)
         else:

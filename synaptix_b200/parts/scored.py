@@ -2,7 +2,8 @@
 
 ``q, k, v = Wq x (+ bq), Wk x (+ bk), Wv x (+ bv)``; per-head RMS norm of q and k with one gain shared by all heads
 (optional); rotation of neighbouring pairs of the first elements of a head (optional, any ``PositionEncoding`` that
-says ``pairs``); then, for the query at position ``i`` and the key at ``j`` (visible iff ``0 <= i - j < window``):
+says ``pairs``); queries times a temperature of their position (``q_temp=(coef, every)``:
+``1 + coef ln(floor((p + 1) / every) + 1)`` at position ``p``; optional); then, for the query at position ``i`` and the key at ``j`` (visible iff ``0 <= i - j < window``):
 
 * ``talk``: the heads' scaled scores are mixed, ``s'_h = sum_g T[h, g] s_g`` with a learned ``[H, H]``;
 * ``head_bias``: a learned number per head is added; ``distance_bias=(rows, far)``: a learned table ``[rows, H]`` gives
@@ -57,6 +58,7 @@ class ScoredAttention(Mixer):
                  biases: bool = False, qk_norm_eps: Optional[float] = None, talk: bool = False, head_bias: bool = False,
                  distance_bias: Optional[Tuple[int, float]] = None, weights: str = "softmax",
                  value_mix: Optional[str] = None, value_key: str = "values", head_gate: bool = False,
+                 q_temp: Optional[Tuple[float, int]] = None,
                  names: Optional[Mapping[str, str]] = None):
         if n_heads % n_kv_heads:
             raise ValueError("n_heads must be a multiple of n_kv_heads")
@@ -74,6 +76,9 @@ class ScoredAttention(Mixer):
         self.talk, self.head_bias, self.distance_bias = bool(talk), bool(head_bias), distance_bias
         self.softmax = weights == "softmax"
         self.value_mix, self.value_key, self.head_gate = value_mix, value_key, bool(head_gate)
+        if q_temp is not None and q_temp[1] <= 0:
+            raise ValueError("q_temp is (coefficient, positions a step), the second > 0")
+        self.q_temp = q_temp
         self.names = n = dict(self.NAMES, **(names or {}))
         parts = [(prefix + n["q"], n_heads * head_dim), (prefix + n["k"], n_kv_heads * head_dim),
                  (prefix + n["v"], n_kv_heads * v_head_dim)]
@@ -156,7 +161,7 @@ class ScoredAttention(Mixer):
                           self.hd, self.vd, q_gain=self.q_gain, k_gain=self.k_gain,
                           eps=self.qk_norm_eps if self.qk_norm_eps is not None else 0.0, inv_freq=inv_freq,
                           rot_dims=rot_dims, magnitude=getattr(self.position, "magnitude", 1.0), v_first_in=v_in,
-                          v_first_out=v_out, lam=self.lam, gate_out=gate)
+                          v_first_out=v_out, lam=self.lam, gate_out=gate, q_temp=self.q_temp)
         a = ops.attn_scored(q, cache_view.k, cache_view.v, ctx, bt, self.nh, self.nkv, self.hd, self.vd, self.scale,
                             self.window, talk=self.talk_matrix, head_bias=self.head_bias_vector,
                             dist_bias=self.distance_table, softmax=self.softmax, gate=gate)
