@@ -295,9 +295,27 @@ def tamovik_config(width, ff, nh, nkv, hd, rh, runs, vocab):
                 embedding=dict(bigram=dict(buckets=vocab - 1, mul_prev=8191, mul_cur=131)), layers=layers)
 
 
+def zekalorn_config(width, ff, nh, nkv, hd, rh, runs, vocab):
+    """``runs`` layer runs: layers (channel_delta, channel_delta, attention) repeated, the first two run twice (a loop).
+    Delta layers: ``2 rh`` heads of ``hd x hd`` with 4 taps and low-rank projections of rank ``hd``; attention: grouped heads
+    of ``hd``, every earlier key visible, a distance table of 32 buckets up to 512, a temperature on the queries; a token
+    input of 256 elements a layer.  The first layer's feed-forward is dense (``ff``), the others have 16 experts of two
+    matrices of ``3/8 ff``, 4 a token (as many active weights as the dense one)."""
+    delta = dict(heads=2 * rh, kv_heads=2 * rh, dim=hd, vdim=hd, conv=4, decay_rank=hd, gate_rank=hd)
+    att = dict(heads=nh, kv_heads=nkv, dim=hd, vdim=hd, scale=hd ** -0.5, bias_max=512, bias_rows=32,
+               q_temp=dict(coef=0.1, every=1024))
+    moe = dict(kind="moe", expert=dict(ff=3 * ff // 8), router=dict(experts=16, top=4))
+    layers = []
+    for i in range(runs - 2):
+        mlp = dict(kind="dense", ff=ff) if i == 0 else moe
+        layers.append(dict(type="attention", mixer=att, mlp=mlp) if i % 3 == 2 else dict(type="channel_delta", mixer=delta, mlp=mlp))
+    return dict(architecture="Zekalorn", vocab=vocab, width=width, norm=dict(eps=1e-5), embedding=dict(scale=1.0),
+                max_positions=8192, token_side=dict(dim=256), loop=dict(start=0, stop=2, times=2), layers=layers)
+
+
 def arch_points(torch, a):
     from synaptix_b200.api import LLM
-    from synaptix_b200.config import LedudraConfig, PidutarConfig, Qwen3Config, TamovikConfig, VemedraConfig
+    from synaptix_b200.config import LedudraConfig, PidutarConfig, Qwen3Config, TamovikConfig, VemedraConfig, ZekalornConfig
     from synaptix_b200.engine import DecodeRow, Entry
     from synaptix_b200.models import model_skeleton
     from synaptix_b200.parts import Runtime
@@ -358,9 +376,13 @@ def arch_points(torch, a):
         width, ff, nh, nkv, hd, rh = VEMEDRA_SIZES[name]
         if a.arch == "tamovik":
             measure(TamovikConfig.from_dict(tamovik_config(width, ff, nh, nkv, hd, rh, RUNS, VOCAB)), f"tamovik_{name}")
-        if a.arch in ("pidutar", "tamovik"):
+        if a.arch == "zekalorn":
+            measure(ZekalornConfig.from_dict(zekalorn_config(width, ff, nh, nkv, hd, rh, RUNS, VOCAB)), f"zekalorn_{name}")
+        if a.only:
+            continue
+        if a.arch in ("pidutar", "tamovik", "zekalorn"):
             measure(PidutarConfig.from_dict(pidutar_config(width, ff, nh, nkv, hd, rh, RUNS, VOCAB)), f"pidutar_{name}")
-        if a.arch == "tamovik":
+        if a.arch in ("tamovik", "zekalorn"):
             pass
         elif a.arch == "ledudra":
             measure(LedudraConfig.from_dict(ledudra_config(width, ff, nh, nkv, hd, rh, RUNS, VOCAB)), f"ledudra_{name}")
@@ -370,7 +392,7 @@ def arch_points(torch, a):
                                            num_key_value_heads=nkv, head_dim=hd, intermediate_size=ff, vocab_size=VOCAB,
                                            tie_word_embeddings=False)), f"qwen3_{name}")
     beside = {"pidutar": "Pidutar beside Vemedra and", "vemedra": "Vemedra beside", "ledudra": "Ledudra beside",
-              "tamovik": "Tamovik beside Pidutar and"}[a.arch]
+              "tamovik": "Tamovik beside Pidutar and", "zekalorn": "Zekalorn beside Pidutar and"}[a.arch]
     return {"metric": f"prompt step and decode step, {beside} Qwen3 at equal sizes (bf16, random weights)", "impl": "ours",
             "layer_runs": RUNS, "vocab": VOCAB, "context": CONTEXT, "steps": K, "warmup": a.warmup, "sizes": VEMEDRA_SIZES,
             "data": "synthetic", "dtype": "bf16", "points": out}
@@ -397,11 +419,12 @@ def main():
     ap.add_argument("--short", action="store_true",
                     help="decode only 5 x --steps + --warmup tokens instead of at least 255 (small cases for profilers: "
                          "every launch under a profiler costs a good part of a second)")
-    ap.add_argument("--arch", default="qwen3", choices=["qwen3", "vemedra", "pidutar", "ledudra", "tamovik"],
+    ap.add_argument("--arch", default="qwen3", choices=["qwen3", "vemedra", "pidutar", "ledudra", "tamovik", "zekalorn"],
                     help="vemedra: the Vemedra decoder beside Qwen3 at equal sizes (prompt step, decode at batch 1 and 8) instead of "
                          "the default run; pidutar: the Pidutar decoder beside both; ledudra: the Ledudra decoder beside Qwen3; "
-                         "tamovik: the Tamovik decoder beside Pidutar and Qwen3")
-    ap.add_argument("--arch-sizes", default="", help="with --arch vemedra, pidutar, ledudra or tamovik: which of 1k,2.5k,4k (default: all)")
+                         "tamovik / zekalorn: that decoder beside Pidutar and Qwen3")
+    ap.add_argument("--arch-sizes", default="", help="with another --arch than qwen3: which of 1k,2.5k,4k (default: all)")
+    ap.add_argument("--only", action="store_true", help="with --arch tamovik or zekalorn: that decoder alone (for profilers)")
     a = ap.parse_args()
 
     if a.impl == "reference":
@@ -415,7 +438,7 @@ def main():
     a.warmup = max(a.warmup, 3)
 
     import torch
-    if a.arch in ("vemedra", "pidutar", "ledudra", "tamovik"):
+    if a.arch != "qwen3":
         a.steps = min(a.steps, 40)
         print(json.dumps(arch_points(torch, a)))
         return 0

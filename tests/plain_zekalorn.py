@@ -64,15 +64,15 @@ def time_conv(u, taps):
 
 
 def delta_rule(q, k, v, decay, beta):
-    """One head: ``q, k, decay [T, D]``, ``v [T, V]``, ``beta [T]`` -> ``o [T, V]``; the state starts at zero."""
-    T, D = k.shape
-    S = torch.zeros(D, v.shape[1], dtype=F)
-    out = torch.zeros(T, v.shape[1], dtype=F)
+    """``q, k, decay [T, H, D]``, ``v [T, H, V]``, ``beta [T, H]`` -> ``o [T, H, V]``; every head's state starts at zero."""
+    T, H, D = k.shape
+    S = torch.zeros(H, D, v.shape[2], dtype=F)
+    out = torch.zeros(T, H, v.shape[2], dtype=F)
     for t in range(T):
-        S = decay[t][:, None] * S
-        u = beta[t] * (v[t] - S.T @ k[t])
-        S = S + torch.outer(k[t], u)
-        out[t] = S.T @ q[t]
+        S = decay[t][:, :, None] * S
+        u = beta[t][:, None] * (v[t] - (S * k[t][:, :, None]).sum(1))
+        S = S + k[t][:, :, None] * u[:, None, :]
+        out[t] = (S * q[t][:, :, None]).sum(1)
     return out
 
 
@@ -94,11 +94,8 @@ def channel_delta(x, w, p, m, eps):
     T = x.shape[0]
     H, G, V = m["heads"], m["kv_heads"], m["vdim"]
     q, k, v, decay, beta = delta_inputs(x, w, p, m)
-    heads = []
-    for h in range(H):
-        g = h // (H // G)
-        heads.append(delta_rule(q[:, g], k[:, g], v[:, h], decay[:, h], beta[:, h]))
-    o = torch.stack(heads, 1)                                     # [T, H, V]
+    of_head = [h // (H // G) for h in range(H)]                   # the query/key head each head reads
+    o = delta_rule(q[:, of_head], k[:, of_head], v, decay, beta)
     gate = torch.sigmoid((x @ w[p + "g1"].to(F).T) @ w[p + "g2"].to(F).T).reshape(T, H, V)
     y = unit_rms(o, eps) * w[p + "norm"].to(F) * gate
     return y.reshape(T, H * V) @ w[p + "o"].to(F).T
