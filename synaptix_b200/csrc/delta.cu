@@ -24,9 +24,9 @@
 //                         b v (so u = Y - X S_0), the weights P_ts = q_t . e^(G_t - G_s) k_s (s <= t), e^(G_t) q_t,
 //                         e^(G_end - G_t) k_t and e^(G_end).  No exponent is ever positive: pairs of tokens within 16 take
 //                         e^(G_t - G_s) itself, pairs across take it in two factors around the border between them.
-//     delta_scan_kernel   a block a (slice of V, head, sequence) walks the chunks: u = Y - X S, o = (e^G q) S + P u,
-//                         S <- diag(e^(G_end)) S + (e^(G_end - G) k)^T u.
-//     delta_finish_kernel a warp a (token, head): output norm, gain, gate.
+//     delta_scan_kernel   a block a (slice of V, head, sequence) walks the chunks: u = Y - X S (left in Y's place), the state
+//                         at the chunk's begin (left for the next kernel), S <- diag(e^(G_end)) S + (e^(G_end - G) k)^T u.
+//     delta_out_kernel    a block a (chunk, head): o = (e^G q) S_begin + P u, output norm, gain, gate.
 #include "common.cuh"
 
 #define DL_THREADS 256
@@ -42,6 +42,15 @@ __device__ __forceinline__ float dl_exp2(float x) {
   return y;
 }
 #define DL_LOG2E 1.4426950408889634f
+// A decay below 2^-40 empties its channel as far as 32-bit sums can tell (1e-12 of the state stays).  In the chunks the
+// logarithms are cut off there, and they are summed from the begin of each half of a chunk: a difference of two running
+// sums, of which decays between two tokens are made, then keeps its last bits whatever strong decays came before.
+#define DL_LOG_MIN -40.f
+__device__ __forceinline__ void dl_cp16(float* smem, const float* gmem) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+__device__ __forceinline__ void dl_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
+template <int N> __device__ __forceinline__ void dl_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
 
 struct DlArgs {
   const void* proj; int row, col, b_col;     // q, k, v columns from col on (2 G D + H V of them), step sizes' from b_col on
@@ -142,22 +151,34 @@ template <int CPL> struct DlLd<bf16, CPL> {
   }
 };
 
+// the activation where the result is rounded to 16 bits' worth anyway (bfloat16 projections), and the precise one
+template <typename T> __device__ __forceinline__ float dl_silu_of(float z);
+template <> __device__ __forceinline__ float dl_silu_of<float>(float z) { return dl_silu(z); }
+template <> __device__ __forceinline__ float dl_silu_of<bf16>(float z) { return __fdividef(z, 1.f + __expf(-z)); }
+
 template <typename T, int CPL, int TAPS>
 __device__ __forceinline__ void dl_prepare_run(const DlArgs& a, const DlPrep& w, int t0, int t1, int unit, int c0, int kind, int lane) {
   const int C = 2 * a.G * a.D + a.H * a.V, c = c0 + lane * CPL;
   const T* src = (const T*)a.proj + a.col + c;
   float wt[CPL][TAPS], win[TAPS][CPL];            // win[j]: the row that tap j reads
+  float raw[DL_RUN][CPL];                         // the run's rows, all asked for at once
+  int seqs[DL_RUN];
+#pragma unroll
+  for (int r = 0; r < DL_RUN; ++r) {
+    const int t = min(t0 + r, t1 - 1);
+    seqs[r] = a.seq_of_token[t];
+    DlLd<T, CPL>::go(src + (size_t)t * a.row, raw[r]);
+  }
 #pragma unroll
   for (int i = 0; i < CPL; ++i)
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) wt[i][j] = a.taps_w[(size_t)(c + i) * TAPS + j];
-  int seq = -1, pos = 0;
-  for (int t = t0; t < t1; ++t) {
-    const int s = a.seq_of_token[t];
-    if (s != seq) {                               // the run's first token, or another sequence's: fetch the rows before it
-      seq = s;
-      pos = a.positions[t];
-      const int past = a.seq_past[s];
+#pragma unroll
+  for (int r = 0; r < DL_RUN; ++r) {
+    const int t = t0 + r;
+    if (t >= t1) break;
+    if (r == 0 || seqs[r] != seqs[r - 1]) {       // the run's first token, or another sequence's: fetch the rows before it
+      const int s = seqs[r], pos = a.positions[t], past = a.seq_past[s];
       const float* hs = a.hist + (size_t)a.seq_slots[s] * TAPS * C + c;
 #pragma unroll
       for (int j = 0; j < TAPS - 1; ++j) {
@@ -171,21 +192,20 @@ __device__ __forceinline__ void dl_prepare_run(const DlArgs& a, const DlPrep& w,
           dl_ld_f32<CPL>(hs + (size_t)(p % TAPS) * C, win[j + 1]);
         }
       }
-    } else {
-      ++pos;
     }
 #pragma unroll
     for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
       for (int i = 0; i < CPL; ++i) win[j][i] = win[j + 1][i];
-    DlLd<T, CPL>::go(src + (size_t)t * a.row, win[TAPS - 1]);
+#pragma unroll
+    for (int i = 0; i < CPL; ++i) win[TAPS - 1][i] = raw[r][i];
     float y[CPL], ss = 0.f;
 #pragma unroll
     for (int i = 0; i < CPL; ++i) {
       float acc = 0.f;
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) acc = fmaf(wt[i][j], win[j][i], acc);
-      y[i] = dl_silu(acc);
+      y[i] = dl_silu_of<T>(acc);
       ss += y[i] * y[i];
     }
     if (kind != 2) {
@@ -205,7 +225,8 @@ __device__ __forceinline__ void dl_prepare_run(const DlArgs& a, const DlPrep& w,
   }
 }
 
-template <typename T, int TAPS>
+// WIDE: some heads have 256 channels
+template <typename T, int TAPS, bool WIDE>
 __global__ void __launch_bounds__(DL_THREADS) delta_prepare_run_kernel(DlArgs a, DlPrep w, int n_tokens) {
   pdl_wait();
   pdl_trigger();
@@ -218,7 +239,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prepare_run_kernel(DlArgs a,
     case 32: dl_prepare_run<T, 1, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;
     case 64: dl_prepare_run<T, 2, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;
     case 128: dl_prepare_run<T, 4, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;
-    default: dl_prepare_run<T, 8, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;      // 256
+    default: if (WIDE) dl_prepare_run<T, 8, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;
   }
 }
 
@@ -323,8 +344,16 @@ static size_t dl_walk_smem(int D, int V, bool in_place) {
 // V / 4 float4, a thread owns one of them in rows r0, r0 + RP, ... (RP = 1024 / V rows a pass, NI passes).
 // low rank: the second halves of the two low-rank projections run here: wz [H D + H V, ra + rg] (row h D + d: a2 in the
 // first ra columns; row H D + h V + c: g2 in the last rg), their inputs in the projection's columns lr_col .. + ra + rg.
+// staged: this head's rows of it come to shared memory (rows of max(ra, rg) padded to whole 16-byte pieces) ahead of the wait.
+// What no kernel of this layer's chain has written (the state, the ring's earlier rows, constants) is asked for ahead of
+// the wait for the kernel before; the state and the ring were written a step (many launches) ago.
 // ---------------------------------------------------------------------------------------------------------------
-struct DlLowRank { const void* wz; int ra, rg, lr_col; };
+struct DlLowRank { const void* wz; int ra, rg, lr_col, staged; };
+
+template <typename TW> __host__ __device__ __forceinline__ int dl_lr_ld(int ra, int rg) {
+  const int m = ra > rg ? ra : rg, q = 16 / (int)sizeof(TW);
+  return (m + q - 1) / q * q;
+}
 
 // rows dot x: 8 lanes a row, 16-byte loads where the row's start and length allow
 template <typename TW>
@@ -332,6 +361,7 @@ __device__ __forceinline__ float dl_row_dot(const TW* wr, const float* x, int n,
   float acc = 0.f;
   constexpr int VE = 16 / sizeof(TW);
   if (vec) {
+#pragma unroll 2
     for (int e = sub * VE; e < n; e += 8 * VE) {
       if (sizeof(TW) == 2) {
         const uint4 u = *reinterpret_cast<const uint4*>(wr + e);
@@ -355,8 +385,10 @@ __device__ __forceinline__ float dl_row_dot(const TW* wr, const float* x, int n,
   return acc;
 }
 
+#define DL_STEP_CH 4                 // convolved channels a thread: 2 D + V <= 1024
+
 template <typename TP, typename TO, int NI>
-__global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(DlArgs a, DlLowRank lr) {
+__global__ void __launch_bounds__(DL_THREADS, NI <= 16 ? 2 : 1) delta_step_kernel(DlArgs a, DlLowRank lr) {
   extern __shared__ __align__(16) float sm[];
   const int D = a.D, V = a.V, H = a.H, G = a.G;
   float* q = sm;                     // D
@@ -368,6 +400,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(DlArgs a, DlLowR
   float* pr = sm + ((3 * D + 2 * V + lr.ra + lr.rg + 3) & ~3);       // 1024: RP rows of V partial sums
   float* pp = pr + 1024;             // 1024
   float* us = pp + 1024;             // V: updates
+  TO* wsm = (TO*)(us + V);           // (D + V) rows, if staged
   __shared__ float red[33];
   __shared__ float sc[3];
   const int h = blockIdx.x, s = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -375,35 +408,85 @@ __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(DlArgs a, DlLowR
   const int slot = a.seq_slots[s];
   float* Sg = a.S + ((size_t)slot * H + h) * D * V + c4;
   float4 S[NI];
-  // the state was written by a kernel of an earlier step (several launches back): asked for before the wait
 #pragma unroll
   for (int i = 0; i < NI; ++i) {
     const int d = r0 + i * RP;
     S[i] = d < D ? *reinterpret_cast<const float4*>(Sg + (size_t)d * V) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
-  pdl_wait();
-  pdl_trigger();
+  const TO* wz = (const TO*)lr.wz;
+  constexpr int VE = 16 / sizeof(TO);
+  const int ld = lr.ra + lr.rg, wld = dl_lr_ld<TO>(lr.ra, lr.rg);
+  if (lr.staged) {
+    const int pa = lr.ra / VE, pg = lr.rg / VE;
+    const int sub = lane & 15;                       // half a warp a row
+#pragma unroll 4
+    for (int r = warp * 2 + (lane >> 4); r < D + V; r += DL_THREADS / 16) {
+      const bool dec = r < D;
+      const TO* wr = dec ? wz + (size_t)(h * D + r) * ld : wz + (size_t)(H * D + h * V + (r - D)) * ld + lr.ra;
+      for (int e = sub; e < (dec ? pa : pg); e += 16) dl_cp16((float*)(wsm + r * wld + e * VE), (const float*)(wr + e * VE));
+    }
+  }
+  dl_commit();
   const int rep = H / G, gq = h / rep, t = s, pos = a.positions[t], taps = a.taps;
   const int C = 2 * G * D + H * V, GD = G * D;
-  const TP* pj = (const TP*)a.proj + (size_t)t * a.row;
   float* hs = a.hist + (size_t)slot * taps * C;
-  for (int i = tid; i < 2 * D + V; i += DL_THREADS) {
-    const bool is_v = i >= 2 * D;
-    const int c = i < D ? gq * D + i : (is_v ? 2 * GD + h * V + (i - 2 * D) : GD + gq * D + (i - D));
-    const float* wt = a.taps_w + (size_t)c * taps;
-    const float now = to_f32(pj[a.col + c]);
-    float acc = 0.f;
-    for (int j = 0; j < taps - 1; ++j) {
-      const int p = pos - taps + 1 + j;
-      if (p >= 0) acc = fmaf(wt[j], hs[(size_t)(p % taps) * C + c], acc);
+  // the rows before this one: the loads of up to four of them all on their way before any is used
+  float past[DL_STEP_CH], w_now[DL_STEP_CH], hr[DL_STEP_CH][4], hw[DL_STEP_CH][4];
+  int ring[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int p = pos - 1 - j;                       // j + 1 rows back, tap taps - 2 - j
+    ring[j] = (j < taps - 1 && p >= 0) ? p % taps : -1;
+  }
+#pragma unroll
+  for (int x = 0; x < DL_STEP_CH; ++x) {
+    const int i = tid + x * DL_THREADS;
+    w_now[x] = 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) hr[x][j] = hw[x][j] = 0.f;
+    if (i < 2 * D + V) {
+      const int c = i < D ? gq * D + i : (i < 2 * D ? GD + gq * D + (i - D) : 2 * GD + h * V + (i - 2 * D));
+      const float* wt = a.taps_w + (size_t)c * taps;
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (ring[j] >= 0) { hr[x][j] = hs[(size_t)ring[j] * C + c]; hw[x][j] = wt[taps - 2 - j]; }
+      w_now[x] = wt[taps - 1];
     }
-    acc = fmaf(wt[taps - 1], now, acc);
-    if (is_v || h % rep == 0) hs[(size_t)(pos % taps) * C + c] = now;        // the ring's free row
-    const float y = dl_silu(acc);
-    if (i < D) q[i] = y; else if (is_v) v[i - 2 * D] = y; else k[i - D] = y;
+  }
+#pragma unroll
+  for (int x = 0; x < DL_STEP_CH; ++x) {
+    const int i = tid + x * DL_THREADS;
+    past[x] = 0.f;
+    if (taps > 5 && i < 2 * D + V) {                 // more rows than that: the older ones one after the other
+      const int c = i < D ? gq * D + i : (i < 2 * D ? GD + gq * D + (i - D) : 2 * GD + h * V + (i - 2 * D));
+      for (int j = 0; j < taps - 5; ++j) {
+        const int p = pos - taps + 1 + j;
+        if (p >= 0) past[x] = fmaf(a.taps_w[(size_t)c * taps + j], hs[(size_t)(p % taps) * C + c], past[x]);
+      }
+    }
+#pragma unroll
+    for (int j = 3; j >= 0; --j) past[x] = fmaf(hw[x][j], hr[x][j], past[x]);
+  }
+  pdl_wait();
+  pdl_trigger();
+  const TP* pj = (const TP*)a.proj + (size_t)t * a.row;
+#pragma unroll
+  for (int x = 0; x < DL_STEP_CH; ++x) {
+    const int i = tid + x * DL_THREADS;
+    if (i < 2 * D + V) {
+      const bool is_v = i >= 2 * D;
+      const int c = i < D ? gq * D + i : (is_v ? 2 * GD + h * V + (i - 2 * D) : GD + gq * D + (i - D));
+      const float now = to_f32(pj[a.col + c]);
+      if (is_v || h % rep == 0) hs[(size_t)(pos % taps) * C + c] = now;      // the ring's free row
+      const float y = dl_silu(fmaf(w_now[x], now, past[x]));
+      if (i < D) q[i] = y; else if (is_v) v[i - 2 * D] = y; else k[i - D] = y;
+    }
   }
   if (lr.wz)
-    for (int i = tid; i < lr.ra + lr.rg; i += DL_THREADS) xs[i] = to_f32(pj[lr.lr_col + i]);
+    for (int i = tid; i < ld; i += DL_THREADS) xs[i] = to_f32(pj[lr.lr_col + i]);
+  const float beta = dl_sigmoid(to_f32(pj[a.b_col + h]));
+  const float ea = expf(a.a_log[h]);
+  dl_wait<0>();
   __syncthreads();
   if (warp == 0) {
     float sq = 0.f, sk = 0.f, kq = 0.f;
@@ -412,15 +495,13 @@ __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(DlArgs a, DlLowR
     const float fq = rsqrtf(sq + a.unit_eps) * a.q_scale, fk = rsqrtf(sk + a.unit_eps);
     if (lane == 0) { sc[0] = fq; sc[1] = fk; sc[2] = kq * fq * fk; }
   }
-  const float ea = expf(a.a_log[h]);
   if (lr.wz) {
-    const TO* wz = (const TO*)lr.wz;
-    const int ld = lr.ra + lr.rg, grp = tid >> 3, sub = tid & 7;
-    constexpr int VE = 16 / sizeof(TO);
+    const int grp = tid >> 3, sub = tid & 7;
     const bool va = lr.ra % VE == 0 && lr.rg % VE == 0;
+#pragma unroll 2
     for (int r = grp; r < D + V; r += DL_THREADS / 8) {           // D + V is a multiple of the warps' 4 rows (checked by the host)
       const bool dec = r < D;
-      const TO* wr = dec ? wz + (size_t)(h * D + r) * ld : wz + (size_t)(H * D + h * V + (r - D)) * ld + lr.ra;
+      const TO* wr = lr.staged ? wsm + r * wld : (dec ? wz + (size_t)(h * D + r) * ld : wz + (size_t)(H * D + h * V + (r - D)) * ld + lr.ra);
       const float zz = dl_row_dot<TO>(wr, dec ? xs : xs + lr.ra, dec ? lr.ra : lr.rg, sub, va);
       if (sub == 0) {
         if (dec) g[r] = expf(-ea * dl_softplus(zz + a.dt_bias[h * D + r]));
@@ -431,7 +512,6 @@ __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(DlArgs a, DlLowR
     for (int i = tid; i < D; i += DL_THREADS) g[i] = expf(-ea * dl_softplus(a.z[(size_t)t * a.z_ld + h * D + i] + a.dt_bias[h * D + i]));
     for (int i = tid; i < V; i += DL_THREADS) og[i] = dl_sigmoid(a.z[(size_t)t * a.z_ld + H * D + h * V + i]);
   }
-  const float beta = dl_sigmoid(to_f32(pj[a.b_col + h]));
   __syncthreads();
   float4 r = make_float4(0.f, 0.f, 0.f, 0.f), p = r;
 #pragma unroll
@@ -473,22 +553,23 @@ __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(DlArgs a, DlLowR
 static bool dl_step_fits(int D, int V, int ra, int rg) {
   if (V < 4 || V > 256 || (V & (V - 1)) || D <= 0 || (D + V) % 4) return false;
   const int NI = (D * V + 1023) / 1024;
-  return NI <= 32 && (size_t)(3 * D + 3 * V + ra + rg + 4 + 2048) * sizeof(float) <= 48 * 1024;
+  return NI <= 32 && 2 * D + V <= DL_STEP_CH * DL_THREADS && (size_t)(3 * D + 3 * V + ra + rg + 4 + 2048) * sizeof(float) <= 48 * 1024;
 }
 extern "C" int sx_delta_step_fits(int D, int V, int ra, int rg) { return dl_step_fits(D, V, ra, rg) ? 1 : 0; }
 
 // ---------------------------------------------------------------------------------------------------------------
-// chunks.  Scratch per (sequence, chunk, head): x, qg, kd [32, D] each, y [32, V], p [32, 32], ge [D].
+// chunks.  Scratch per (sequence, chunk, head): x, qg, kd [32, D] each, y [32, V], p [32, 32], ge [D], sb [D, V] (the state
+// at the chunk's begin).
 // ---------------------------------------------------------------------------------------------------------------
-struct DlChunks { float* x; float* qg; float* kd; float* y; float* p; float* ge; float* o; int P; };     // o [T, H V]
+struct DlChunks { float* x; float* qg; float* kd; float* y; float* p; float* ge; float* sb; int P; };
 
 template <typename TP>
-__global__ void __launch_bounds__(DL_THREADS, 2) delta_intra_kernel(DlArgs a, DlPrep w, DlChunks ch) {
+__global__ void __launch_bounds__(DL_THREADS, 3) delta_intra_kernel(DlArgs a, DlPrep w, DlChunks ch) {
   extern __shared__ __align__(16) float sm[];
   const int D = a.D, V = a.V, H = a.H, DS = D + 4, G = a.G;
   float* ks = sm;                        // 32 * DS
   float* qs = ks + DL_C * DS;            // 32 * DS
-  float* Gs = qs + DL_C * DS;            // 32 * DS: running sums of the decays' logarithms, base 2
+  float* Gs = qs + DL_C * DS;            // 32 * DS: running sums of the decays' logarithms, base 2, from token 0 and from token 16 on
   float* As = Gs + DL_C * DS;            // 32 * DL_LD
   float* bs = As + DL_C * DL_LD;         // 32
   pdl_wait();
@@ -501,26 +582,33 @@ __global__ void __launch_bounds__(DL_THREADS, 2) delta_intra_kernel(DlArgs a, Dl
   const int D4 = D >> 2;
   for (int i = tid; i < DL_C * D4; i += DL_THREADS) {
     const int t = i / D4, d = (i - t * D4) * 4;
-    float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), qv = kv;
     if (t < L) {
       const size_t at = (size_t)(t0 + t) * G * D + gq * D + d;
-      kv = *reinterpret_cast<const float4*>(w.k + at);
-      qv = *reinterpret_cast<const float4*>(w.q + at);
+      dl_cp16(ks + t * DS + d, w.k + at);
+      dl_cp16(qs + t * DS + d, w.q + at);
+    } else {
+      *reinterpret_cast<float4*>(ks + t * DS + d) = make_float4(0.f, 0.f, 0.f, 0.f);
+      *reinterpret_cast<float4*>(qs + t * DS + d) = make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    *reinterpret_cast<float4*>(ks + t * DS + d) = kv;
-    *reinterpret_cast<float4*>(qs + t * DS + d) = qv;
   }
+  dl_commit();
   if (tid < DL_C) bs[tid] = tid < L ? dl_sigmoid(to_f32(((const TP*)a.proj)[(size_t)(t0 + tid) * a.row + a.b_col + h])) : 0.f;
   for (int i = tid; i < DL_C * DL_LD; i += DL_THREADS) As[i] = 0.f;
-  if (tid < D) {
-    const float ea = -expf(a.a_log[h]) * DL_LOG2E, c = a.dt_bias[h * D + tid];
-    const float* z = a.z + (size_t)t0 * a.z_ld + h * D + tid;
+  {   // running sums: a thread a channel and half of the chunk (D <= 128) or a channel
+    const int parts = D <= DL_THREADS / 2 ? 2 : 1, part = parts == 2 && tid >= DL_THREADS / 2 ? 1 : 0, d = tid - part * (DL_THREADS / 2);
+    const int ta = part * 16, tb = parts == 2 ? ta + 16 : DL_C;
     float acc = 0.f;
+    if (d < D) {
+      const float ea = -expf(a.a_log[h]) * DL_LOG2E, c = a.dt_bias[h * D + d];
+      const float* z = a.z + (size_t)t0 * a.z_ld + h * D + d;
 #pragma unroll 8
-    for (int t = 0; t < DL_C; ++t) {
-      if (t < L) acc = fmaf(ea, dl_softplus(z[(size_t)t * a.z_ld] + c), acc);
-      Gs[t * DS + tid] = acc;
+      for (int t = ta; t < tb; ++t) {
+        if (t == 16) acc = 0.f;
+        if (t < L) acc += fmaxf(ea * dl_softplus(z[(size_t)t * a.z_ld] + c), DL_LOG_MIN);
+        Gs[t * DS + d] = acc;
+      }
     }
+    dl_wait<0>();
   }
   __syncthreads();
   // pairs within 16 tokens: thread (i, j): j < i the first half's pair (i, j), j > i the second half's (16 + j, 16 + i)
@@ -562,17 +650,17 @@ __global__ void __launch_bounds__(DL_THREADS, 2) delta_intra_kernel(DlArgs a, Dl
     float* Q = ch.qg + ci * DL_C * D + tid;
     float* K = ch.kd + ci * DL_C * D + tid;
     float *gp = Gs + tid, *kp = ks + tid, *qp = qs + tid;      // walked row by row: 32 addresses held at once would spill
-    const float gm = Gs[15 * DS + tid], ge = Gs[(DL_C - 1) * DS + tid];
-    ch.ge[ci * D + tid] = dl_exp2(ge);
+    const float gm = Gs[15 * DS + tid], gl = Gs[(DL_C - 1) * DS + tid];        // the two halves' whole sums
+    ch.ge[ci * D + tid] = dl_exp2(gm + gl);
 #pragma unroll
     for (int t = 0; t < DL_C; ++t) {
       asm volatile("" ::: "memory");
       const float gt = *gp, kt = *kp, qt = *qp;
-      const float e = dl_exp2(gt);
+      const float e = dl_exp2(t < 16 ? gt : gm + gt);
       rhs[t] = bs[t] * e * kt;
       *Q = e * qt;
-      *K = dl_exp2(ge - gt) * kt;
-      const float f = dl_exp2(t < 16 ? gm - gt : gt - gm);
+      *K = dl_exp2(t < 16 ? (gm - gt) + gl : gl - gt) * kt;
+      const float f = dl_exp2(t < 16 ? gm - gt : gt);
       *kp = f * kt;
       *qp = f * qt;
       Q += D; K += D; gp += DS; kp += DS; qp += DS;
@@ -638,229 +726,290 @@ __global__ void __launch_bounds__(DL_THREADS, 2) delta_intra_kernel(DlArgs a, Dl
 
 static size_t dl_intra_smem(int D) { return (size_t)(3 * DL_C * (D + 4) + DL_C * DL_LD + DL_C) * sizeof(float); }
 
-__device__ __forceinline__ void dl_cp16(float* smem, const float* gmem) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
-}
-__device__ __forceinline__ void dl_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
-template <int N> __device__ __forceinline__ void dl_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
 
-// VS: columns of the state a block owns (32 or 16)
-template <int VS>
+// VS: columns of the state a block owns (16 or 32); ND: tiles of the state a thread owns (D <= 128 ND)
+template <int VS, int ND>
 __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DlArgs a, DlChunks ch) {
   extern __shared__ __align__(16) float sm[];
   constexpr int SS = VS + 4;
-  constexpr int CG = VS / 4;                       // groups of four columns
-  constexpr int KSPLIT = DL_THREADS / (16 * CG);   // 2 or 4: parts of D in the products with S
+  constexpr int CG = VS / 4;                       // groups of four columns in the product with S
+  constexpr int KSPLIT = DL_THREADS / (8 * CG);    // 8 or 4: parts of D in that product
+  constexpr int CP = VS / 8;                       // columns a thread of u and of the state's tiles
   const int D = a.D, V = a.V, H = a.H, DS = D + 4;
-  float* xq = sm;                                  // 64 * DS: X above e^G q
-  float* kd = xq + 2 * DL_C * DS;                  // 32 * DS
-  float* S = kd + DL_C * DS;                       // D * SS
-  float* P = S + D * SS;                           // 32 * DL_LD
-  float* U = P + DL_C * DL_LD;                     // 32 * SS: u of the chunk
-  float* O = U + DL_C * SS;                        // 32 * SS: (e^G q) S
-  float* part = O + DL_C * SS;                     // (KSPLIT - 1) * 64 * SS
-  float* ge = part + (KSPLIT - 1) * 64 * SS;       // D
+  float* xs = sm;                                  // 2 * 32 * DS: X, two chunks
+  float* kd = xs + 2 * DL_C * DS;                  // 2 * 32 * DS: e^(G_end - G) k
+  float* S = kd + 2 * DL_C * DS;                   // D * SS
+  float* U = S + D * SS;                           // 32 * SS
+  float* part = U + DL_C * SS;                     // KSPLIT * 32 * SS
   pdl_wait();
   pdl_trigger();
   const int v0 = blockIdx.x * VS, h = blockIdx.y, s = blockIdx.z, tid = threadIdx.x;
   const int tok0 = a.cu_seqlens[s], n = a.cu_seqlens[s + 1] - tok0, np = (n + DL_C - 1) / DL_C;
+  if (np <= 0) return;
   float* Sg = a.S + ((size_t)a.seq_slots[s] * H + h) * D * V;
   const int D4 = D >> 2;
-  auto load_xq = [&](int p) {
-    const size_t ci = ((size_t)s * ch.P + p) * H + h;
-    const float *x = ch.x + ci * DL_C * D, *q = ch.qg + ci * DL_C * D;
-    for (int i = tid; i < DL_C * D4; i += DL_THREADS) {
-      const int t = i / D4, d = (i - t * D4) * 4;
-      dl_cp16(xq + t * DS + d, x + (size_t)t * D + d);
-      dl_cp16(xq + (DL_C + t) * DS + d, q + (size_t)t * D + d);
-    }
-    dl_commit();
+  auto chunk = [&](int p) { return ((size_t)s * ch.P + p) * H + h; };
+  auto load = [&](int p) {
+    const float *x = ch.x + chunk(p) * DL_C * D, *k = ch.kd + chunk(p) * DL_C * D;
+    float *xd = xs + (p & 1) * DL_C * DS, *kk = kd + (p & 1) * DL_C * DS;
+    for (int d = (tid & 31) * 4; d < D; d += 128)
+#pragma unroll
+      for (int t = 0; t < DL_C; t += DL_THREADS / 32) {
+        const int r = t + (tid >> 5);
+        dl_cp16(xd + r * DS + d, x + r * D + d);
+        dl_cp16(kk + r * DS + d, k + r * D + d);
+      }
   };
-  auto load_kp = [&](int p) {
-    const size_t ci = ((size_t)s * ch.P + p) * H + h;
-    const float *k = ch.kd + ci * DL_C * D, *pg = ch.p + ci * DL_C * DL_C, *g = ch.ge + ci * D;
-    for (int i = tid; i < DL_C * D4; i += DL_THREADS) {
-      const int t = i / D4, d = (i - t * D4) * 4;
-      dl_cp16(kd + t * DS + d, k + (size_t)t * D + d);
+  // this thread's place in u (row ur, CP columns from uc on) and in the state (rows 4 sd .., the same columns)
+  const int ur = tid >> 3, uc = (tid & 7) * CP, sd = tid >> 3;
+  float st[ND][4][CP], y[CP], ge[ND][4];
+  auto load_small = [&](int p) {                   // what goes to registers: u's right side, the chunk's whole decay
+    const float* yg = ch.y + chunk(p) * DL_C * V + (size_t)ur * V + v0 + uc;
+#pragma unroll
+    for (int j = 0; j < CP; ++j) y[j] = v0 + uc + j < V ? yg[j] : 0.f;
+#pragma unroll
+    for (int b = 0; b < ND; ++b) {
+      const int d = (sd + 32 * b) * 4;
+      if (d < D) {
+        const float4 f = *reinterpret_cast<const float4*>(ch.ge + chunk(p) * D + d);
+        ge[b][0] = f.x; ge[b][1] = f.y; ge[b][2] = f.z; ge[b][3] = f.w;
+      }
     }
-    for (int i = tid; i < DL_C * DL_C / 4; i += DL_THREADS) dl_cp16(P + (i >> 3) * DL_LD + (i & 7) * 4, pg + i * 4);
-    for (int i = tid; i < D4; i += DL_THREADS) dl_cp16(ge + i * 4, g + i * 4);
-    dl_commit();
   };
-  if (np > 0) { load_xq(0); load_kp(0); }
-  for (int i = tid; i < D * VS; i += DL_THREADS) {
-    const int d = i / VS, c = i - d * VS;
-    S[d * SS + c] = v0 + c < V ? Sg[(size_t)d * V + v0 + c] : 0.f;
-  }
-  const int kg = tid / (16 * CG), rem = tid - kg * 16 * CG, rg = rem / CG, cg = rem - rg * CG;
+  load(0);
+  dl_commit();
+  load_small(0);
+#pragma unroll
+  for (int b = 0; b < ND; ++b)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int d = (sd + 32 * b) * 4 + i;
+#pragma unroll
+      for (int j = 0; j < CP; ++j) st[b][i][j] = d < D && v0 + uc + j < V ? Sg[(size_t)d * V + v0 + uc + j] : 0.f;
+    }
+  const int kg = tid / (8 * CG), rem = tid - kg * 8 * CG, rg = rem / CG, cg = rem - rg * CG;
   const int dper = (D4 + KSPLIT - 1) / KSPLIT * 4, da = kg * dper, db = min(D, da + dper);
   for (int p = 0; p < np; ++p) {
-    const size_t ci = ((size_t)s * ch.P + p) * H + h;
-    const int L = min(DL_C, n - p * DL_C);
-    dl_wait<1>();
-    __syncthreads();                               // X, q of this chunk and S of the last are in place
+    // the state at the chunk's begin: to shared memory for the product, to memory for the output kernel
+    float* sb = ch.sb + chunk(p) * D * V;
+#pragma unroll
+    for (int b = 0; b < ND; ++b)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int d = (sd + 32 * b) * 4 + i;
+        if (d < D) {
+#pragma unroll
+          for (int j = 0; j < CP; ++j) S[d * SS + uc + j] = st[b][i][j];
+          if ((V & 3) == 0 && v0 + uc + CP <= V) {
+            if (CP == 4) *reinterpret_cast<float4*>(sb + (size_t)d * V + v0 + uc) = make_float4(st[b][i][0], st[b][i][1], st[b][i][2 % CP], st[b][i][3 % CP]);
+            else *reinterpret_cast<float2*>(sb + (size_t)d * V + v0 + uc) = make_float2(st[b][i][0], st[b][i][1]);
+          } else {
+#pragma unroll
+            for (int j = 0; j < CP; ++j)
+              if (v0 + uc + j < V) sb[(size_t)d * V + v0 + uc + j] = st[b][i][j];
+          }
+        }
+      }
+    dl_wait<0>();
+    __syncthreads();                               // X, k of this chunk and S are in place; the other buffers are read out
+    if (p + 1 < np) load(p + 1);
+    dl_commit();
+    const float *xd = xs + (p & 1) * DL_C * DS, *kk = kd + (p & 1) * DL_C * DS;
     float acc[4][4];
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
       for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-    for (int d = da; d < db; d += 4) {             // rows rg, rg + 16, rg + 32, rg + 48
+#pragma unroll 2
+    for (int d = da; d < db; d += 4) {             // rows rg, rg + 8, rg + 16, rg + 24
       float4 b[4];
 #pragma unroll
       for (int x = 0; x < 4; ++x) b[x] = *reinterpret_cast<const float4*>(S + (d + x) * SS + cg * 4);
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float4 m = *reinterpret_cast<const float4*>(xq + (rg + 16 * i) * DS + d);
+        const float4 m = *reinterpret_cast<const float4*>(xd + (rg + 8 * i) * DS + d);
         acc[i][0] = fmaf(m.x, b[0].x, fmaf(m.y, b[1].x, fmaf(m.z, b[2].x, fmaf(m.w, b[3].x, acc[i][0]))));
         acc[i][1] = fmaf(m.x, b[0].y, fmaf(m.y, b[1].y, fmaf(m.z, b[2].y, fmaf(m.w, b[3].y, acc[i][1]))));
         acc[i][2] = fmaf(m.x, b[0].z, fmaf(m.y, b[1].z, fmaf(m.z, b[2].z, fmaf(m.w, b[3].z, acc[i][2]))));
         acc[i][3] = fmaf(m.x, b[0].w, fmaf(m.y, b[1].w, fmaf(m.z, b[2].w, fmaf(m.w, b[3].w, acc[i][3]))));
       }
     }
-    if (kg > 0) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      *reinterpret_cast<float4*>(part + (kg * DL_C + rg + 8 * i) * SS + cg * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+    __syncthreads();
+    {   // u = Y - X S, left in Y's place for the output kernel
+      float u[CP];
+#pragma unroll
+      for (int j = 0; j < CP; ++j) u[j] = y[j];
+#pragma unroll
+      for (int x = 0; x < KSPLIT; ++x)
+#pragma unroll
+        for (int j = 0; j < CP; ++j) u[j] -= part[(x * DL_C + ur) * SS + uc + j];
+      float* yg = ch.y + chunk(p) * DL_C * V + (size_t)ur * V + v0 + uc;
+#pragma unroll
+      for (int j = 0; j < CP; ++j) {
+        U[ur * SS + uc + j] = u[j];
+        if (v0 + uc + j < V) yg[j] = u[j];
+      }
+    }
+#pragma unroll
+    for (int b = 0; b < ND; ++b)
 #pragma unroll
       for (int i = 0; i < 4; ++i)
-        *reinterpret_cast<float4*>(part + ((kg - 1) * 64 + rg + 16 * i) * SS + cg * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
-    }
-    __syncthreads();                               // X and q are read out
-    if (p + 1 < np) load_xq(p + 1); else dl_commit();
-    if (kg == 0) {
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int r = rg + 16 * i;
-        float4 v = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+        for (int j = 0; j < CP; ++j) st[b][i][j] *= ge[b][i];
+    if (p + 1 < np) load_small(p + 1);
+    __syncthreads();
 #pragma unroll
-        for (int x = 0; x < KSPLIT - 1; ++x) {
-          const float4 o = *reinterpret_cast<const float4*>(part + (x * 64 + r) * SS + cg * 4);
-          v.x += o.x; v.y += o.y; v.z += o.z; v.w += o.w;
-        }
-        if (i < 2) {                               // u = Y - X S
-          const float* Y = ch.y + ci * DL_C * V + (size_t)r * V + v0 + cg * 4;
-          const int left = V - (v0 + cg * 4);
-          float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (left >= 4 && (V & 3) == 0) y = *reinterpret_cast<const float4*>(Y);
-          else {
-            if (left > 0) y.x = Y[0];
-            if (left > 1) y.y = Y[1];
-            if (left > 2) y.z = Y[2];
-            if (left > 3) y.w = Y[3];
-          }
-          *reinterpret_cast<float4*>(U + r * SS + cg * 4) = make_float4(y.x - v.x, y.y - v.y, y.z - v.z, y.w - v.w);
-        } else {
-          *reinterpret_cast<float4*>(O + (r - DL_C) * SS + cg * 4) = v;
-        }
-      }
-    }
-    dl_wait<1>();
-    __syncthreads();                               // u, the first half of o, and this chunk's k, P, e^(G_end)
-    {   // o: a thread two rows and VS / 16 columns
-      constexpr int OC = VS / 16;
-      const int r = (tid >> 4) * 2, c = (tid & 15) * OC;
-      float o[2][OC];
-#pragma unroll
-      for (int i = 0; i < 2; ++i)
-#pragma unroll
-        for (int j = 0; j < OC; ++j) o[i][j] = O[(r + i) * SS + c + j];
-      for (int u = 0; u <= r + 1; u += 4) {        // P is zero above its diagonal
-        const float4 p0 = *reinterpret_cast<const float4*>(P + r * DL_LD + u), p1 = *reinterpret_cast<const float4*>(P + (r + 1) * DL_LD + u);
-#pragma unroll
-        for (int j = 0; j < OC; ++j) {
-          const float u0 = U[u * SS + c + j], u1 = U[(u + 1) * SS + c + j], u2 = U[(u + 2) * SS + c + j], u3 = U[(u + 3) * SS + c + j];
-          o[0][j] = fmaf(p0.x, u0, fmaf(p0.y, u1, fmaf(p0.z, u2, fmaf(p0.w, u3, o[0][j]))));
-          o[1][j] = fmaf(p1.x, u0, fmaf(p1.y, u1, fmaf(p1.z, u2, fmaf(p1.w, u3, o[1][j]))));
-        }
-      }
-#pragma unroll
-      for (int i = 0; i < 2; ++i)
-        if (r + i < L) {
-          float* og = ch.o + (size_t)(tok0 + p * DL_C + r + i) * H * V + h * V;
-#pragma unroll
-          for (int j = 0; j < OC; ++j)
-            if (v0 + c + j < V) og[v0 + c + j] = o[i][j];
-        }
-    }
-    {   // S: tiles of RT rows x 4 columns
-      constexpr int RT = VS == 32 ? 4 : 2;
-      const int tiles = (D / RT) * CG;
-      for (int tile = tid; tile < tiles; tile += DL_THREADS) {
-        const int d = (tile / CG) * RT, c = (tile % CG) * 4;
-        float4 x[RT];
-#pragma unroll
-        for (int i = 0; i < RT; ++i) {
-          const float e = ge[d + i];
-          x[i] = *reinterpret_cast<const float4*>(S + (d + i) * SS + c);
-          x[i].x *= e; x[i].y *= e; x[i].z *= e; x[i].w *= e;
-        }
+    for (int b = 0; b < ND; ++b) {
+      const int d = (sd + 32 * b) * 4;
+      if (d < D) {
 #pragma unroll 8
         for (int t = 0; t < DL_C; ++t) {
-          const float4 u = *reinterpret_cast<const float4*>(U + t * SS + c);
-          float kk[4];
-          if (RT == 4) {
-            const float4 f = *reinterpret_cast<const float4*>(kd + t * DS + d);
-            kk[0] = f.x; kk[1] = f.y; kk[2] = f.z; kk[3] = f.w;
-          } else {
-            const float2 f = *reinterpret_cast<const float2*>(kd + t * DS + d);
-            kk[0] = f.x; kk[1] = f.y;
-          }
+          const float4 f = *reinterpret_cast<const float4*>(kk + t * DS + d);
+          float u[CP];
 #pragma unroll
-          for (int i = 0; i < RT; ++i) {
-            x[i].x = fmaf(kk[i], u.x, x[i].x); x[i].y = fmaf(kk[i], u.y, x[i].y);
-            x[i].z = fmaf(kk[i], u.z, x[i].z); x[i].w = fmaf(kk[i], u.w, x[i].w);
+          for (int j = 0; j < CP; ++j) u[j] = U[t * SS + uc + j];
+#pragma unroll
+          for (int j = 0; j < CP; ++j) {
+            st[b][0][j] = fmaf(f.x, u[j], st[b][0][j]);
+            st[b][1][j] = fmaf(f.y, u[j], st[b][1][j]);
+            st[b][2][j] = fmaf(f.z, u[j], st[b][2][j]);
+            st[b][3][j] = fmaf(f.w, u[j], st[b][3][j]);
           }
         }
-#pragma unroll
-        for (int i = 0; i < RT; ++i) *reinterpret_cast<float4*>(S + (d + i) * SS + c) = x[i];
       }
     }
-    __syncthreads();                               // k, P and u are read out
-    if (p + 1 < np) load_kp(p + 1); else dl_commit();
   }
-  dl_wait<0>();
-  __syncthreads();
-  for (int i = tid; i < D * VS; i += DL_THREADS) {
-    const int d = i / VS, c = i - d * VS;
-    if (v0 + c < V) Sg[(size_t)d * V + v0 + c] = S[d * SS + c];
-  }
+#pragma unroll
+  for (int b = 0; b < ND; ++b)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int d = (sd + 32 * b) * 4 + i;
+#pragma unroll
+      for (int j = 0; j < CP; ++j)
+        if (d < D && v0 + uc + j < V) Sg[(size_t)d * V + v0 + uc + j] = st[b][i][j];
+    }
 }
 
 static size_t dl_scan_smem(int D, int VS) {
-  const int SS = VS + 4, ksplit = DL_THREADS / (16 * (VS / 4));
-  return (size_t)(3 * DL_C * (D + 4) + D * SS + DL_C * DL_LD + 2 * DL_C * SS + (ksplit - 1) * 64 * SS + D) * sizeof(float);
+  const int SS = VS + 4, ksplit = DL_THREADS / (2 * VS);
+  return (size_t)(4 * DL_C * (D + 4) + D * SS + DL_C * SS + ksplit * DL_C * SS) * sizeof(float);
 }
 
-// a warp a (token, head): o / rms(o) * gain * sigmoid(gate)
-template <typename TO>
-__global__ void __launch_bounds__(DL_THREADS) delta_finish_kernel(DlArgs a, const float* __restrict__ o, int n_tokens) {
+// a block a (chunk, head): o = [e^G q | P] [S_begin; u], then the output norm, gain and gate.  A warp owns four rows of all
+// columns (NT tiles of 128), so the norm is a warp's business; both factors lie in shared memory whole, in two portions
+// that arrive one after the other.
+template <typename TO, int NT>
+__global__ void __launch_bounds__(DL_THREADS, 2) delta_out_kernel(DlArgs a, DlChunks ch) {
+  extern __shared__ __align__(16) float sm[];
+  const int D = a.D, V = a.V, H = a.H, DS = D + DL_C + 4, BS = ((V + 3) & ~3) + 4;
+  float* A = sm;                                   // 32 * DS: e^G q, then P
+  float* B = A + DL_C * DS;                        // (D + 32) * BS: S_begin, then u
   pdl_wait();
   pdl_trigger();
-  const int V = a.V, H = a.H, lane = threadIdx.x & 31;
-  const long long item = (long long)blockIdx.x * (DL_THREADS / 32) + (threadIdx.x >> 5);
-  if (item >= (long long)n_tokens * H) return;
-  const int t = (int)(item / H), h = (int)(item % H);
-  const float* x = o + (size_t)item * V;
-  const float* z = a.z + (size_t)t * a.z_ld + H * a.D + h * V;
-  TO* out = (TO*)a.out + (size_t)item * V;
-  if (V == 128) {
-    const float4 f = reinterpret_cast<const float4*>(x)[lane];
-    const float4 gt = make_float4(z[lane * 4], z[lane * 4 + 1], z[lane * 4 + 2], z[lane * 4 + 3]);
-    const float inv = rsqrtf(warp_sum(f.x * f.x + f.y * f.y + f.z * f.z + f.w * f.w) / 128.f + a.eps);
-    const float* gn = a.gain + lane * 4;
-    out[lane * 4] = from_f32<TO>(f.x * inv * gn[0] * dl_sigmoid(gt.x));
-    out[lane * 4 + 1] = from_f32<TO>(f.y * inv * gn[1] * dl_sigmoid(gt.y));
-    out[lane * 4 + 2] = from_f32<TO>(f.z * inv * gn[2] * dl_sigmoid(gt.z));
-    out[lane * 4 + 3] = from_f32<TO>(f.w * inv * gn[3] * dl_sigmoid(gt.w));
-    return;
+  const int p = blockIdx.x, h = blockIdx.y, s = blockIdx.z, tid = threadIdx.x;
+  const int t0 = a.cu_seqlens[s] + p * DL_C, len = a.cu_seqlens[s + 1] - t0;
+  if (len <= 0) return;
+  const int L = min(DL_C, len);
+  const size_t ci = ((size_t)s * ch.P + p) * H + h;
+  const float *qg = ch.qg + ci * DL_C * D, *pg = ch.p + ci * DL_C * DL_C, *sb = ch.sb + ci * D * V, *ug = ch.y + ci * DL_C * V;
+  const int warp = tid >> 5, lane = tid & 31;
+  auto load_rows = [&](float* dst, const float* src, int rows) {        // rows of V columns
+    if ((V & 3) == 0) {
+      for (int c = lane * 4; c < V; c += 128)
+        for (int r = warp; r < rows; r += DL_THREADS / 32) dl_cp16(dst + r * BS + c, src + (size_t)r * V + c);
+    } else {
+      for (int c = lane; c < V; c += 32)
+        for (int r = warp; r < rows; r += DL_THREADS / 32) dst[r * BS + c] = src[(size_t)r * V + c];
+    }
+  };
+  const int half = D / 2 & ~3;
+  for (int d = lane * 4; d < D; d += 128)
+    for (int t = warp; t < DL_C; t += DL_THREADS / 32) dl_cp16(A + t * DS + d, qg + t * D + d);
+  load_rows(B, sb, half);
+  dl_commit();
+  dl_cp16(A + (tid >> 3) * DS + D + (tid & 7) * 4, pg + tid * 4);
+  load_rows(B + half * BS, sb + (size_t)half * V, D - half);
+  load_rows(B + D * BS, ug, DL_C);
+  dl_commit();
+  float acc[NT][4][4];
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[n][i][j] = 0.f;
+  auto product = [&](int k0, int k1) {
+#pragma unroll 4
+    for (int k = k0; k < k1; k += 4) {
+      float4 m[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) m[i] = *reinterpret_cast<const float4*>(A + (warp * 4 + i) * DS + k);
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        const int c = n * 128 + lane * 4;
+        if (c < V) {
+          float4 x[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) x[e] = *reinterpret_cast<const float4*>(B + (k + e) * BS + c);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            acc[n][i][0] = fmaf(m[i].x, x[0].x, fmaf(m[i].y, x[1].x, fmaf(m[i].z, x[2].x, fmaf(m[i].w, x[3].x, acc[n][i][0]))));
+            acc[n][i][1] = fmaf(m[i].x, x[0].y, fmaf(m[i].y, x[1].y, fmaf(m[i].z, x[2].y, fmaf(m[i].w, x[3].y, acc[n][i][1]))));
+            acc[n][i][2] = fmaf(m[i].x, x[0].z, fmaf(m[i].y, x[1].z, fmaf(m[i].z, x[2].z, fmaf(m[i].w, x[3].z, acc[n][i][2]))));
+            acc[n][i][3] = fmaf(m[i].x, x[0].w, fmaf(m[i].y, x[1].w, fmaf(m[i].z, x[2].w, fmaf(m[i].w, x[3].w, acc[n][i][3]))));
+          }
+        }
+      }
+    }
+  };
+  dl_wait<1>();
+  __syncthreads();
+  product(0, half);
+  dl_wait<0>();
+  __syncthreads();
+  float z[NT][4][4];                               // the gates' pre-activations: on their way during the second product
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int c = n * 128 + lane * 4, r = min(warp * 4 + i, L - 1);
+      const float* zr = a.z + (size_t)(t0 + r) * a.z_ld + H * D + h * V + c;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) z[n][i][j] = c + j < V ? zr[j] : 0.f;
+    }
+  product(half, D + DL_C);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int r = warp * 4 + i;
+    float ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (n * 128 + lane * 4 + j < V) ss += acc[n][i][j] * acc[n][i][j];
+    const float inv = rsqrtf(warp_sum(ss) / (float)V + a.eps);
+    if (r < L) {
+      TO* out = (TO*)a.out + (size_t)(t0 + r) * H * V + h * V;
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int c = n * 128 + lane * 4 + j;
+          if (c < V) out[c] = from_f32<TO>(acc[n][i][j] * inv * a.gain[c] * dl_sigmoid(z[n][i][j]));
+        }
+    }
   }
-  float ss = 0.f;
-  for (int c = lane; c < V; c += 32) ss += x[c] * x[c];
-  const float inv = rsqrtf(warp_sum(ss) / (float)V + a.eps);
-  for (int c = lane; c < V; c += 32) out[c] = from_f32<TO>(x[c] * inv * a.gain[c] * dl_sigmoid(z[c]));
 }
+
+static size_t dl_out_smem(int D, int V) { return (size_t)(DL_C * (D + DL_C + 4) + (D + DL_C) * (((V + 3) & ~3) + 4)) * sizeof(float); }
 
 extern "C" int sx_delta_chunk_tokens() { return DL_C; }
 extern "C" int sx_delta_chunks_fit(int D, int V) {
-  return (D % 4 == 0 && D <= DL_THREADS && dl_intra_smem(D) <= 220 * 1024 && dl_scan_smem(D, 32) <= 220 * 1024 &&
-          dl_scan_smem(D, 16) <= 220 * 1024 && V > 0) ? 1 : 0;
+  return (D % 4 == 0 && D <= DL_THREADS && V <= 256 && dl_intra_smem(D) <= 220 * 1024 && dl_scan_smem(D, 32) <= 220 * 1024 &&
+          dl_scan_smem(D, 16) <= 220 * 1024 && dl_out_smem(D, V) <= 220 * 1024) ? 1 : 0;
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -887,11 +1036,20 @@ static int dl_check(int n_seqs, int H, int G, int D, int V, int taps) {
 }
 
 template <typename TP, typename TO>
-static int dl_step_launch(const DlArgs& a, const DlLowRank& lr, int n_seqs, cudaStream_t stream) {
-  const size_t smem = (size_t)(3 * a.D + 3 * a.V + lr.ra + lr.rg + 4 + 2048) * sizeof(float);
+static int dl_step_launch(const DlArgs& a, DlLowRank lr, int n_seqs, cudaStream_t stream) {
+  size_t smem = (size_t)(((3 * a.D + 2 * a.V + lr.ra + lr.rg + 3) & ~3) + 2048 + a.V) * sizeof(float);
+  constexpr int VE = 16 / sizeof(TO);
+  if (lr.wz && lr.ra % VE == 0 && lr.rg % VE == 0) {
+    const size_t w = (size_t)(a.D + a.V) * dl_lr_ld<TO>(lr.ra, lr.rg) * sizeof(TO);
+    if (smem + w <= 100 * 1024) { lr.staged = 1; smem += w; }
+  }
   const int NI = (a.D * a.V + 1023) / 1024;
   const dim3 grid(a.H, n_seqs), block(DL_THREADS);
-#define DL_STEP(N) return sx_launch(delta_step_kernel<TP, TO, N>, grid, block, smem, stream, a, lr)
+#define DL_STEP(N)                                                                                                              \
+  do {                                                                                                                          \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(delta_step_kernel<TP, TO, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    return sx_launch(delta_step_kernel<TP, TO, N>, grid, block, smem, stream, a, lr);                                           \
+  } while (0)
   if (NI <= 2) DL_STEP(2);
   if (NI <= 4) DL_STEP(4);
   if (NI <= 8) DL_STEP(8);
@@ -907,7 +1065,7 @@ extern "C" int sx_delta_step(DL_FORMALS, const void* wz, int ra, int rg, int lr_
   if (wz == nullptr && z == nullptr) return SX_ERR_SIZE;
   if ((uintptr_t)S % 16 || (uintptr_t)wz % 16) return SX_ERR_ALIGN;
   const DlArgs a = dl_args(DL_ACTUALS);
-  const DlLowRank lr = {wz, wz ? ra : 0, wz ? rg : 0, lr_col};
+  const DlLowRank lr = {wz, wz ? ra : 0, wz ? rg : 0, lr_col, 0};
   if (proj_dt == SX_F32 && out_dt == SX_F32) return dl_step_launch<float, float>(a, lr, n_seqs, stream);
   if (proj_dt == SX_F32 && out_dt == SX_BF16) return dl_step_launch<float, bf16>(a, lr, n_seqs, stream);
   if (proj_dt == SX_BF16 && out_dt == SX_BF16) return dl_step_launch<bf16, bf16>(a, lr, n_seqs, stream);
@@ -922,9 +1080,14 @@ static int dl_prepare_launch(const DlArgs& a, const DlPrep& w, int n_tokens, int
   int rc;
   if (lane_vec(a.D) && lane_vec(a.V) && aligned && a.taps >= 2 && a.taps <= 4) {
     const dim3 grid((n_tokens + DL_RUN - 1) / DL_RUN, (units + DL_THREADS / 32 - 1) / (DL_THREADS / 32));
-    if (a.taps == 2) rc = sx_launch(delta_prepare_run_kernel<TP, 2>, grid, dim3(DL_THREADS), 0, stream, a, w, n_tokens);
-    else if (a.taps == 3) rc = sx_launch(delta_prepare_run_kernel<TP, 3>, grid, dim3(DL_THREADS), 0, stream, a, w, n_tokens);
-    else rc = sx_launch(delta_prepare_run_kernel<TP, 4>, grid, dim3(DL_THREADS), 0, stream, a, w, n_tokens);
+    const bool wide = a.D == 256 || a.V == 256;
+#define DL_RUN_GO(N)                                                                                                     \
+  rc = wide ? sx_launch(delta_prepare_run_kernel<TP, N, true>, grid, dim3(DL_THREADS), 0, stream, a, w, n_tokens)        \
+            : sx_launch(delta_prepare_run_kernel<TP, N, false>, grid, dim3(DL_THREADS), 0, stream, a, w, n_tokens)
+    if (a.taps == 2) DL_RUN_GO(2);
+    else if (a.taps == 3) DL_RUN_GO(3);
+    else DL_RUN_GO(4);
+#undef DL_RUN_GO
   } else {
     const long long items = (long long)n_tokens * units;
     rc = sx_launch(delta_prepare_kernel<TP>, dim3((unsigned)((items + DL_THREADS / 32 - 1) / (DL_THREADS / 32))), dim3(DL_THREADS), 0, stream, a, w, n_tokens);
@@ -966,38 +1129,43 @@ extern "C" int sx_delta_walk(DL_FORMALS, float* q, float* k, float* v, cudaStrea
 }
 
 template <typename TP, typename TO>
-static int dl_chunks_launch(const DlArgs& a, const DlPrep& w, const DlChunks& ch, int n_tokens, int n_seqs, int slice, cudaStream_t stream) {
+static int dl_chunks_launch(const DlArgs& a, const DlPrep& w, const DlChunks& ch, int n_seqs, int slice, cudaStream_t stream) {
   const size_t si = dl_intra_smem(a.D);
   if (si > 48 * 1024) cudaFuncSetAttribute(delta_intra_kernel<TP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)si);
   int rc = sx_launch(delta_intra_kernel<TP>, dim3(ch.P, a.H, n_seqs), dim3(DL_THREADS), si, stream, a, w, ch);
   if (rc) return rc;
   const size_t ss = dl_scan_smem(a.D, slice);
   const dim3 grid((a.V + slice - 1) / slice, a.H, n_seqs);
-  if (slice == 32) {
-    if (ss > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ss);
-    rc = sx_launch(delta_scan_kernel<32>, grid, dim3(DL_THREADS), ss, stream, a, ch);
-  } else {
-    if (ss > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ss);
-    rc = sx_launch(delta_scan_kernel<16>, grid, dim3(DL_THREADS), ss, stream, a, ch);
-  }
+#define DL_SCAN(VS, ND)                                                                                                       \
+  do {                                                                                                                        \
+    if (ss > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<VS, ND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ss); \
+    rc = sx_launch(delta_scan_kernel<VS, ND>, grid, dim3(DL_THREADS), ss, stream, a, ch);                                      \
+  } while (0)
+  if (slice == 32) { if (a.D <= 128) DL_SCAN(32, 1); else DL_SCAN(32, 2); }
+  else { if (a.D <= 128) DL_SCAN(16, 1); else DL_SCAN(16, 2); }
+#undef DL_SCAN
   if (rc) return rc;
-  const long long items = (long long)n_tokens * a.H;
-  return sx_launch(delta_finish_kernel<TO>, dim3((unsigned)((items + DL_THREADS / 32 - 1) / (DL_THREADS / 32))), dim3(DL_THREADS), 0, stream, a,
-                   (const float*)ch.o, n_tokens);
+  const size_t so = dl_out_smem(a.D, a.V);
+  if (a.V <= 128) {
+    if (so > 48 * 1024) cudaFuncSetAttribute(delta_out_kernel<TO, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)so);
+    return sx_launch(delta_out_kernel<TO, 1>, dim3(ch.P, a.H, n_seqs), dim3(DL_THREADS), so, stream, a, ch);
+  }
+  if (so > 48 * 1024) cudaFuncSetAttribute(delta_out_kernel<TO, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)so);
+  return sx_launch(delta_out_kernel<TO, 2>, dim3(ch.P, a.H, n_seqs), dim3(DL_THREADS), so, stream, a, ch);
 }
 
 // chunks of DL_C tokens (the caller has asked sx_delta_chunks_fit); slice: columns of the state a block of the scan owns
 extern "C" int sx_delta_chunks(DL_FORMALS, float* q, float* k, float* v, float* x, float* qg, float* kd, float* y, float* p,
-                               float* ge, float* o, int chunks, int slice, cudaStream_t stream) {
+                               float* ge, float* sb, int chunks, int slice, cudaStream_t stream) {
   if (n_tokens <= 0 || n_seqs <= 0) return 0;
   if (dl_check(n_seqs, H, G, D, V, taps) || !sx_delta_chunks_fit(D, V) || (slice != 16 && slice != 32) || chunks <= 0) return SX_ERR_SIZE;
-  if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)x | (uintptr_t)qg | (uintptr_t)kd | (uintptr_t)y | (uintptr_t)p | (uintptr_t)ge | (uintptr_t)o) % 16)
+  if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)x | (uintptr_t)qg | (uintptr_t)kd | (uintptr_t)y | (uintptr_t)p | (uintptr_t)ge | (uintptr_t)sb) % 16)
     return SX_ERR_ALIGN;
   const DlArgs a = dl_args(DL_ACTUALS);
   const DlPrep w = {q, k, v};
-  const DlChunks ch = {x, qg, kd, y, p, ge, o, chunks};
-  if (proj_dt == SX_F32 && out_dt == SX_F32) return dl_chunks_launch<float, float>(a, w, ch, n_tokens, n_seqs, slice, stream);
-  if (proj_dt == SX_F32 && out_dt == SX_BF16) return dl_chunks_launch<float, bf16>(a, w, ch, n_tokens, n_seqs, slice, stream);
-  if (proj_dt == SX_BF16 && out_dt == SX_BF16) return dl_chunks_launch<bf16, bf16>(a, w, ch, n_tokens, n_seqs, slice, stream);
+  const DlChunks ch = {x, qg, kd, y, p, ge, sb, chunks};
+  if (proj_dt == SX_F32 && out_dt == SX_F32) return dl_chunks_launch<float, float>(a, w, ch, n_seqs, slice, stream);
+  if (proj_dt == SX_F32 && out_dt == SX_BF16) return dl_chunks_launch<float, bf16>(a, w, ch, n_seqs, slice, stream);
+  if (proj_dt == SX_BF16 && out_dt == SX_BF16) return dl_chunks_launch<bf16, bf16>(a, w, ch, n_seqs, slice, stream);
   return SX_ERR_DTYPE;
 }

@@ -6,7 +6,7 @@
 //                       sum of rows of a, sum_k wts[t, k] a[place[t, k]], a mixture of experts' chosen results), or
 //                 v   = f * (rms_norm(a) ga + rms_norm(b) gb)     (one or two terms with gains: mixers side by side)
 //                 d   = gp ? rms_norm(v) gp : v                   (the branch's own norm)
-//                 acc = h ? h[t] + d : d;   if write_h: h[t] = acc
+//                 acc = h ? h[t] + d : d;   acc += vec (a vector over the width, optional);   if write_h: h[t] = acc
 //                 y[r] = go ? rms_norm(acc) go : acc              (the next reader's rows: a cast, or the final norm)
 //                 rms_norm(x) = x / sqrt(mean(x^2) + eps).  Rows: r = 0..R-1, t = rows ? rows[r] : r.
 //   embed_bigram: out[t] = E[id_t] + B[(prev_t * mp + id_t * mc) mod n], row n of B for a sequence's first token;
@@ -59,7 +59,7 @@ __global__ void __launch_bounds__(1024) add_normed_kernel(
     float* __restrict__ h, const void* __restrict__ a, int a_dt, const float* __restrict__ ga,
     const void* __restrict__ b, int b_dt, const float* __restrict__ gb, float factor, const float* __restrict__ gp,
     const float* __restrict__ go, float eps, TO* __restrict__ y, const int* __restrict__ rows, int H, int write_h,
-    const int* __restrict__ place, const float* __restrict__ wts, int top) {
+    const int* __restrict__ place, const float* __restrict__ wts, int top, const float* __restrict__ vec) {
   extern __shared__ __align__(16) float row[];
   __shared__ float red[33];
   pdl_wait();
@@ -138,6 +138,11 @@ __global__ void __launch_bounds__(1024) add_normed_kernel(
       ldfv<W>(h, base + i, u);
 #pragma unroll
       for (int j = 0; j < W; ++j) v[j] += u[j];
+      if (vec) {
+        ldfv<W>(vec, i, u);
+#pragma unroll
+        for (int j = 0; j < W; ++j) v[j] += u[j];
+      }
       if (write_h) stfv<W>(h, base + i, v);
     }
     stfv<W>(row, i, v);
@@ -167,7 +172,7 @@ __global__ void __launch_bounds__(1024) add_normed_kernel(
 template <typename TO, int W>
 static int add_normed_launch(float* h, const void* a, int a_dt, const float* ga, const void* b, int b_dt, const float* gb,
                              float factor, const float* gp, const float* go, float eps, void* y, const int* rows, int R, int H,
-                             int write_h, const int* place, const float* wts, int top, cudaStream_t stream) {
+                             int write_h, const int* place, const float* wts, int top, const float* vec, cudaStream_t stream) {
   const size_t smem = (size_t)H * sizeof(float);
   if (smem > 48 * 1024) cudaFuncSetAttribute(add_normed_kernel<TO, W>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   // few rows (single-token steps): a thread an element or a handful, so that each pass is one trip to memory; many rows:
@@ -175,20 +180,21 @@ static int add_normed_launch(float* h, const void* a, int a_dt, const float* ga,
   const int per = (H / W + 31) / 32 * 32;
   const int nt = R <= 296 ? (per > 1024 ? 1024 : (per < 128 ? 128 : per)) : 256;
   return sx_launch(add_normed_kernel<TO, W>, dim3(R), dim3(nt), smem, stream, h, a, a_dt, ga, b, b_dt, gb, factor, gp, go, eps,
-                   (TO*)y, rows, H, write_h, place, wts, top);
+                   (TO*)y, rows, H, write_h, place, wts, top, vec);
 }
 
 extern "C" int sx_add_normed(float* h, const void* a, int a_dt, const float* ga, const void* b, int b_dt, const float* gb,
                              float factor, const float* gp, const float* go, float eps, void* y, int y_dt, const int* rows,
-                             int R, int H, int write_h, const int* place, const float* wts, int top, cudaStream_t stream) {
+                             int R, int H, int write_h, const int* place, const float* wts, int top, const float* vec,
+                             cudaStream_t stream) {
   if (R <= 0) return 0;
   if (H <= 0 || (b != nullptr && (a == nullptr || ga == nullptr || gb == nullptr))) return SX_ERR_SIZE;
   if (place != nullptr && (a == nullptr || a_dt != SX_F32 || ga != nullptr || wts == nullptr || top <= 0)) return SX_ERR_SIZE;
-  if ((size_t)H * sizeof(float) > 200 * 1024) return SX_ERR_SIZE;
+  if ((size_t)H * sizeof(float) > 200 * 1024 || (vec != nullptr && h == nullptr)) return SX_ERR_SIZE;
   const uintptr_t all = (uintptr_t)h | (uintptr_t)a | (uintptr_t)ga | (uintptr_t)b | (uintptr_t)gb | (uintptr_t)gp | (uintptr_t)go |
-                        (uintptr_t)y;
+                        (uintptr_t)y | (uintptr_t)vec;
   const bool v4 = (H % 4 == 0) && (all % 16 == 0);
-#define AN_GO(TO, W) return add_normed_launch<TO, W>(h, a, a_dt, ga, b, b_dt, gb, factor, gp, go, eps, y, rows, R, H, write_h, place, wts, top, stream)
+#define AN_GO(TO, W) return add_normed_launch<TO, W>(h, a, a_dt, ga, b, b_dt, gb, factor, gp, go, eps, y, rows, R, H, write_h, place, wts, top, vec, stream)
   if (y == nullptr || y_dt == SX_F32) { if (v4) AN_GO(float, 4); AN_GO(float, 1); }
   if (y_dt == SX_BF16) { if (v4) AN_GO(bf16, 4); AN_GO(bf16, 1); }
 #undef AN_GO

@@ -25,7 +25,7 @@ import torch
 
 from ..cache.store import CacheRequest
 from .. import ops
-from ..parts.base import Norm, Part, PendingLinear, Runtime, StepContext, plain, to_device_f32
+from ..parts.base import Norm, NormedDelta, Part, PendingLinear, Runtime, StepContext, plain, to_device_f32
 from ..parts.embedding import Embedding, OutputHead
 from ..weights.loader import TensorSpec, WeightSource, bind_tensors
 
@@ -137,6 +137,11 @@ class DecoderModel(Part):
         n_run = 0
         for run in self.steps:
             if isinstance(run, Inject):
+                if (isinstance(pending, NormedDelta) and pending.is_rms and pending.vec is None and not run.embedding
+                        and run.row is not None and observe is None):
+                    # a branch that is normed on its way into the stream takes the vector along in the same kernel
+                    pending = pending.with_vector(self.stream_vectors.table[run.row])
+                    continue
                 ops.stream_add(h, plain(pending), h0 if run.embedding else None,
                                self.stream_vectors.table[run.row] if run.row is not None else None)
                 pending = None

@@ -86,12 +86,12 @@ def delta_rule(proj: torch.Tensor, col: int, b_col: int, heads: int, kv_heads: i
         n = ctx.n_seqs * chunks * heads
         x, qg, kd = (torch.empty((n, C_, dim), **f32) for _ in range(3))
         y, p, ge = torch.empty((n, C_, vdim), **f32), torch.empty((n, C_, C_), **f32), torch.empty((n, dim), **f32)
-        o = torch.empty((T, heads * vdim), **f32)
+        sb = torch.empty((n, dim, vdim), **f32)
         # narrow slices of the state where wide ones would leave SMs idle
         sms = torch.cuda.get_device_properties(proj.device).multi_processor_count
         slice_ = 32 if ctx.n_seqs * heads * ((vdim + 31) // 32) >= sms else 16
         check(fn("delta", "sx_delta_chunks")(*common(), ptr(q), ptr(k), ptr(v), ptr(x), ptr(qg), ptr(kd), ptr(y), ptr(p), ptr(ge),
-                                             ptr(o), c_int(chunks), c_int(slice_), stream()), "delta_chunks", launches=3)
+                                             ptr(sb), c_int(chunks), c_int(slice_), stream()), "delta_chunks", launches=3)
     else:
         check(fn("delta", "sx_delta_walk")(*common(), ptr(q), ptr(k), ptr(v), stream()), "delta_walk")
     return out

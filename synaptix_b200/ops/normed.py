@@ -33,14 +33,15 @@ class WeightedRows:
 
 def add_normed(h: Optional[torch.Tensor], terms: Sequence, post_gain: Optional[torch.Tensor], eps: float,
                out_dtype: Optional[torch.dtype], *, factor: float = 1.0, out_gain: Optional[torch.Tensor] = None,
-               rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+               rows: Optional[torch.Tensor] = None, vec: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """One pass per row over a branch on its way into the residual stream ``h`` (float32 ``[T, width]``, summed into in
     place unless ``rows`` is given; ``None``: there is no stream and the result is the branch alone).
 
     ``terms``: none (nothing is added), one ``(x, None)`` (the branch is ``x``; ``x`` may be a ``WeightedRows``, the
     weighted sum of rows that a mixture of experts hands on), or one or two ``(x_i, gain_i)``: the
     branch is ``factor * sum_i rms_norm(x_i) * gain_i`` (mixers side by side, each with a norm of its own).  With
-    ``post_gain`` the branch is normed once more, ``rms_norm(branch) * post_gain``, before it is added.  Returned: the
+    ``post_gain`` the branch is normed once more, ``rms_norm(branch) * post_gain``, before it is added.  ``vec`` (float32 over the width) is added into every
+    row of the stream as well.  Returned: the
     rows after the sum in ``out_dtype`` (what the next sublayer reads), or ``rms_norm`` of them times ``out_gain``; all
     rows or ``rows`` (int32) only; ``out_dtype=None``: nothing is returned.  Norms and sums are 32-bit."""
     terms = list(terms)
@@ -58,7 +59,7 @@ def add_normed(h: Optional[torch.Tensor], terms: Sequence, post_gain: Optional[t
             raise KernelError("add_normed: the rows of a weighted sum are float32")
     else:
         a_shape = None if a is None else tuple(a.shape)
-    require_cuda(h, a, ga, b, gb, post_gain, out_gain, rows, place, wts)
+    require_cuda(h, a, ga, b, gb, post_gain, out_gain, rows, place, wts, vec)
     if h is None and a is None:
         raise KernelError("add_normed: neither a stream nor a branch")
     T, H = h.shape if h is not None else a_shape
@@ -67,9 +68,9 @@ def add_normed(h: Optional[torch.Tensor], terms: Sequence, post_gain: Optional[t
     ref = h if h is not None else a
     if b is not None and tuple(b.shape) != (T, H):
         raise KernelError("add_normed: a branch must have the stream's shape")
-    for g in (ga, gb, post_gain, out_gain):
+    for g in (ga, gb, post_gain, out_gain, vec):
         if g is not None and (g.dtype != torch.float32 or g.numel() != H):
-            raise KernelError("add_normed: gains are float32 vectors over the width")
+            raise KernelError("add_normed: gains and added vectors are float32 over the width")
     if h is not None and h.dtype != torch.float32:
         raise KernelError("add_normed: the residual stream is float32")
     R = T if rows is None else rows.numel()
@@ -78,7 +79,8 @@ def add_normed(h: Optional[torch.Tensor], terms: Sequence, post_gain: Optional[t
         ptr(h), ptr(a), c_int(dt_code(a.dtype) if a is not None else 0), ptr(ga), ptr(b),
         c_int(dt_code(b.dtype) if b is not None else 0), ptr(gb), c_float(factor), ptr(post_gain), ptr(out_gain), c_float(eps),
         ptr(y), c_int(dt_code(out_dtype) if out_dtype is not None else 0), ptr(rows), c_int(R), c_int(H),
-        c_int(1 if (rows is None and h is not None) else 0), ptr(place), ptr(wts), c_int(top), stream()), "add_normed")
+        c_int(1 if (rows is None and h is not None) else 0), ptr(place), ptr(wts), c_int(top), ptr(vec), stream()),
+        "add_normed")
     return y
 
 

@@ -183,12 +183,13 @@ class NormedDelta:
     ``mult * norm(x + bias)`` as one float32 tensor.
 
     ``norm`` may also be an RMS norm (it has no ``bias`` vector; ``mult`` is then 1 and there is no product bias), and
-    ``x`` may then be a ``NormedSum`` or a mixture of experts' ``WeightedRows``."""
-    __slots__ = ("x", "norm", "mult", "bias", "_sum")
+    ``x`` may then be a ``NormedSum`` or a mixture of experts' ``WeightedRows``.  Such a branch may also carry ``vec``, a
+    float32 vector over the width that is added into every row of the stream along with it (``with_vector``)."""
+    __slots__ = ("x", "norm", "mult", "bias", "vec", "_sum")
 
     def __init__(self, x, norm, mult: float = 1.0, bias=None):
         self.x, self.norm, self.mult, self.bias = x, norm, float(mult), bias
-        self._sum = None
+        self.vec = self._sum = None
         if not hasattr(norm, "bias") and (self.mult != 1.0 or bias is not None):
             raise ValueError("a branch behind an RMS norm has neither a factor nor a product bias")
 
@@ -199,6 +200,12 @@ class NormedDelta:
     @property
     def is_rms(self) -> bool:
         return not hasattr(self.norm, "bias")
+
+    def with_vector(self, vec: torch.Tensor) -> "NormedDelta":
+        """The same branch behind an RMS norm, with ``vec`` to be added beside it."""
+        out = NormedDelta(self.x, self.norm)
+        out.vec = vec
+        return out
 
     def rms_terms(self):
         """``(terms, factor)`` as ``ops.add_normed`` takes them."""
@@ -214,7 +221,10 @@ class NormedDelta:
             from .. import ops
             if self.is_rms:
                 terms, factor = self.rms_terms()
-                self._sum = ops.add_normed(None, terms, self.norm.weight, self.norm.eps, torch.float32, factor=factor)
+                base = None
+                if self.vec is not None:         # onto rows of zeros, so that the vector joins them
+                    base = torch.zeros(tuple(self.shape), dtype=torch.float32, device=self.vec.device)
+                self._sum = ops.add_normed(base, terms, self.norm.weight, self.norm.eps, torch.float32, factor=factor, vec=self.vec)
                 return self._sum
             zero = torch.zeros(self.x.shape, dtype=torch.float32, device=self.x.device)
             _, self._sum = ops.add_layernorm(zero, self.x, self.norm.weight, self.norm.bias, self.norm.eps, torch.float32,

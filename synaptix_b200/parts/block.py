@@ -195,7 +195,7 @@ class ParallelBlock(Part):
         if isinstance(pending, NormedDelta) and pending.is_rms and pending.norm.eps == self.norm1.eps and len(gains) == 1:
             # a branch with a norm of its own: its norm, the sum and this block's norm in one kernel
             terms, factor = pending.rms_terms()
-            x = ops.add_normed(h, terms, pending.norm.weight, self.norm1.eps, dtype, factor=factor, out_gain=gains[0])
+            x = ops.add_normed(h, terms, pending.norm.weight, self.norm1.eps, dtype, factor=factor, out_gain=gains[0], vec=pending.vec)
             return x, x
         if isinstance(pending, ScaledSum):
             terms = pending.terms
@@ -331,7 +331,7 @@ class PostNormBlock(Part):
         want = None if dtype == torch.float32 else dtype
         if isinstance(pending, NormedDelta) and pending.is_rms:
             terms, factor = pending.rms_terms()
-            x = ops.add_normed(h, terms, pending.norm.weight, pending.norm.eps, want, factor=factor)
+            x = ops.add_normed(h, terms, pending.norm.weight, pending.norm.eps, want, factor=factor, vec=pending.vec)
         else:
             pending = plain(pending)
             if pending is None and want is None:

@@ -49,7 +49,7 @@ class RMSNorm(Norm):
             # the branch's norm, the sum into the stream and this norm in one kernel
             terms, factor = delta.rms_terms()
             return ops.add_normed(h, terms, delta.norm.weight, self.eps, self._dtype, factor=factor, out_gain=self.weight,
-                                  rows=rows)
+                                  rows=rows, vec=delta.vec)
         if isinstance(delta, NormedDelta):
             delta = delta.materialize()
         if isinstance(delta, ScaledSum):
