@@ -12,7 +12,7 @@ from typing import Optional
 import torch
 
 from ..csrc.build import KernelsUnavailable
-from ._lib import KernelError, current_gate, gate_activation, set_launch_counter
+from ._lib import KernelError, current_gate, gate_activation, late_launch, set_launch_counter
 from .attention import (TC_TILE_ROWS, attn_decode, attn_decode_ex, attn_decode_prep, attn_decode_tma, attn_prefill,
                         attn_prefill_ex, attn_prefill_tc,
                         fast_supported, pick_splits, query_tiles, tc_prefill_supported, tma_decode_supported)
@@ -41,7 +41,7 @@ __all__ = ["OPTIONS", "KernelOptions", "options", "set_options", "KernelsUnavail
            "add_rmsnorm_conv", "capped_glu", "mingru", "retention", "stream_add", "gate_activation",
            "add_normed", "WeightedRows", "embed_bigram", "convqk_prepare", "sigmoid_gate", "add_scaled", "add_scaled_rmsnorm", "scale_rows", "add_layernorm", "attn_scored", "heads_prepare", "latent_attention", "latent_output", "latent_prepare",
            "latent_query", "latent_gather", "latent_expand", "latent_rotate_q", "head_gate", "mlstm", "ExpertPlan", "moe_combine", "moe_down", "moe_gate_up", "moe_route", "moe_sort", "moe_up",
-           "side_gate", "DeltaWeights", "delta_rule", "delta_step_fits"]
+           "late_launch", "side_gate", "DeltaWeights", "delta_rule", "delta_step_fits"]
 
 
 _STATUS_READERS = {"gemm_tc": ("the tcgen05 matrix product (gemm_tc)", "gemm_tc_status"),

@@ -8,6 +8,7 @@ from typing import Optional
 import torch
 
 from ..csrc.build import KernelsUnavailable, load_library
+from .options import OPTIONS as _PDL_OPTION
 
 _DT = {torch.float32: 0, torch.bfloat16: 1}
 
@@ -88,7 +89,7 @@ def _library(lib: str):
     h = _LIBS.get(lib)
     if h is None:
         h = _LIBS[lib] = load_library(lib)
-        _set_pdl(h)
+        _set_pdl(lib)
     return h
 
 
@@ -96,17 +97,43 @@ def loaded(lib: str) -> bool:
     return lib in _LIBS
 
 
-def _set_pdl(handle) -> None:
-    from .options import OPTIONS
-    f = getattr(handle, "sx_set_pdl", None)
+# Whether kernels are launched with programmatic dependent launch: the option of that name, and off inside
+# ``late_launch``.  A library is told when one of its functions is next asked for.
+_LATE = [0]
+_LIB_PDL = {}
+
+
+def _want_pdl() -> bool:
+    return bool(_PDL_OPTION.pdl) and not _LATE[0]
+
+
+def _set_pdl(lib: str) -> None:
+    want = _want_pdl()
+    f = getattr(_LIBS[lib], "sx_set_pdl", None)
     if f is not None:
-        f(ctypes.c_int(1 if OPTIONS.pdl else 0))
+        f(ctypes.c_int(1 if want else 0))
+    _LIB_PDL[lib] = want
 
 
 def apply_pdl() -> None:
     """Tell every loaded library whether kernels are launched with programmatic dependent launch."""
-    for h in _LIBS.values():
-        _set_pdl(h)
+    for lib in _LIBS:
+        _set_pdl(lib)
+
+
+@contextlib.contextmanager
+def late_launch(on: bool = True):
+    """Kernels launched inside are scheduled when the kernel before them has ended, not while it runs.  For a kernel whose
+    blocks would otherwise hold the SMs' shared memory and registers, waiting, while another branch's kernel that could
+    run looks for room (blocks that run beside each other on two streams)."""
+    if not on:
+        yield
+        return
+    _LATE[0] += 1
+    try:
+        yield
+    finally:
+        _LATE[0] -= 1
 
 
 def fn(lib: str, name: str):
@@ -116,6 +143,8 @@ def fn(lib: str, name: str):
         f = getattr(_library(lib), name)
         f.restype = ctypes.c_int
         _FN_CACHE[key] = f
+    if _LIB_PDL[lib] is not (not _LATE[0] and _PDL_OPTION.pdl):
+        _set_pdl(lib)
     return f
 
 

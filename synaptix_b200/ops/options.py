@@ -29,7 +29,8 @@ switches in its runtime options (crates/synaptix-config/src/runtime.rs, ``AttnBa
 ``branch_streams``  single-token steps of a block whose mixer and feed-forward read the same stream: the feed-forward's
                     kernels run on a second CUDA stream beside the mixer's (inside a captured step: two branches of
                     the graph), else one after the other; likewise the second of two mixers that run side by side
-                    behind norms of their own
+                    behind norms of their own.  A branch's last product is then launched late (``late_launch``): scheduled
+                    early it holds the room that the other branch's kernels need (a Zekalorn step at batch 1: 0.87 -> 0.70 ms)
 """
 from __future__ import annotations
 

@@ -62,11 +62,12 @@ class StepContext:
     """
     __slots__ = ("token_ids", "positions", "seq_of_token", "cu_seqlens", "seq_past", "seq_lens",
                  "seq_slots", "block_tables", "want_rows", "n_tokens", "n_seqs", "n_want",
-                 "max_new", "max_len", "all_single", "runtime", "scratch", "host", "want_all", "observe")
+                 "max_new", "max_len", "all_single", "runtime", "scratch", "host", "want_all", "observe", "branches")
 
     def __init__(self, **kw):
         self.scratch = {}
         self.host = None
+        self.branches = False      # inside a block whose branches run on two streams: last products launch late (ops.late_launch)
         self.want_all = False      # want_rows is 0..n_tokens-1 in order
         self.observe = None        # callable(run number, h, pending): called after every layer run (debugging, tests)
         for k, v in kw.items():

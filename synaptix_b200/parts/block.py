@@ -221,11 +221,15 @@ class ParallelBlock(Part):
                 fork = torch.cuda.Event()
                 fork.record(main)
                 side.wait_event(fork)
-                with torch.cuda.stream(side):
-                    b = self._ffn(x2, ctx)
-                    join = torch.cuda.Event()
-                    join.record(side)
-                a = self.mixer.forward(x1, ctx, cache_view, write_cache)
+                ctx.branches = True
+                try:
+                    with torch.cuda.stream(side):
+                        b = self._ffn(x2, ctx)
+                        join = torch.cuda.Event()
+                        join.record(side)
+                    a = self.mixer.forward(x1, ctx, cache_view, write_cache)
+                finally:
+                    ctx.branches = False
                 main.wait_event(join)
             else:
                 a = self.mixer.forward(x1, ctx, cache_view, write_cache)

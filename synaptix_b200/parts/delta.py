@@ -114,4 +114,7 @@ class ChannelDelta(Mixer):
             a = ops.linear(x, self.proj[:lr_col])                   # q, k, v and the step sizes
             z = ops.linear(ops.linear(x, self.proj[lr_col:]), self.low_rank, out_dtype=torch.float32)
             y = ops.delta_rule(a, 0, C, *args, z=z)
-        return self.o.deferred(y) if defer_output else self.o.forward(y)
+        if defer_output:
+            return self.o.deferred(y)
+        with ops.late_launch(ctx.branches):
+            return self.o.forward(y)

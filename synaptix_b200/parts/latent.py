@@ -162,4 +162,5 @@ class LatentAttention(Mixer):
         qa = ops.latent_query(q, self.uk, self.heads, self.dim, self.rot_dim, self.kv_rank, inv_freq, rot_dims, pairs, ctx, mag)
         ol = ops.latent_attention(qa, cache_view.k, ctx, bt, self.heads, self.kv_rank, self.rot_dim, self.scale, self.window)
         y = ops.latent_output(ol, self.uv, self.heads, self.vdim, self.kv_rank, p, self.col_g, x.dtype)
-        return self.o.forward(y)
+        with ops.late_launch(ctx.branches):
+            return self.o.forward(y)

@@ -46,7 +46,10 @@ class SwiGLU(FeedForward):
 
     def forward(self, x: torch.Tensor, ctx: StepContext, defer_output: bool = False) -> torch.Tensor:
         z = self.gate_up.forward(x, epilogue="silu_mul")
-        return self.down.deferred(z) if defer_output else self.down.forward(z)
+        if defer_output:
+            return self.down.deferred(z)
+        with ops.late_launch(ctx.branches):
+            return self.down.forward(z)
 
 
 class CappedGLU(FeedForward):
@@ -154,7 +157,8 @@ class MixtureOfExperts(FeedForward):
                 z = ops.moe_gate_up(x, self.gate_up, plan, self.top)
         else:
             z = ops.moe_gate_up(x, self.gate_up, plan, self.top)
-        y = ops.moe_down(z, self.down, plan)
+        with ops.late_launch(ctx.branches):
+            y = ops.moe_down(z, self.down, plan)
         if defer_combine:           # a block that norms this branch on its way into the stream forms the sum there
             return ops.WeightedRows(y, plan.place, weights, x.dtype)
         return ops.moe_combine(y, plan, weights, x.dtype)

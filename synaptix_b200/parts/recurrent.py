@@ -202,4 +202,6 @@ class MLSTM(Mixer):
                          state[0], state[1], state[2], ctx)
 
     def forward(self, x: torch.Tensor, ctx: StepContext, state, write_cache: bool = True):
-        return self.o.forward(self.mix(self.proj.forward(x), 0, ctx, state, write_cache, x=x))
+        y = self.mix(self.proj.forward(x), 0, ctx, state, write_cache, x=x)
+        with ops.late_launch(ctx.branches):
+            return self.o.forward(y)

@@ -165,4 +165,5 @@ class ScoredAttention(Mixer):
         a = ops.attn_scored(q, cache_view.k, cache_view.v, ctx, bt, self.nh, self.nkv, self.hd, self.vd, self.scale,
                             self.window, talk=self.talk_matrix, head_bias=self.head_bias_vector,
                             dist_bias=self.distance_table, softmax=self.softmax, gate=gate)
-        return self.o.forward(a)
+        with ops.late_launch(ctx.branches):
+            return self.o.forward(a)
