@@ -162,37 +162,31 @@ __device__ __forceinline__ void dl_prepare_run(const DlArgs& a, const DlPrep& w,
   const T* src = (const T*)a.proj + a.col + c;
   float wt[CPL][TAPS], win[TAPS][CPL];            // win[j]: the row that tap j reads
   float raw[DL_RUN][CPL];                         // the run's rows, all asked for at once
-  int seqs[DL_RUN];
 #pragma unroll
-  for (int r = 0; r < DL_RUN; ++r) {
-    const int t = min(t0 + r, t1 - 1);
-    seqs[r] = a.seq_of_token[t];
-    DlLd<T, CPL>::go(src + (size_t)t * a.row, raw[r]);
+  for (int r = 0; r < DL_RUN; ++r) DlLd<T, CPL>::go(src + (size_t)min(t0 + r, t1 - 1) * a.row, raw[r]);
+  const int s = a.seq_of_token[t0], pos = a.positions[t0], past = a.seq_past[s];
+  const float* hs = a.hist + (size_t)a.seq_slots[s] * TAPS * C + c;
+#pragma unroll
+  for (int j = 0; j < TAPS - 1; ++j) {
+    const int p = pos - TAPS + 1 + j;             // goes to place j + 1: the shift below brings it to place j
+    if (p < 0) {
+#pragma unroll
+      for (int i = 0; i < CPL; ++i) win[j + 1][i] = 0.f;
+    } else if (p >= past) {
+      DlLd<T, CPL>::go(src + (size_t)(t0 - (pos - p)) * a.row, win[j + 1]);
+    } else {
+      dl_ld_f32<CPL>(hs + (size_t)(p % TAPS) * C, win[j + 1]);
+    }
   }
 #pragma unroll
   for (int i = 0; i < CPL; ++i)
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) wt[i][j] = a.taps_w[(size_t)(c + i) * TAPS + j];
+  float* dst = dl_prep_dst(a, w, t0, unit, kind) + lane * CPL;
+  const size_t ld = kind == 2 ? (size_t)a.H * a.V : (size_t)a.G * a.D;
 #pragma unroll
   for (int r = 0; r < DL_RUN; ++r) {
-    const int t = t0 + r;
-    if (t >= t1) break;
-    if (r == 0 || seqs[r] != seqs[r - 1]) {       // the run's first token, or another sequence's: fetch the rows before it
-      const int s = seqs[r], pos = a.positions[t], past = a.seq_past[s];
-      const float* hs = a.hist + (size_t)a.seq_slots[s] * TAPS * C + c;
-#pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) {
-        const int p = pos - TAPS + 1 + j;         // goes to place j + 1: the shift below brings it to place j
-        if (p < 0) {
-#pragma unroll
-          for (int i = 0; i < CPL; ++i) win[j + 1][i] = 0.f;
-        } else if (p >= past) {
-          DlLd<T, CPL>::go(src + (size_t)(t - (pos - p)) * a.row, win[j + 1]);
-        } else {
-          dl_ld_f32<CPL>(hs + (size_t)(p % TAPS) * C, win[j + 1]);
-        }
-      }
-    }
+    if (t0 + r >= t1) break;
 #pragma unroll
     for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
@@ -213,7 +207,6 @@ __device__ __forceinline__ void dl_prepare_run(const DlArgs& a, const DlPrep& w,
 #pragma unroll
       for (int i = 0; i < CPL; ++i) y[i] *= f;
     }
-    float* dst = dl_prep_dst(a, w, t, unit, kind) + lane * CPL;
     if (CPL % 4 == 0) {
 #pragma unroll
       for (int i = 0; i < CPL / 4; ++i)
@@ -222,6 +215,7 @@ __device__ __forceinline__ void dl_prepare_run(const DlArgs& a, const DlPrep& w,
 #pragma unroll
       for (int i = 0; i < CPL; ++i) dst[i] = y[i];
     }
+    dst += ld;
   }
 }
 
@@ -232,14 +226,19 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prepare_run_kernel(DlArgs a,
   pdl_trigger();
   const int unit = blockIdx.y * (DL_THREADS / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (unit >= 2 * a.G + a.H) return;
-  const int t0 = blockIdx.x * DL_RUN, t1 = min(n_tokens, t0 + DL_RUN);
+  const int begin = blockIdx.x * DL_RUN, end = min(n_tokens, begin + DL_RUN);
   int c0, n, kind;
   dl_unit(a, unit, c0, n, kind);
-  switch (n) {
-    case 32: dl_prepare_run<T, 1, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;
-    case 64: dl_prepare_run<T, 2, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;
-    case 128: dl_prepare_run<T, 4, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;
-    default: if (WIDE) dl_prepare_run<T, 8, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;
+  // a run that lies in one sequence goes through whole, others in stretches of a sequence each
+  for (int t0 = begin; t0 < end;) {
+    const int t1 = min(end, a.cu_seqlens[a.seq_of_token[t0] + 1]);
+    switch (n) {
+      case 32: dl_prepare_run<T, 1, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;
+      case 64: dl_prepare_run<T, 2, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;
+      case 128: dl_prepare_run<T, 4, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;
+      default: if (WIDE) dl_prepare_run<T, 8, TAPS>(a, w, t0, t1, unit, c0, kind, lane); break;
+    }
+    t0 = t1;
   }
 }
 
@@ -558,7 +557,8 @@ static bool dl_step_fits(int D, int V, int ra, int rg) {
 extern "C" int sx_delta_step_fits(int D, int V, int ra, int rg) { return dl_step_fits(D, V, ra, rg) ? 1 : 0; }
 
 // ---------------------------------------------------------------------------------------------------------------
-// chunks.  Scratch per (sequence, chunk, head): x, qg, kd [32, D] each, y [32, V], p [32, 32], ge [D], sb [D, V] (the state
+// chunks, numbered through the step: chunk p of sequence s is number cu_seqlens[s] / 32 + s + p, so that sequences of
+// unequal lengths need no more than (tokens / 32 + sequences) of them.  Scratch per (chunk, head): x, qg, kd [32, D] each, y [32, V], p [32, 32], ge [D], sb [D, V] (the state
 // at the chunk's begin).
 // ---------------------------------------------------------------------------------------------------------------
 struct DlChunks { float* x; float* qg; float* kd; float* y; float* p; float* ge; float* sb; int P; };
@@ -578,7 +578,7 @@ __global__ void __launch_bounds__(DL_THREADS, 3) delta_intra_kernel(DlArgs a, Dl
   const int t0 = a.cu_seqlens[s] + p * DL_C, len = a.cu_seqlens[s + 1] - t0;
   if (len <= 0) return;
   const int L = min(DL_C, len);
-  const size_t ci = ((size_t)s * ch.P + p) * H + h;
+  const size_t ci = (size_t)(a.cu_seqlens[s] / DL_C + s + p) * H + h;
   const int D4 = D >> 2;
   for (int i = tid; i < DL_C * D4; i += DL_THREADS) {
     const int t = i / D4, d = (i - t * D4) * 4;
@@ -594,18 +594,31 @@ __global__ void __launch_bounds__(DL_THREADS, 3) delta_intra_kernel(DlArgs a, Dl
   dl_commit();
   if (tid < DL_C) bs[tid] = tid < L ? dl_sigmoid(to_f32(((const TP*)a.proj)[(size_t)(t0 + tid) * a.row + a.b_col + h])) : 0.f;
   for (int i = tid; i < DL_C * DL_LD; i += DL_THREADS) As[i] = 0.f;
+  // the right sides of the value columns come early too: their loads run beside the others
+  float rhs[DL_C];
+  if (tid >= D && tid < D + V) {
+    const float* vp = w.v + (size_t)t0 * H * V + h * V + (tid - D);
+#pragma unroll
+    for (int t = 0; t < DL_C; ++t) {
+      rhs[t] = *vp;                                  // rows behind the chunk's end: its last row again, times 0 below
+      if (t + 1 < L) vp += (size_t)H * V;
+    }
+  }
   {   // running sums: a thread a channel and half of the chunk (D <= 128) or a channel
     const int parts = D <= DL_THREADS / 2 ? 2 : 1, part = parts == 2 && tid >= DL_THREADS / 2 ? 1 : 0, d = tid - part * (DL_THREADS / 2);
-    const int ta = part * 16, tb = parts == 2 ? ta + 16 : DL_C;
-    float acc = 0.f;
     if (d < D) {
       const float ea = -expf(a.a_log[h]) * DL_LOG2E, c = a.dt_bias[h * D + d];
-      const float* z = a.z + (size_t)t0 * a.z_ld + h * D + d;
-#pragma unroll 8
-      for (int t = ta; t < tb; ++t) {
-        if (t == 16) acc = 0.f;
-        if (t < L) acc += fmaxf(ea * dl_softplus(z[(size_t)t * a.z_ld] + c), DL_LOG_MIN);
-        Gs[t * DS + d] = acc;
+      for (int half = part; half < (parts == 2 ? part + 1 : 2); ++half) {
+        const float* z = a.z + (size_t)(t0 + half * 16) * a.z_ld + h * D + d;
+        const int n = L - half * 16;                 // rows of this half
+        float zz[16], acc = 0.f;
+#pragma unroll
+        for (int t = 0; t < 16; ++t) zz[t] = t < n ? z[(size_t)t * a.z_ld] : 0.f;
+#pragma unroll
+        for (int t = 0; t < 16; ++t) {
+          if (t < n) acc += fmaxf(ea * dl_softplus(zz[t] + c), DL_LOG_MIN);
+          Gs[(half * 16 + t) * DS + d] = acc;
+        }
       }
     }
     dl_wait<0>();
@@ -644,7 +657,6 @@ __global__ void __launch_bounds__(DL_THREADS, 3) delta_intra_kernel(DlArgs a, Dl
   }
   __syncthreads();
   // a thread a channel: what the scan reads, the right side b e^G k in registers, then k and q around the border (token 15)
-  float rhs[DL_C];
   float* X = ch.x + ci * DL_C * D;
   if (tid < D) {
     float* Q = ch.qg + ci * DL_C * D + tid;
@@ -666,12 +678,8 @@ __global__ void __launch_bounds__(DL_THREADS, 3) delta_intra_kernel(DlArgs a, Dl
       Q += D; K += D; gp += DS; kp += DS; qp += DS;
     }
   } else if (tid < D + V) {
-    const float* vp = w.v + (size_t)t0 * H * V + h * V + (tid - D);
 #pragma unroll
-    for (int t = 0; t < DL_C; ++t) {
-      rhs[t] = t < L ? bs[t] * *vp : 0.f;
-      if (t + 1 < L) vp += (size_t)H * V;
-    }
+    for (int t = 0; t < DL_C; ++t) rhs[t] *= bs[t];          // 0 behind the chunk's end
   }
   __syncthreads();
   {   // pairs across the border: row 16 + i, column j
@@ -727,13 +735,14 @@ __global__ void __launch_bounds__(DL_THREADS, 3) delta_intra_kernel(DlArgs a, Dl
 static size_t dl_intra_smem(int D) { return (size_t)(3 * DL_C * (D + 4) + DL_C * DL_LD + DL_C) * sizeof(float); }
 
 
-// VS: columns of the state a block owns (16 or 32); ND: tiles of the state a thread owns (D <= 128 ND)
+// VS: columns of the state a block owns (16 or 32); ND: tiles of the state a thread owns (D <= 128 ND).
+#define DL_SCAN_THREADS 256
 template <int VS, int ND>
-__global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DlArgs a, DlChunks ch) {
+__global__ void __launch_bounds__(DL_SCAN_THREADS) delta_scan_kernel(DlArgs a, DlChunks ch) {
   extern __shared__ __align__(16) float sm[];
   constexpr int SS = VS + 4;
   constexpr int CG = VS / 4;                       // groups of four columns in the product with S
-  constexpr int KSPLIT = DL_THREADS / (8 * CG);    // 8 or 4: parts of D in that product
+  constexpr int KSPLIT = DL_SCAN_THREADS / (8 * CG);   // 8 or 4: parts of D in that product
   constexpr int CP = VS / 8;                       // columns a thread of u and of the state's tiles
   const int D = a.D, V = a.V, H = a.H, DS = D + 4;
   float* xs = sm;                                  // 2 * 32 * DS: X, two chunks
@@ -748,37 +757,44 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DlArgs a, DlChun
   if (np <= 0) return;
   float* Sg = a.S + ((size_t)a.seq_slots[s] * H + h) * D * V;
   const int D4 = D >> 2;
-  auto chunk = [&](int p) { return ((size_t)s * ch.P + p) * H + h; };
-  auto load = [&](int p) {
-    const float *x = ch.x + chunk(p) * DL_C * D, *k = ch.kd + chunk(p) * DL_C * D;
-    float *xd = xs + (p & 1) * DL_C * DS, *kk = kd + (p & 1) * DL_C * DS;
-    for (int d = (tid & 31) * 4; d < D; d += 128)
+  const size_t c0 = (size_t)(tok0 / DL_C + s) * H + h;      // the first chunk; the next lies H further
+  // pointers that walk from chunk to chunk
+  const float *xg = ch.x + c0 * DL_C * D + (tid >> 5) * D + (tid & 31) * 4, *kg_ = ch.kd + c0 * DL_C * D + (tid >> 5) * D + (tid & 31) * 4;
+  const size_t step_x = (size_t)H * DL_C * D;
+  const int soff = (tid >> 5) * DS + (tid & 31) * 4;
+  auto load = [&](int p) {                         // called for 0, 1, 2, ... in order
+    float *xd = xs + (p & 1) * DL_C * DS + soff, *kk = kd + (p & 1) * DL_C * DS + soff;
+    for (int d = (tid & 31) * 4, o = 0; d < D; d += 128, o += 128)
 #pragma unroll
-      for (int t = 0; t < DL_C; t += DL_THREADS / 32) {
-        const int r = t + (tid >> 5);
-        dl_cp16(xd + r * DS + d, x + r * D + d);
-        dl_cp16(kk + r * DS + d, k + r * D + d);
+      for (int t = 0; t < DL_C; t += DL_SCAN_THREADS / 32) {
+        dl_cp16(xd + t * DS + o, xg + t * D + o);
+        dl_cp16(kk + t * DS + o, kg_ + t * D + o);
       }
+    xg += step_x;
+    kg_ += step_x;
   };
   // this thread's place in u (row ur, CP columns from uc on) and in the state (rows 4 sd .., the same columns)
   const int ur = tid >> 3, uc = (tid & 7) * CP, sd = tid >> 3;
   float st[ND][4][CP], y[CP], ge[ND][4];
-  auto load_small = [&](int p) {                   // what goes to registers: u's right side, the chunk's whole decay
-    const float* yg = ch.y + chunk(p) * DL_C * V + (size_t)ur * V + v0 + uc;
+  float* yg = ch.y + c0 * DL_C * V + (size_t)ur * V + v0 + uc;         // this chunk's right side (and then its u)
+  const float* gg = ch.ge + c0 * D;
+  float* sb = ch.sb + c0 * D * V + (size_t)sd * 4 * V + v0 + uc;
+  const size_t step_y = (size_t)H * DL_C * V, step_s = (size_t)H * D * V;
+  auto load_small = [&](const float* yg, const float* gg) {            // u's right side and the chunk's whole decay, to registers
 #pragma unroll
     for (int j = 0; j < CP; ++j) y[j] = v0 + uc + j < V ? yg[j] : 0.f;
 #pragma unroll
     for (int b = 0; b < ND; ++b) {
       const int d = (sd + 32 * b) * 4;
       if (d < D) {
-        const float4 f = *reinterpret_cast<const float4*>(ch.ge + chunk(p) * D + d);
+        const float4 f = *reinterpret_cast<const float4*>(gg + d);
         ge[b][0] = f.x; ge[b][1] = f.y; ge[b][2] = f.z; ge[b][3] = f.w;
       }
     }
   };
   load(0);
   dl_commit();
-  load_small(0);
+  load_small(yg, gg);
 #pragma unroll
   for (int b = 0; b < ND; ++b)
 #pragma unroll
@@ -791,7 +807,6 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DlArgs a, DlChun
   const int dper = (D4 + KSPLIT - 1) / KSPLIT * 4, da = kg * dper, db = min(D, da + dper);
   for (int p = 0; p < np; ++p) {
     // the state at the chunk's begin: to shared memory for the product, to memory for the output kernel
-    float* sb = ch.sb + chunk(p) * D * V;
 #pragma unroll
     for (int b = 0; b < ND; ++b)
 #pragma unroll
@@ -800,13 +815,14 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DlArgs a, DlChun
         if (d < D) {
 #pragma unroll
           for (int j = 0; j < CP; ++j) S[d * SS + uc + j] = st[b][i][j];
+          float* sr = sb + (b * 128 + i) * V;
           if ((V & 3) == 0 && v0 + uc + CP <= V) {
-            if (CP == 4) *reinterpret_cast<float4*>(sb + (size_t)d * V + v0 + uc) = make_float4(st[b][i][0], st[b][i][1], st[b][i][2 % CP], st[b][i][3 % CP]);
-            else *reinterpret_cast<float2*>(sb + (size_t)d * V + v0 + uc) = make_float2(st[b][i][0], st[b][i][1]);
+            if (CP == 4) *reinterpret_cast<float4*>(sr) = make_float4(st[b][i][0], st[b][i][1], st[b][i][2 % CP], st[b][i][3 % CP]);
+            else *reinterpret_cast<float2*>(sr) = make_float2(st[b][i][0], st[b][i][1]);
           } else {
 #pragma unroll
             for (int j = 0; j < CP; ++j)
-              if (v0 + uc + j < V) sb[(size_t)d * V + v0 + uc + j] = st[b][i][j];
+              if (v0 + uc + j < V) sr[j] = st[b][i][j];
           }
         }
       }
@@ -846,7 +862,6 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DlArgs a, DlChun
       for (int x = 0; x < KSPLIT; ++x)
 #pragma unroll
         for (int j = 0; j < CP; ++j) u[j] -= part[(x * DL_C + ur) * SS + uc + j];
-      float* yg = ch.y + chunk(p) * DL_C * V + (size_t)ur * V + v0 + uc;
 #pragma unroll
       for (int j = 0; j < CP; ++j) {
         U[ur * SS + uc + j] = u[j];
@@ -859,7 +874,10 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DlArgs a, DlChun
       for (int i = 0; i < 4; ++i)
 #pragma unroll
         for (int j = 0; j < CP; ++j) st[b][i][j] *= ge[b][i];
-    if (p + 1 < np) load_small(p + 1);
+    yg += step_y;
+    gg += (size_t)H * D;
+    sb += step_s;
+    if (p + 1 < np) load_small(yg, gg);
     __syncthreads();
 #pragma unroll
     for (int b = 0; b < ND; ++b) {
@@ -894,7 +912,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DlArgs a, DlChun
 }
 
 static size_t dl_scan_smem(int D, int VS) {
-  const int SS = VS + 4, ksplit = DL_THREADS / (2 * VS);
+  const int SS = VS + 4, ksplit = DL_SCAN_THREADS / (2 * VS);
   return (size_t)(4 * DL_C * (D + 4) + D * SS + DL_C * SS + ksplit * DL_C * SS) * sizeof(float);
 }
 
@@ -913,7 +931,7 @@ __global__ void __launch_bounds__(DL_THREADS, 2) delta_out_kernel(DlArgs a, DlCh
   const int t0 = a.cu_seqlens[s] + p * DL_C, len = a.cu_seqlens[s + 1] - t0;
   if (len <= 0) return;
   const int L = min(DL_C, len);
-  const size_t ci = ((size_t)s * ch.P + p) * H + h;
+  const size_t ci = (size_t)(a.cu_seqlens[s] / DL_C + s + p) * H + h;
   const float *qg = ch.qg + ci * DL_C * D, *pg = ch.p + ci * DL_C * DL_C, *sb = ch.sb + ci * D * V, *ug = ch.y + ci * DL_C * V;
   const int warp = tid >> 5, lane = tid & 31;
   auto load_rows = [&](float* dst, const float* src, int rows) {        // rows of V columns
@@ -1139,7 +1157,7 @@ static int dl_chunks_launch(const DlArgs& a, const DlPrep& w, const DlChunks& ch
 #define DL_SCAN(VS, ND)                                                                                                       \
   do {                                                                                                                        \
     if (ss > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<VS, ND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ss); \
-    rc = sx_launch(delta_scan_kernel<VS, ND>, grid, dim3(DL_THREADS), ss, stream, a, ch);                                      \
+    rc = sx_launch(delta_scan_kernel<VS, ND>, grid, dim3(DL_SCAN_THREADS), ss, stream, a, ch);                                      \
   } while (0)
   if (slice == 32) { if (a.D <= 128) DL_SCAN(32, 1); else DL_SCAN(32, 2); }
   else { if (a.D <= 128) DL_SCAN(16, 1); else DL_SCAN(16, 2); }

@@ -206,61 +206,6 @@ __global__ void __launch_bounds__(256) side_gate_kernel(const float* __restrict_
   g[i] = from_f32<T>(id >= 0 && id < V ? y * to_f32(e[(size_t)id * n + c]) : 0.f);
 }
 
-// the same behind the gate's product, for few rows: g[t, c] = gelu_tanh(w[c] . x[t]) * e[ids[t], c].  A warp an output of a
-// token (its weights asked for before the wait, from L2 for all tokens but one)
-template <typename T>
-__global__ void __launch_bounds__(256) side_gate_rows_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ e,
-                                                             const int* __restrict__ ids, T* __restrict__ g, int K, int n, int V) {
-  constexpr int VE = 16 / sizeof(T), HELD = 16;      // 16-byte pieces a lane holds: K <= 32 * 16 * VE
-  const int c = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, t = blockIdx.y;
-  uint4 wv[HELD];
-  const int pieces = K / VE;
-#pragma unroll
-  for (int i = 0; i < HELD; ++i) {
-    const int at = lane + 32 * i;
-    if (c < n && at < pieces) wv[i] = reinterpret_cast<const uint4*>(w + (size_t)c * K)[at];
-  }
-  pdl_wait();
-  pdl_trigger();
-  if (c >= n) return;
-  const uint4* xr = reinterpret_cast<const uint4*>(x + (size_t)t * K);
-  float acc = 0.f;
-#pragma unroll
-  for (int i = 0; i < HELD; ++i) {
-    const int at = lane + 32 * i;
-    if (at < pieces) {
-      const uint4 xv = xr[at];
-      const T *xp = reinterpret_cast<const T*>(&xv), *wp = reinterpret_cast<const T*>(&wv[i]);
-#pragma unroll
-      for (int j = 0; j < VE; ++j) acc = fmaf(to_f32(xp[j]), to_f32(wp[j]), acc);
-    }
-  }
-  const float z = warp_sum(acc);
-  if (lane == 0) {
-    const int id = ids[t];
-    const float y = 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-    g[(size_t)t * n + c] = from_f32<T>(id >= 0 && id < V ? y * to_f32(e[(size_t)id * n + c]) : 0.f);
-  }
-}
-
-#define SIDE_ROWS_MAX 8
-extern "C" int sx_side_gate_rows_fit(int n_tokens, int K, int dt) {
-  const int ve = dt == SX_BF16 ? 8 : 4;
-  return n_tokens <= SIDE_ROWS_MAX && K % ve == 0 && K / ve <= 32 * 16 ? 1 : 0;
-}
-extern "C" int sx_side_gate_rows(const void* x, const void* w, const void* e, const int* ids, void* g, int n_tokens, int K, int n, int V,
-                                 int dt, cudaStream_t stream) {
-  if (n_tokens <= 0) return 0;
-  if (n <= 0 || V <= 0 || K <= 0 || !sx_side_gate_rows_fit(n_tokens, K, dt)) return SX_ERR_SIZE;
-  if (((uintptr_t)x | (uintptr_t)w) % 16) return SX_ERR_ALIGN;
-  const dim3 grid((n + 7) / 8, n_tokens);
-  if (dt == SX_F32)
-    return sx_launch(side_gate_rows_kernel<float>, grid, dim3(256), 0, stream, (const float*)x, (const float*)w, (const float*)e, ids, (float*)g, K, n, V);
-  if (dt == SX_BF16)
-    return sx_launch(side_gate_rows_kernel<bf16>, grid, dim3(256), 0, stream, (const bf16*)x, (const bf16*)w, (const bf16*)e, ids, (bf16*)g, K, n, V);
-  return SX_ERR_DTYPE;
-}
-
 extern "C" int sx_side_gate(const float* u, const void* e, const int* ids, void* g, int n_tokens, int n, int V, int dt, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (n <= 0 || V <= 0) return SX_ERR_SIZE;

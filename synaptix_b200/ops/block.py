@@ -93,23 +93,13 @@ def scale_rows(x: torch.Tensor, s: float) -> None:
     check(fn("parallel", "sx_scale_rows")(ptr(x), c_longlong(x.numel()), c_float(s), stream()), "scale_rows")
 
 
-def side_gate(x: torch.Tensor, w: torch.Tensor, table: torch.Tensor, token_ids: torch.Tensor) -> torch.Tensor:
-    """``gelu_tanh(x[t] @ w.T) * table[id_t]`` in ``table``'s dtype: ``x [T, K]``, ``w [n, K]``, ``table [vocab, n]``.  One
-    kernel for a few rows, else the product (32-bit results) and one kernel behind it."""
-    require_cuda(x, w, table, token_ids)
-    T, K = x.shape
-    n = w.shape[0]
-    if (w.shape[1] != K or table.shape[1] != n or w.dtype != x.dtype or table.dtype != x.dtype or token_ids.dtype != torch.int32
-            or token_ids.numel() != T):
+def side_gate(u: torch.Tensor, table: torch.Tensor, token_ids: torch.Tensor) -> torch.Tensor:
+    """``gelu_tanh(u[t]) * table[id_t]`` in ``table``'s dtype: ``u`` float32 ``[T, n]``, ``table [vocab, n]``."""
+    require_cuda(u, table, token_ids)
+    T, n = u.shape
+    if u.dtype != torch.float32 or table.shape[1] != n or token_ids.dtype != torch.int32 or token_ids.numel() != T:
         raise KernelError("side_gate: sizes or dtypes do not fit")
-    g = torch.empty((T, n), dtype=table.dtype, device=x.device)
-    dt = c_int(dt_code(table.dtype))
-    if fn("parallel", "sx_side_gate_rows_fit")(c_int(T), c_int(K), dt):
-        check(fn("parallel", "sx_side_gate_rows")(ptr(x), ptr(w), ptr(table), ptr(token_ids), ptr(g), c_int(T), c_int(K), c_int(n),
-                                                  c_int(table.shape[0]), dt, stream()), "side_gate_rows")
-        return g
-    from . import linear
-    u = linear(x, w, out_dtype=torch.float32)
-    check(fn("parallel", "sx_side_gate")(ptr(u), ptr(table), ptr(token_ids), ptr(g), c_int(T), c_int(n), c_int(table.shape[0]), dt,
-                                         stream()), "side_gate")
+    g = torch.empty((T, n), dtype=table.dtype, device=u.device)
+    check(fn("parallel", "sx_side_gate")(ptr(u), ptr(table), ptr(token_ids), ptr(g), c_int(T), c_int(n), c_int(table.shape[0]),
+                                         c_int(dt_code(table.dtype)), stream()), "side_gate")
     return g

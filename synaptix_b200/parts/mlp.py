@@ -48,7 +48,7 @@ class SwiGLU(FeedForward):
         z = self.gate_up.forward(x, epilogue="silu_mul")
         if defer_output:
             return self.down.deferred(z)
-        with ops.late_launch(ctx.branches):
+        with ops.late_launch(ctx is not None and ctx.branches):
             return self.down.forward(z)
 
 
@@ -157,7 +157,7 @@ class MixtureOfExperts(FeedForward):
                 z = ops.moe_gate_up(x, self.gate_up, plan, self.top)
         else:
             z = ops.moe_gate_up(x, self.gate_up, plan, self.top)
-        with ops.late_launch(ctx.branches):
+        with ops.late_launch(ctx is not None and ctx.branches):
             y = ops.moe_down(z, self.down, plan)
         if defer_combine:           # a block that norms this branch on its way into the stream forms the sum there
             return ops.WeightedRows(y, plan.place, weights, x.dtype)

@@ -47,5 +47,6 @@ class TokenSide(Part):
         """Adds ``terms`` (the layer's branches, as a ``ScaledSum`` holds them) into the stream ``h`` and returns this
         input's branch, to be normed and added by whoever adds it."""
         x = ops.add_scaled_rmsnorm(h, terms, [None], 0.0, ctx.runtime.dtype)[0]
-        g = ops.side_gate(x, self.gate.weight, self.table, ctx.token_ids)
+        u = self.gate.forward(x, out_dtype=torch.float32)
+        g = ops.side_gate(u, self.table, ctx.token_ids)
         return NormedDelta(self.proj.forward(g), self.norm)
