@@ -735,14 +735,14 @@ __global__ void __launch_bounds__(DL_THREADS, 3) delta_intra_kernel(DlArgs a, Dl
 static size_t dl_intra_smem(int D) { return (size_t)(3 * DL_C * (D + 4) + DL_C * DL_LD + DL_C) * sizeof(float); }
 
 
-// VS: columns of the state a block owns (16 or 32); ND: tiles of the state a thread owns (D <= 128 ND).
+// VS: columns of the state a block owns (8, 16 or 32); ND: tiles of the state a thread owns (D <= 128 ND).
 #define DL_SCAN_THREADS 256
 template <int VS, int ND>
 __global__ void __launch_bounds__(DL_SCAN_THREADS) delta_scan_kernel(DlArgs a, DlChunks ch) {
   extern __shared__ __align__(16) float sm[];
   constexpr int SS = VS + 4;
   constexpr int CG = VS / 4;                       // groups of four columns in the product with S
-  constexpr int KSPLIT = DL_SCAN_THREADS / (8 * CG);   // 8 or 4: parts of D in that product
+  constexpr int KSPLIT = DL_SCAN_THREADS / (8 * CG);   // 16, 8 or 4: parts of D in that product
   constexpr int CP = VS / 8;                       // columns a thread of u and of the state's tiles
   const int D = a.D, V = a.V, H = a.H, DS = D + 4;
   float* xs = sm;                                  // 2 * 32 * DS: X, two chunks
@@ -817,8 +817,9 @@ __global__ void __launch_bounds__(DL_SCAN_THREADS) delta_scan_kernel(DlArgs a, D
           for (int j = 0; j < CP; ++j) S[d * SS + uc + j] = st[b][i][j];
           float* sr = sb + (b * 128 + i) * V;
           if ((V & 3) == 0 && v0 + uc + CP <= V) {
-            if (CP == 4) *reinterpret_cast<float4*>(sr) = make_float4(st[b][i][0], st[b][i][1], st[b][i][2 % CP], st[b][i][3 % CP]);
-            else *reinterpret_cast<float2*>(sr) = make_float2(st[b][i][0], st[b][i][1]);
+            if (CP == 4) *reinterpret_cast<float4*>(sr) = make_float4(st[b][i][0], st[b][i][1 % CP], st[b][i][2 % CP], st[b][i][3 % CP]);
+            else if (CP == 2) *reinterpret_cast<float2*>(sr) = make_float2(st[b][i][0], st[b][i][1 % CP]);
+            else *sr = st[b][i][0];
           } else {
 #pragma unroll
             for (int j = 0; j < CP; ++j)
@@ -1027,7 +1028,7 @@ static size_t dl_out_smem(int D, int V) { return (size_t)(DL_C * (D + DL_C + 4) 
 extern "C" int sx_delta_chunk_tokens() { return DL_C; }
 extern "C" int sx_delta_chunks_fit(int D, int V) {
   return (D % 4 == 0 && D <= DL_THREADS && V <= 256 && dl_intra_smem(D) <= 220 * 1024 && dl_scan_smem(D, 32) <= 220 * 1024 &&
-          dl_scan_smem(D, 16) <= 220 * 1024 && dl_out_smem(D, V) <= 220 * 1024) ? 1 : 0;
+          dl_scan_smem(D, 16) <= 220 * 1024 && dl_scan_smem(D, 8) <= 220 * 1024 && dl_out_smem(D, V) <= 220 * 1024) ? 1 : 0;
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -1160,7 +1161,8 @@ static int dl_chunks_launch(const DlArgs& a, const DlPrep& w, const DlChunks& ch
     rc = sx_launch(delta_scan_kernel<VS, ND>, grid, dim3(DL_SCAN_THREADS), ss, stream, a, ch);                                      \
   } while (0)
   if (slice == 32) { if (a.D <= 128) DL_SCAN(32, 1); else DL_SCAN(32, 2); }
-  else { if (a.D <= 128) DL_SCAN(16, 1); else DL_SCAN(16, 2); }
+  else if (slice == 16) { if (a.D <= 128) DL_SCAN(16, 1); else DL_SCAN(16, 2); }
+  else { if (a.D <= 128) DL_SCAN(8, 1); else DL_SCAN(8, 2); }
 #undef DL_SCAN
   if (rc) return rc;
   const size_t so = dl_out_smem(a.D, a.V);
@@ -1176,7 +1178,7 @@ static int dl_chunks_launch(const DlArgs& a, const DlPrep& w, const DlChunks& ch
 extern "C" int sx_delta_chunks(DL_FORMALS, float* q, float* k, float* v, float* x, float* qg, float* kd, float* y, float* p,
                                float* ge, float* sb, int chunks, int slice, cudaStream_t stream) {
   if (n_tokens <= 0 || n_seqs <= 0) return 0;
-  if (dl_check(n_seqs, H, G, D, V, taps) || !sx_delta_chunks_fit(D, V) || (slice != 16 && slice != 32) || chunks <= 0) return SX_ERR_SIZE;
+  if (dl_check(n_seqs, H, G, D, V, taps) || !sx_delta_chunks_fit(D, V) || (slice != 8 && slice != 16 && slice != 32) || chunks <= 0) return SX_ERR_SIZE;
   if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)x | (uintptr_t)qg | (uintptr_t)kd | (uintptr_t)y | (uintptr_t)p | (uintptr_t)ge | (uintptr_t)sb) % 16)
     return SX_ERR_ALIGN;
   const DlArgs a = dl_args(DL_ACTUALS);

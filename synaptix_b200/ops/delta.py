@@ -87,9 +87,11 @@ def delta_rule(proj: torch.Tensor, col: int, b_col: int, heads: int, kv_heads: i
         x, qg, kd = (torch.empty((n, C_, dim), **f32) for _ in range(3))
         y, p, ge = torch.empty((n, C_, vdim), **f32), torch.empty((n, C_, C_), **f32), torch.empty((n, dim), **f32)
         sb = torch.empty((n, dim, vdim), **f32)
-        # narrow slices of the state where wide ones would leave SMs idle
+        # columns of the state a block of the scan owns: narrow slices where wide ones would leave SMs idle (every slice
+        # reads the chunks' keys again)
         sms = torch.cuda.get_device_properties(proj.device).multi_processor_count
-        slice_ = 32 if ctx.n_seqs * heads * ((vdim + 31) // 32) >= sms else 16
+        blocks = ctx.n_seqs * heads
+        slice_ = next((v for v in (32, 16) if blocks * ((vdim + v - 1) // v) >= 0.8 * sms), 8)
         # each of the three fills the SMs' shared memory: waiting blocks of the next would only take the running one's room
         # (16 heads of 128 x 128, 2,048 tokens: 447 us scheduled early, 365 late)
         with late_launch():

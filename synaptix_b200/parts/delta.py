@@ -7,9 +7,9 @@ Per head ``h`` (which reads query/key head ``h // (heads / kv_heads)``), with ``
     S <- diag(a) S,   u = b (v - S^T k),   S <- S + k u^T,   o = S^T q,
     out = Wo (o / rms(o) * gain * sigmoid(Wg2 (Wg1 x)))
 
-``conv`` is a short causal convolution over time per channel.  The state starts at zero, lives in 32-bit in the cache's
-per-sequence storage and goes on from step to step, beside the convolutions' last inputs (a ring of ``taps`` projected
-rows, the row of position ``p`` at ``p mod taps``).  Everything that enters the recurrence behind the projections is 32-bit.
+``conv`` is a short causal convolution over time per channel.  State of a sequence, in the cache's per-sequence storage: the
+float32 matrices ``S`` (zero in a fresh slot) and a ring of the last ``taps`` projected rows for the convolutions (the row
+of position ``p`` at ``p mod taps``).  Behind the projections everything on the way into ``S`` is 32-bit.
 """
 from __future__ import annotations
 

@@ -143,7 +143,9 @@ class DeltaCase:
 
 
 SHAPES = [(4, 2, 12, 20, 4), (2, 1, 64, 64, 3), (3, 3, 128, 128, 4), (4, 4, 64, 32, 2), (2, 2, 32, 256, 4), (6, 3, 6, 8, 5),
-          (2, 1, 256, 64, 1), (1, 1, 8, 1, 4), (4, 1, 20, 36, 3), (1, 1, 1, 4, 2), (2, 2, 100, 16, 6)]
+          (2, 1, 256, 64, 1), (1, 1, 8, 1, 4), (4, 1, 20, 36, 3), (1, 1, 1, 4, 2), (2, 2, 100, 16, 6),
+          # as many (sequence, head) pairs as give the scan wide and middle slices of the state, with one tile of it and two
+          (40, 40, 16, 32, 2), (20, 10, 16, 36, 3), (30, 30, 132, 16, 2), (15, 5, 136, 32, 4)]
 CUTS = [[200], [1] * 200, [2] * 100, [3, 1, 2, 64, 7, 1, 1, 150], [17, 15, 33, 1, 31, 32, 90], [100, 1, 1, 1, 1, 1, 100]]
 
 
@@ -154,7 +156,7 @@ def test_delta_rule_over_portions(heads, kv_heads, dim, vdim, taps, dtype):
     the low-rank products inside, portions shorter than the taps reach back), in batches of unequal sequences."""
     lengths, slots = [150, 9, 77, 1], [2, 0, 5, 3]
     case = DeltaCase(heads, kv_heads, dim, vdim, taps, lengths, heads * dim + taps, dtype)
-    for cuts in CUTS:
+    for cuts in (CUTS if heads < 10 else CUTS[:1] + CUTS[3:5]):
         for low_rank in ((False, True) if 1 in cuts else (False,)):
             for o, r in zip(case.run(slots, cuts, low_rank), case.refs):
                 near(o, r, dtype, f32=2e-4, bf16=3e-2)
