@@ -37,6 +37,7 @@ struct AtPrep {
   float eps;
   int write;                // 0: this layer reads a cache another layer wrote (the token's key and value are there)
   int n_pages;
+  int row;                  // elements between two tokens' projections ((nh + 2 nkv) HD, or nh HD: query heads alone)
 };
 
 template <int HD, bool PREP, bool EX = false>
@@ -84,8 +85,7 @@ __global__ void __launch_bounds__(AT_THREADS) attn_decode_kernel(
     // has ended.
     first_pages();
     constexpr int half = HD / 2;
-    const int heads = nh + 2 * nkv;
-    const bf16* tok = q + (size_t)seq * heads * HD;
+    const bf16* tok = q + (size_t)seq * prep.row;
     float cs[2] = {1.f, 1.f}, sn[2] = {0.f, 0.f};
     const int p = 2 * lane;                                   // this lane's pairs (p, p + half), (p + 1, p + 1 + half)
     if (prep.inv_freq && p < half) {
@@ -166,7 +166,7 @@ __global__ void __launch_bounds__(AT_THREADS) attn_decode_kernel(
   const float sl_m = (EX && (ex.cap_log2 > 0.f || ex.dist)) ? 1.f : scale_log2;
   const float* dist_lo = (EX && ex.dist) ? ex.dist + (size_t)(kvh * G + min(g, G - 1)) * ex.dist_n : nullptr;
   const float* dist_hi = (EX && ex.dist) ? ex.dist + (size_t)(kvh * G + min(g + 8, G - 1)) * ex.dist_n : nullptr;
-  if (EX && ex.sinks && warp == 0 && split == 0) {            // the sink counts once: in the first warp of the first split
+  if (ex.sinks && warp == 0 && split == 0) {            // the sink counts once: in the first warp of the first split
     if (g < G) { m[0] = ex.sinks[kvh * G + g] * 1.4426950408889634f / sl_m; l[0] = t == 0 ? 1.f : 0.f; }
     if (g + 8 < G) { m[1] = ex.sinks[kvh * G + g + 8] * 1.4426950408889634f / sl_m; l[1] = t == 0 ? 1.f : 0.f; }
   }
@@ -352,8 +352,8 @@ __global__ void __launch_bounds__(AT_THREADS, 3) attn_prefill_kernel(
     }
   }
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  if (EX && ex.sinks) {                                       // the sink: a term exp(sink) of the denominator without a key
-    const float s0 = ex.sinks[h] * 1.4426950408889634f / ((ex.cap_log2 > 0.f || ex.dist) ? 1.f : scale_log2);
+  if (ex.sinks) {                                             // the sink: a term exp(sink) of the denominator without a key
+    const float s0 = ex.sinks[h] * 1.4426950408889634f / ((EX && (ex.cap_log2 > 0.f || ex.dist)) ? 1.f : scale_log2);
     m[0] = m[1] = s0;
     l[0] = l[1] = t == 0 ? 1.f : 0.f;
   }
@@ -440,7 +440,7 @@ __global__ void __launch_bounds__(AT_THREADS, 3) attn_prefill_kernel(
 template <int HD, bool PREP>
 static int decode_launch(const bf16* q, bf16* k, bf16* v, bf16* out, float* part_o, float* part_ml,
                          const int* seq_lens, const int* bt, int maxp, int S, int nh, int nkv, float scale_log2,
-                         int window, int n_splits, int* counters, const AtPrep& prep, cudaStream_t stream) {
+                         int window, int n_splits, int* counters, const AtPrep& prep, const float* sinks, cudaStream_t stream) {
   using L = AtLayout<HD>;
   const size_t merge_bytes = (size_t)(4 * 16 * HD + 4 * 16 * 2) * sizeof(float);
   const size_t last_bytes = (size_t)(2 * 16 * n_splits + 16) * sizeof(float);
@@ -450,7 +450,7 @@ static int decode_launch(const bf16* q, bf16* k, bf16* v, bf16* out, float* part
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   dim3 grid(n_splits, nkv, S);
-  const AtExtra no_extra = {0.f, 0.f, nullptr, 0, 0, 1.f, nullptr, 0};
+  const AtExtra no_extra = {0.f, 0.f, sinks, 0, 0, 1.f, nullptr, 0};
   int rc = sx_launch(kern, grid, dim3(AT_THREADS), smem, stream, q, k, v, out, part_o, part_ml, seq_lens, bt, maxp, nh, nkv,
                      scale_log2, window, n_splits, counters, prep, no_extra);
   if (rc || n_splits == 1 || counters) return rc;
@@ -463,7 +463,7 @@ static int decode_launch(const bf16* q, bf16* k, bf16* v, bf16* out, float* part
 static int attn_decode_any(const void* q, const void* k_pages, const void* v_pages, void* out, float* part_o,
                            float* part_ml, const int* seq_lens, const int* block_table, int maxp, int S, int nh,
                            int nkv, int hd, float scale, int window, int n_splits, int* counters, const AtPrep* prep,
-                           cudaStream_t stream) {
+                           const float* sinks, cudaStream_t stream) {
   if (S <= 0) return 0;
   if (nkv <= 0 || nh % nkv != 0 || nh / nkv > 16 || n_splits < 1 || nkv > 65535 || S > 65535) return SX_ERR_SIZE;
   // the merge keeps two floats a split in shared memory: refused before anything is launched
@@ -472,12 +472,12 @@ static int attn_decode_any(const void* q, const void* k_pages, const void* v_pag
   const float sl = scale * 1.4426950408889634f;
   const bf16* qb = (const bf16*)q;
   bf16 *kb = (bf16*)const_cast<void*>(k_pages), *vb = (bf16*)const_cast<void*>(v_pages), *ob = (bf16*)out;
-  const AtPrep none = {nullptr, nullptr, nullptr, 0.f, 0, 0};
+  const AtPrep none = {nullptr, nullptr, nullptr, 0.f, 0, 0, 0};
 #define AT_GO(HD)                                                                                                            \
   return prep ? decode_launch<HD, true>(qb, kb, vb, ob, part_o, part_ml, seq_lens, block_table, maxp, S, nh, nkv, sl, window, \
-                                        n_splits, counters, *prep, stream)                                                     \
+                                        n_splits, counters, *prep, sinks, stream)                                                     \
               : decode_launch<HD, false>(qb, kb, vb, ob, part_o, part_ml, seq_lens, block_table, maxp, S, nh, nkv, sl, window, \
-                                         n_splits, counters, none, stream)
+                                         n_splits, counters, none, sinks, stream)
   if (hd == 128) AT_GO(128);
   if (hd == 64) AT_GO(64);
   if (hd == 32) AT_GO(32);
@@ -485,12 +485,13 @@ static int attn_decode_any(const void* q, const void* k_pages, const void* v_pag
   return SX_ERR_SIZE;
 }
 
-// the splits are merged by a second kernel
+// the splits are merged by a second kernel; sinks [nh] (null: none): exp(sink) joins the denominator of the head's softmax
 extern "C" int sx_attn_decode(const void* q, const void* k_pages, const void* v_pages, void* out, float* part_o,
                               float* part_ml, const int* seq_lens, const int* block_table, int maxp, int S, int nh,
-                              int nkv, int hd, float scale, int window, int n_splits, cudaStream_t stream) {
+                              int nkv, int hd, float scale, int window, int n_splits, const float* sinks,
+                              cudaStream_t stream) {
   return attn_decode_any(q, k_pages, v_pages, out, part_o, part_ml, seq_lens, block_table, maxp, S, nh, nkv, hd, scale,
-                         window, n_splits, nullptr, nullptr, stream);
+                         window, n_splits, nullptr, nullptr, sinks, stream);
 }
 
 // The same for a step's raw fused projection qkv [S, (nh + 2 nkv) hd]: per-head RMSNorm of q and k (gains wq, wk in
@@ -499,12 +500,14 @@ extern "C" int sx_attn_decode(const void* q, const void* k_pages, const void* v_
 extern "C" int sx_attn_decode_prep(const void* qkv, void* k_pages, void* v_pages, void* out, float* part_o, float* part_ml,
                                    const float* wq, const float* wk, const float* inv_freq, float eps, int write,
                                    long long n_pages, const int* seq_lens, const int* block_table, int maxp, int S, int nh,
-                                   int nkv, int hd, float scale, int window, int n_splits, cudaStream_t stream) {
+                                   int nkv, int hd, float scale, int window, int n_splits, const float* sinks, int row,
+                                   cudaStream_t stream) {
   if (((uintptr_t)qkv & 15) || ((uintptr_t)k_pages & 15) || ((uintptr_t)v_pages & 15)) return SX_ERR_ALIGN;
   if (n_pages <= 0 || n_pages > 0x7fffffffLL) return SX_ERR_SIZE;
-  const AtPrep prep = {wq, wk, inv_freq, eps, write, (int)n_pages};
+  if (row != (nh + 2 * nkv) * hd && !(row == nh * hd && !write)) return SX_ERR_SIZE;
+  const AtPrep prep = {wq, wk, inv_freq, eps, write, (int)n_pages, row};
   return attn_decode_any(qkv, k_pages, v_pages, out, part_o, part_ml, seq_lens, block_table, maxp, S, nh, nkv, hd, scale,
-                         window, n_splits, nullptr, &prep, stream);
+                         window, n_splits, nullptr, &prep, sinks, stream);
 }
 
 // the splits are merged inside the kernel by whichever block of a (sequence, kv head) finishes last;
@@ -514,7 +517,7 @@ extern "C" int sx_attn_decode_fused(const void* q, const void* k_pages, const vo
                                     int maxp, int S, int nh, int nkv, int hd, float scale, int window, int n_splits,
                                     cudaStream_t stream) {
   return attn_decode_any(q, k_pages, v_pages, out, part_o, part_ml, seq_lens, block_table, maxp, S, nh, nkv, hd, scale,
-                         window, n_splits, counters, nullptr, stream);
+                         window, n_splits, counters, nullptr, nullptr, stream);
 }
 
 // ---------------------------------------------------------------------------------------
@@ -572,19 +575,19 @@ extern "C" int sx_attn_decode_noalloc(const void* q, const void* k_pages, const 
     part_ml = base + slots * hd;            // [slots][2]; slots * hd * 4 bytes keeps it 8-byte aligned
   }
   return sx_attn_decode(q, k_pages, v_pages, out, part_o, part_ml, seq_lens, block_table, maxp, S, nh, nkv, hd, scale,
-                        window, n_splits, stream);
+                        window, n_splits, nullptr, stream);
 }
 
 template <int HD>
 static int prefill_launch(const bf16* q, const bf16* k, const bf16* v, bf16* out, const int* tile_seq, const int* tile_q0,
                           int n_tiles, const int* cu, const int* past, const int* lens, const int* bt, int maxp, int nh,
-                          int nkv, float scale_log2, int window, cudaStream_t stream) {
+                          int nkv, float scale_log2, int window, const float* sinks, cudaStream_t stream) {
   using L = AtLayout<HD, AT_STAGES_PREFILL>;
   auto kern = attn_prefill_kernel<HD>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)L::SMEM);
   if (e != cudaSuccess) return (int)e;
   dim3 grid(n_tiles, nh);
-  const AtExtra no_extra = {0.f, 0.f, nullptr, 0, 0, 1.f, nullptr, 0};
+  const AtExtra no_extra = {0.f, 0.f, sinks, 0, 0, 1.f, nullptr, 0};
   return sx_launch(kern, grid, dim3(AT_THREADS), L::SMEM, stream, q, k, v, out, tile_seq, tile_q0, cu, past, lens, bt, maxp, nh,
                    nkv, scale_log2, window, no_extra);
 }
@@ -645,7 +648,7 @@ static int decode_ex_launch(const bf16* q, bf16* k, bf16* v, bf16* out, const in
   auto kern = attn_decode_kernel<HD, false, true>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
-  const AtPrep none = {nullptr, nullptr, nullptr, 0.f, 0, 0};
+  const AtPrep none = {nullptr, nullptr, nullptr, 0.f, 0, 0, 0};
   return sx_launch(kern, dim3(1, nkv, S), dim3(AT_THREADS), smem, stream, q, k, v, out, (float*)nullptr, (float*)nullptr, seq_lens,
                    bt, maxp, nh, nkv, scale_log2, window, 1, (int*)nullptr, none, ex);
 }
@@ -671,13 +674,13 @@ extern "C" int sx_attn_decode_ex(const void* q, const void* k_pages, const void*
 extern "C" int sx_attn_prefill(const void* q, const void* k_pages, const void* v_pages, void* out,
                                const int* tile_seq, const int* tile_q0, int n_tiles, const int* cu_seqlens,
                                const int* seq_past, const int* seq_lens, const int* block_table, int maxp, int nh,
-                               int nkv, int hd, float scale, int window, cudaStream_t stream) {
+                               int nkv, int hd, float scale, int window, const float* sinks, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (nkv <= 0 || nh % nkv != 0 || nh > 65535) return SX_ERR_SIZE;
   const float sl = scale * 1.4426950408889634f;
   const bf16 *qb = (const bf16*)q, *kb = (const bf16*)k_pages, *vb = (const bf16*)v_pages;
-  if (hd == 128) return prefill_launch<128>(qb, kb, vb, (bf16*)out, tile_seq, tile_q0, n_tiles, cu_seqlens, seq_past, seq_lens, block_table, maxp, nh, nkv, sl, window, stream);
-  if (hd == 64) return prefill_launch<64>(qb, kb, vb, (bf16*)out, tile_seq, tile_q0, n_tiles, cu_seqlens, seq_past, seq_lens, block_table, maxp, nh, nkv, sl, window, stream);
-  if (hd == 32) return prefill_launch<32>(qb, kb, vb, (bf16*)out, tile_seq, tile_q0, n_tiles, cu_seqlens, seq_past, seq_lens, block_table, maxp, nh, nkv, sl, window, stream);
+  if (hd == 128) return prefill_launch<128>(qb, kb, vb, (bf16*)out, tile_seq, tile_q0, n_tiles, cu_seqlens, seq_past, seq_lens, block_table, maxp, nh, nkv, sl, window, sinks, stream);
+  if (hd == 64) return prefill_launch<64>(qb, kb, vb, (bf16*)out, tile_seq, tile_q0, n_tiles, cu_seqlens, seq_past, seq_lens, block_table, maxp, nh, nkv, sl, window, sinks, stream);
+  if (hd == 32) return prefill_launch<32>(qb, kb, vb, (bf16*)out, tile_seq, tile_q0, n_tiles, cu_seqlens, seq_past, seq_lens, block_table, maxp, nh, nkv, sl, window, sinks, stream);
   return SX_ERR_SIZE;
 }

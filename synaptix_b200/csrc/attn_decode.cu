@@ -62,6 +62,7 @@ struct AdPrep {
   float eps;
   int write;                // 0: this layer reads a cache another layer wrote (the token's key and value are there)
   int n_pages;
+  int row;                  // elements between two tokens' projections ((nh + 2 nkv) HD, or nh HD: query heads alone)
 };
 
 __device__ __forceinline__ uint32_t ad_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -232,7 +233,7 @@ __global__ void __launch_bounds__(AD_THREADS, 2) attn_decode_tma_kernel(
     const bf16* __restrict__ q, bf16* __restrict__ k_pages, bf16* __restrict__ v_pages, bf16* __restrict__ out,
     float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ seq_lens,
     const int* __restrict__ block_table, int maxp, int nh, int nkv, float scale_log2, int window, int n_splits,
-    const AdPrep prep, int* __restrict__ status) {
+    const AdPrep prep, const float* __restrict__ sinks, int* __restrict__ status) {
   using L = AdLayout<HD>;
   extern __shared__ unsigned char smem_raw[];
   __shared__ __align__(16) bf16 q_s[PREP ? 16 * HD : 8];       // the group's prepared query heads
@@ -308,8 +309,7 @@ __global__ void __launch_bounds__(AD_THREADS, 2) attn_decode_tma_kernel(
   // -------------------------------------------------------------------- compute warps
   if (PREP) {
     constexpr int half = HD / 2;
-    const int heads = nh + 2 * nkv;
-    const bf16* tok = q + (size_t)seq * heads * HD;
+    const bf16* tok = q + (size_t)seq * prep.row;
     float cs[2] = {1.f, 1.f}, sn[2] = {0.f, 0.f};
     const int p = 2 * lane;                                   // this lane's pairs (p, p + half), (p + 1, p + 1 + half)
     if (prep.inv_freq && p < half) {
@@ -386,6 +386,11 @@ __global__ void __launch_bounds__(AD_THREADS, 2) attn_decode_tma_kernel(
     }
   }
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  if (sinks != nullptr && warp == 0 && split == 0) {          // the sink counts once: in the first warp of the first split
+    const float inv = 1.4426950408889634f / scale_log2;
+    if (g < G) { m[0] = sinks[kvh * G + g] * inv; l[0] = t == 0 ? 1.f : 0.f; }
+    if (g + 8 < G) { m[1] = sinks[kvh * G + g + 8] * inv; l[1] = t == 0 ? 1.f : 0.f; }
+  }
   float o[HD / 8][4];
 #pragma unroll
   for (int n = 0; n < HD / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
@@ -545,7 +550,7 @@ static int* ad_status_word() {
 template <int HD, bool PREP>
 static int ad_launch(const CUtensorMap& mk, const CUtensorMap& mv, const bf16* q, bf16* k, bf16* v, bf16* out, float* part_o,
                      float* part_ml, const int* seq_lens, const int* bt, int maxp, int S, int nh, int nkv, float scale_log2,
-                     int window, int n_splits, const AdPrep& prep, int* status, cudaStream_t stream) {
+                     int window, int n_splits, const AdPrep& prep, const float* sinks, int* status, cudaStream_t stream) {
   using L = AdLayout<HD>;
   static_assert(AD_STAGES == AD_COMPUTE_WARPS, "a stage has one consumer");
   static_assert(AD_STAGES * L::STAGE >= (AD_COMPUTE_WARPS + 1) * (16 * HD + 16 * 2) * (int)sizeof(float),
@@ -556,13 +561,13 @@ static int ad_launch(const CUtensorMap& mk, const CUtensorMap& mv, const bf16* q
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)L::SMEM);
     if (e != cudaSuccess) return (int)e;
     return sx_launch_cluster(kern, dim3(n_splits, nkv, S), dim3(AD_THREADS), (size_t)L::SMEM, stream, n_splits, mk, mv, q, k,
-                             v, out, part_o, part_ml, seq_lens, bt, maxp, nh, nkv, scale_log2, window, n_splits, prep, status);
+                             v, out, part_o, part_ml, seq_lens, bt, maxp, nh, nkv, scale_log2, window, n_splits, prep, sinks, status);
   }
   auto kern = attn_decode_tma_kernel<HD, PREP, false>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)L::SMEM);
   if (e != cudaSuccess) return (int)e;
   int rc = sx_launch(kern, dim3(n_splits, nkv, S), dim3(AD_THREADS), (size_t)L::SMEM, stream, mk, mv, q, k, v, out, part_o,
-                     part_ml, seq_lens, bt, maxp, nh, nkv, scale_log2, window, n_splits, prep, status);
+                     part_ml, seq_lens, bt, maxp, nh, nkv, scale_log2, window, n_splits, prep, sinks, status);
   if (rc || n_splits == 1) return rc;
   return sx_launch(attn_merge_kernel<HD>, dim3(S * nh), dim3(HD), 2 * n_splits * sizeof(float), stream,
                    (const float*)part_o, (const float*)part_ml, out, n_splits);
@@ -572,6 +577,8 @@ static int ad_launch(const CUtensorMap& mk, const CUtensorMap& mv, const bf16* q
 // step's fused projection [S, (nh + 2 nkv) hd]: per-head RMSNorm of q and k (gains wq, wk in float32, or null),
 // rotate-half rotation of the whole head by seq_lens[s] - 1 (inv_freq [hd / 2], or null), and (write != 0) the new
 // key and value into the cache happen inside the kernel.  k_pages / v_pages [n_pages, nkv, 64, hd]; out [S, nh * hd];
+// `row`: elements between two tokens' projections; with write == 0 that may be nh * hd (query heads alone).  `sinks` [nh]
+// (null: none): exp(sink) joins the denominator of the head's softmax, once, without a key and unscaled.
 // part_o f32 [S * nh * n_splits * hd] and part_ml f32 [S * nh * n_splits * 2] are scratch (unused with one split).
 // Without scratch (both null) and 2, 4, 8 or 16 splits, the splits of a (sequence, kv head) run as a thread-block
 // cluster and merge through one another's shared memory; other split counts need the scratch.  Head size 64 or 128.
@@ -579,7 +586,7 @@ extern "C" int sx_attn_decode_tma(const void* q, void* k_pages, void* v_pages, v
                                   int prep_on, const float* wq, const float* wk, const float* inv_freq, float eps,
                                   int write, long long n_pages, const int* seq_lens, const int* block_table, int maxp,
                                   int S, int nh, int nkv, int hd, float scale, int window, int n_splits,
-                                  cudaStream_t stream) {
+                                  const float* sinks, int row, cudaStream_t stream) {
   if (S <= 0) return 0;
   if (nkv <= 0 || nh % nkv != 0 || nh / nkv > 16 || n_splits < 1 || nkv > 65535 || S > 65535) return SX_ERR_SIZE;
   if (hd != 64 && hd != 128) return SX_ERR_SIZE;
@@ -595,14 +602,15 @@ extern "C" int sx_attn_decode_tma(const void* q, void* k_pages, void* v_pages, v
   if (rc) return rc;
   if ((rc = ad_map_pages(&mv, v_pages, n_pages, nkv, hd))) return rc;
   const float sl = scale * 1.4426950408889634f;
-  const AdPrep prep = {wq, wk, inv_freq, eps, write, (int)n_pages};
+  if (prep_on && row != (nh + 2 * nkv) * hd && !(row == nh * hd && !write)) return SX_ERR_SIZE;
+  const AdPrep prep = {wq, wk, inv_freq, eps, write, (int)n_pages, row};
   const bf16* qb = (const bf16*)q;
   bf16 *kb = (bf16*)k_pages, *vb = (bf16*)v_pages, *ob = (bf16*)out;
 #define AD_GO(HD)                                                                                                          \
   return prep_on ? ad_launch<HD, true>(mk, mv, qb, kb, vb, ob, part_o, part_ml, seq_lens, block_table, maxp, S, nh, nkv, sl, \
-                                       window, n_splits, prep, status, stream)                                              \
+                                       window, n_splits, prep, sinks, status, stream)                                              \
                  : ad_launch<HD, false>(mk, mv, qb, kb, vb, ob, part_o, part_ml, seq_lens, block_table, maxp, S, nh, nkv, sl, \
-                                        window, n_splits, prep, status, stream)
+                                        window, n_splits, prep, sinks, status, stream)
   if (hd == 128) AD_GO(128);
   AD_GO(64);
 #undef AD_GO

@@ -26,6 +26,9 @@
 // Rows of V at or beyond the sequence's length are zeroed in shared memory before P V (their P is
 // zero, but 0 * NaN is NaN), scores against such keys are replaced before they are used.
 //
+// `sinks` (null: none): a number per query head whose exponential joins the softmax's denominator (no key, no value, not
+// scaled): the row's reference point starts at the sink and its sum at 1.
+//
 // Every wait on an mbarrier is bounded; a wait that runs out sets the status word
 // (sx_attn_tc_status) and the block still frees its tensor memory.
 //
@@ -187,7 +190,7 @@ __global__ void __launch_bounds__(FT_THREADS, 1) attn_tc_prefill_kernel(
     const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, const int* __restrict__ tile_seq,
     const int* __restrict__ tile_q0, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_past,
     const int* __restrict__ seq_lens, const int* __restrict__ block_table, int maxp, int nh, int nkv,
-    float scale_log2, int window, int* __restrict__ status) {
+    float scale_log2, int window, const float* __restrict__ sinks, int* __restrict__ status) {
   extern __shared__ unsigned char ft_smem_raw[];
   unsigned char* tiles = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(ft_smem_raw) + 1023) & ~(uintptr_t)1023);
   unsigned char* kv_s = tiles;                                   // [FT_KV_STAGES][K tile, V tile]
@@ -329,6 +332,10 @@ __global__ void __launch_bounds__(FT_THREADS, 1) attn_tc_prefill_kernel(
     const uint32_t t_row = tmem_base + ((uint32_t)((warp & 3) * 32) << 16);
     const int pos = r < rows ? past + q0 + r : -1;
     float m = -INFINITY, l = 0.f;                                 // l: this thread's columns only
+    if (sinks != nullptr) {                // a sink: a term exp(sink) of the denominator without a key, counted by one half
+      m = sinks[h] * 1.4426950408889634f / scale_log2;
+      l = hf == 0 ? 1.f : 0.f;
+    }
     bool ok = true;
     // this thread's half row of Q (64 values = one swizzled chunk row) from shared into tensor memory
     if (!ft_mbar_wait(bar(FT_B_QFULL), 0)) { sx_set_status(status, 6); ok = false; }
@@ -523,7 +530,8 @@ static int* ft_status_word() {
 extern "C" int sx_attn_prefill_tc(const void* q, const void* k_pages, const void* v_pages, void* out, long long T,
                                   long long n_pages, const int* tile_seq, const int* tile_q0, int n_tiles,
                                   const int* cu_seqlens, const int* seq_past, const int* seq_lens, const int* block_table,
-                                  int maxp, int nh, int nkv, int hd, float scale, int window, cudaStream_t stream) {
+                                  int maxp, int nh, int nkv, int hd, float scale, int window, const float* sinks,
+                                  cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (hd != FT_HD || nkv <= 0 || nh % nkv != 0 || n_tiles > 65535 || T <= 0 || n_pages <= 0) return SX_ERR_SIZE;
   if (((uintptr_t)q & 15) || ((uintptr_t)k_pages & 15) || ((uintptr_t)v_pages & 15) || ((uintptr_t)out & 15)) return SX_ERR_ALIGN;
@@ -539,7 +547,7 @@ extern "C" int sx_attn_prefill_tc(const void* q, const void* k_pages, const void
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   return sx_launch(kern, dim3(nh, n_tiles), dim3(FT_THREADS), smem, stream, mq, mk, mv, (bf16*)out, tile_seq, tile_q0,
-                   cu_seqlens, seq_past, seq_lens, block_table, maxp, nh, nkv, scale * 1.4426950408889634f, window, status);
+                   cu_seqlens, seq_past, seq_lens, block_table, maxp, nh, nkv, scale * 1.4426950408889634f, window, sinks, status);
 }
 
 // 0, or which bounded wait ran out (1 producer, 2-5 MMA issuer, 6-9 softmax)

@@ -44,6 +44,7 @@ LIBRARIES: Dict[str, tuple] = {
     "normed": ("normed.cu", []),
     "convqk": ("convqk.cu", []),
     "layernorm": ("layernorm.cu", []),
+    "dyntanh": ("dyntanh.cu", []),
     "attn_scored": ("attn_scored.cu", []),
     "mlstm": ("mlstm.cu", []),
     "delta": ("delta.cu", []),

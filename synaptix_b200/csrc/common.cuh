@@ -199,6 +199,11 @@ __device__ __forceinline__ float gate_mul(float g, float u, const GateAct a) {
   }
   return g / (1.f + __expf(-g)) * u;
 }
+// cap * tanh(z / cap); cap <= 0: z as it is
+__device__ __forceinline__ float soft_limit(float z, float cap) { return cap > 0.f ? cap * tanhf(z / cap) : z; }
+// The norm without statistics of a row: tanh(alpha v) * w + b, every element on its own.  Because it needs nothing of the
+// row's other elements, a product that adds itself into the residual stream finishes this norm in its epilogue.
+__device__ __forceinline__ float dyn_tanh(float v, float alpha, float w, float b) { return fmaf(tanhf(alpha * v), w, b); }
 static GateAct g_sx_gate = {0.f, 0.f, SX_GATE_SIGMOID};
 extern "C" void sx_set_gate_act(float alpha, float limit, int form) { g_sx_gate.alpha = alpha; g_sx_gate.limit = limit; g_sx_gate.form = form; }
 

@@ -49,7 +49,9 @@ __device__ __forceinline__ uint4 ld_stream16(const void* p) {
   return v;
 }
 
-enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_SILU_MUL = 2, EPI_RESID = 3 };
+//   A bias per output (SkNorm::bias) joins the results in every epilogue.  EPI_RESID_TANH is EPI_RESID with the norm
+//   without statistics behind the sum (dyn_tanh): the kernel writes the finished rows, and nothing is left to the consumer.
+enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_SILU_MUL = 2, EPI_RESID = 3, EPI_RESID_TANH = 4 };
 
 struct SkNorm {
   // consumer side: the rows of x lack the factor rsqrt(sum_i ssq_in[b * n_in + i] / K + eps_in); null: they do not
@@ -60,6 +62,10 @@ struct SkNorm {
   float* h_io;
   const float* gain_next;
   float* ssq_out;
+  const float* bias;      // [N] or null: added to the results (a stacked [gate; up] matrix: gate biases, then up biases)
+  float cap;              // EPI_F32: soft_limit of the results (0: none)
+  float alpha;            // EPI_RESID_TANH: out = bf16(tanh(alpha h) * gain_next + shift)
+  const float* shift;
 };
 
 // NT: activation rows in tiles of 8 (M <= 8 NT);  KS: warps that split K;  RT = SK_WARPS / KS row tiles per block
@@ -129,10 +135,19 @@ __global__ void __launch_bounds__(KS > SK_WARPS ? KS * 32 : SK_THREADS) skinny_g
     }
   }
   // the next norm's gains of this warp's columns (EPI_RESID) are weights as well
-  float gnext[2] = {0.f, 0.f};
-  if (EPI == EPI_RESID && tile_ok) {
+  constexpr bool RESID = EPI == EPI_RESID || EPI == EPI_RESID_TANH;
+  float gnext[2] = {0.f, 0.f}, shift[2] = {0.f, 0.f}, bias[2] = {0.f, 0.f};
+  if (RESID && tile_ok) {
     gnext[0] = __ldg(nrm.gain_next + row_lo);
     gnext[1] = __ldg(nrm.gain_next + row_hi);
+    if (EPI == EPI_RESID_TANH) {
+      shift[0] = __ldg(nrm.shift + row_lo);
+      shift[1] = __ldg(nrm.shift + row_hi);
+    }
+  }
+  if (nrm.bias && tile_ok) {
+    bias[0] = __ldg(nrm.bias + row_lo);
+    bias[1] = __ldg(nrm.bias + row_hi);
   }
   pdl_wait();          // the weights depend on no earlier kernel; everything below may
   pdl_trigger();
@@ -288,8 +303,8 @@ __global__ void __launch_bounds__(KS > SK_WARPS ? KS * 32 : SK_THREADS) skinny_g
   }
 
   // EPI_RESID: the residual stream's values of this warp's results, asked for before the add-up hides the trip
-  float hv[EPI == EPI_RESID ? NT : 1][4];
-  if (EPI == EPI_RESID && ks == 0 && tile_ok) {
+  float hv[RESID ? NT : 1][4];
+  if (RESID && ks == 0 && tile_ok) {
     const int n0 = tile * 16 + g, n1 = n0 + 8;
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt)
@@ -332,7 +347,32 @@ __global__ void __launch_bounds__(KS > SK_WARPS ? KS * 32 : SK_THREADS) skinny_g
         acc[nt][2 + j] *= f;
       }
   }
-  if (EPI == EPI_RESID) {
+  if (nrm.bias) {
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int j = 0; j < 2; ++j) { acc[nt][j] += bias[0]; acc[nt][2 + j] += bias[1]; }
+  }
+  if (EPI == EPI_RESID_TANH) {
+    const int n0 = tile * 16 + g, n1 = n0 + 8;
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const int b = nt * 8 + t * 2 + j;
+        if (b >= M) continue;
+        if (n0 < N) {
+          const float v = hv[nt][j] + acc[nt][j];
+          nrm.h_io[(size_t)b * N + n0] = v;
+          reinterpret_cast<bf16*>(out)[(size_t)b * N + n0] = __float2bfloat16_rn(dyn_tanh(v, nrm.alpha, gnext[0], shift[0]));
+        }
+        if (n1 < N) {
+          const float v = hv[nt][2 + j] + acc[nt][2 + j];
+          nrm.h_io[(size_t)b * N + n1] = v;
+          reinterpret_cast<bf16*>(out)[(size_t)b * N + n1] = __float2bfloat16_rn(dyn_tanh(v, nrm.alpha, gnext[1], shift[1]));
+        }
+      }
+  } else if (EPI == EPI_RESID) {
     const int n0 = tile * 16 + g, n1 = n0 + 8;
     const int tiles = (N + 15) >> 4;
 #pragma unroll
@@ -378,8 +418,8 @@ __global__ void __launch_bounds__(KS > SK_WARPS ? KS * 32 : SK_THREADS) skinny_g
       } else {
         const int n0 = tile * 16 + g, n1 = n0 + 8;
         if (EPI == EPI_F32) {
-          if (n0 < N) reinterpret_cast<float*>(out)[(size_t)b * N + n0] = acc[nt][j];
-          if (n1 < N) reinterpret_cast<float*>(out)[(size_t)b * N + n1] = acc[nt][2 + j];
+          if (n0 < N) reinterpret_cast<float*>(out)[(size_t)b * N + n0] = soft_limit(acc[nt][j], nrm.cap);
+          if (n1 < N) reinterpret_cast<float*>(out)[(size_t)b * N + n1] = soft_limit(acc[nt][2 + j], nrm.cap);
         } else {
           if (n0 < N) reinterpret_cast<bf16*>(out)[(size_t)b * N + n0] = __float2bfloat16_rn(acc[nt][j]);
           if (n1 < N) reinterpret_cast<bf16*>(out)[(size_t)b * N + n1] = __float2bfloat16_rn(acc[nt][2 + j]);
@@ -431,10 +471,11 @@ static int skinny_pick_nt(int ks, const bf16* x, const bf16* W, void* out, int M
 // x [M, K] bf16 (or, with h_in, computed as rmsnorm(h_in + delta) * gain), W [N, K] bf16.
 // epi 0: out bf16 [M, N];  1: out f32 [M, N];  2: W is [gate; up] stacked, out bf16 [M, N/2] = silu(gate) * up.
 // ks: warps that split K (8, or 16 with blocks of 16 warps).  Requires K % 32 == 0, 16-byte aligned x and W, M <= 16
-// (M <= XS_ROWS = 2 with the norm prologue).
+// (M <= XS_ROWS = 2 with the norm prologue).  bias [N] (or null) is added to the product; epi 1 then limits the sum
+// softly at cap (0: not at all).
 extern "C" int sx_skinny_gemm(const void* x, const void* W, void* out, int M, int N, int K, int epi, int ks,
                               const float* h_in, const void* delta, float* h_out, const float* gain, float eps,
-                              cudaStream_t stream) {
+                              const float* bias, float cap, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || (K & 31) || M > 16) return SX_ERR_SIZE;
   if (epi == EPI_SILU_MUL && (N & 1)) return SX_ERR_SIZE;
@@ -442,7 +483,7 @@ extern "C" int sx_skinny_gemm(const void* x, const void* W, void* out, int M, in
   const bf16* xb = (const bf16*)x;
   const bf16* wb = (const bf16*)W;
   const bf16* db = (const bf16*)delta;
-  const SkNorm none = {nullptr, 0, 0.f, nullptr, nullptr, nullptr};
+  const SkNorm none = {nullptr, 0, 0.f, nullptr, nullptr, nullptr, bias, cap, 0.f, nullptr};
   if (h_in) {
     if (M > XS_ROWS || K > 4096 || (K & 3)) return SX_ERR_SIZE;   // the prologue holds a row in registers
     switch (epi) {
@@ -475,7 +516,7 @@ extern "C" int sx_skinny_gemm_norm(const void* x, const void* W, void* out, int 
   if (((uintptr_t)W & 15) || ((uintptr_t)x & 15)) return SX_ERR_ALIGN;
   const bf16* xb = (const bf16*)x;
   const bf16* wb = (const bf16*)W;
-  const SkNorm nrm = {ssq_in, n_in, eps_in, h_io, gain_next, ssq_out};
+  const SkNorm nrm = {ssq_in, n_in, eps_in, h_io, gain_next, ssq_out, nullptr, 0.f, 0.f, nullptr};
   switch (epi) {
     case EPI_BF16: return skinny_pick_nt<EPI_BF16, false>(ks, xb, wb, out, M, N, K, nullptr, nullptr, nullptr, nullptr, 0.f, nrm, stream);
     case EPI_F32: return skinny_pick_nt<EPI_F32, false>(ks, xb, wb, out, M, N, K, nullptr, nullptr, nullptr, nullptr, 0.f, nrm, stream);
@@ -483,4 +524,16 @@ extern "C" int sx_skinny_gemm_norm(const void* x, const void* W, void* out, int 
     case EPI_RESID: return skinny_pick_nt<EPI_RESID, false>(ks, xb, wb, out, M, N, K, nullptr, nullptr, nullptr, nullptr, 0.f, nrm, stream);
     default: return SX_ERR_DTYPE;
   }
+}
+
+// h_io f32 [M, N] += x W^T + bias in place (bias may be null), out bf16 [M, N] = tanh(alpha h_io) * gain + shift.
+extern "C" int sx_skinny_gemm_resid_tanh(const void* x, const void* W, void* out, int M, int N, int K, int ks, float* h_io,
+                                         const float* bias, float alpha, const float* gain, const float* shift,
+                                         cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (K <= 0 || (K & 31) || M > 16 || !x || !h_io || !gain || !shift) return SX_ERR_SIZE;
+  if (((uintptr_t)W & 15) || ((uintptr_t)x & 15)) return SX_ERR_ALIGN;
+  const SkNorm nrm = {nullptr, 0, 0.f, h_io, gain, nullptr, bias, 0.f, alpha, shift};
+  return skinny_pick_nt<EPI_RESID_TANH, false>(ks, (const bf16*)x, (const bf16*)W, out, M, N, K, nullptr, nullptr, nullptr, nullptr,
+                                               0.f, nrm, stream);
 }

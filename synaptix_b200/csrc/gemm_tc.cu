@@ -27,10 +27,10 @@
 #define TC_A_BYTES (TC_BM * TC_BK * 2)            // 16 KB
 #define TC_THREADS 192
 // (the epilogue that prepares heads has eight epilogue warps, one group of four per head of the tile)
-template <int EPI> struct TcThreads { static constexpr int N = EPI == 4 ? 320 : TC_THREADS; };
+template <int EPI> struct TcThreads { static constexpr int N = (EPI == 4 || EPI == 6) ? 320 : TC_THREADS; };
 #define TC_RED_ROWS 6
 
-enum { TC_EPI_BF16 = 0, TC_EPI_F32 = 1, TC_EPI_SILU_MUL = 2, TC_EPI_PARTIAL = 3, TC_EPI_QKV = 4 };
+enum { TC_EPI_BF16 = 0, TC_EPI_F32 = 1, TC_EPI_SILU_MUL = 2, TC_EPI_PARTIAL = 3, TC_EPI_QKV = 4, TC_EPI_RESID_TANH = 5, TC_EPI_QKV_BIAS = 6 };
 
 // TC_EPI_QKV: the product is the fused q/k/v projection of a prompt step with heads of 128, and its epilogue is the head
 // preparation (what sx_qkv_prepare does to the projection): a 128 x 256 tile holds two whole heads of 128 tokens, an
@@ -41,6 +41,7 @@ struct TcQkv {
   bf16* q_out;
   bf16* k_pages;
   bf16* v_pages;
+  const float* bias;        // TC_EPI_QKV_BIAS: [N], added to the projection
   const float* wq;
   const float* wk;
   const float* cs;
@@ -50,6 +51,19 @@ struct TcQkv {
   const int* block_table;
   int maxp, nh, nkv, n_pages;
   float eps;
+};
+
+// What an epilogue does besides rounding.  bias [N] (a stacked [gate; up] matrix: gate biases, then up biases) is added to
+// the product ahead of everything else; cap limits float32 results softly; TC_EPI_RESID_TANH adds the product into the
+// float32 residual stream h [M, N] in place and stores that sum's norm without statistics, tanh(alpha h) * gain + shift.
+struct TcEp {
+  GateAct act;
+  const float* bias;
+  float cap;
+  float* h;
+  float alpha;
+  const float* gain;
+  const float* shift;
 };
 
 // BN: columns of W per block (256, or 128 for the split-K form); stages fill the shared memory
@@ -214,41 +228,157 @@ __device__ __forceinline__ void tc_mbar_arrive(uint32_t bar) {
   asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(bar) : "memory");
 }
 
+// Four columns of one row: a[] the product, b[] (a stacked [gate; up] matrix) the up half's; bias, epilogue, store.  `cols`
+// of the four are inside the matrix.
 template <int EPI>
-__device__ __forceinline__ void tc_store_chunk(const uint32_t (&v)[32], const uint32_t (&u)[32], void* __restrict__ out,
-                                               int row, int col, int n_out, const GateAct act) {
-  float f[32];
-#pragma unroll
-  for (int i = 0; i < 32; ++i) {
-    f[i] = __uint_as_float(v[i]);
-    if (EPI == TC_EPI_SILU_MUL) f[i] = gate_mul(f[i], __uint_as_float(u[i]), act);
-  }
-  const int ncol = min(32, n_out - col);
-  if (EPI == TC_EPI_F32) {
-    float* dst = reinterpret_cast<float*>(out) + (size_t)row * n_out + col;
-    if (ncol == 32 && (n_out % 4) == 0) {
-#pragma unroll
-      for (int i = 0; i < 8; ++i) reinterpret_cast<float4*>(dst)[i] = make_float4(f[4 * i], f[4 * i + 1], f[4 * i + 2], f[4 * i + 3]);
-    } else {
-#pragma unroll
-      for (int i = 0; i < 32; ++i) if (i < ncol) dst[i] = f[i];
-    }
-  } else {
-    bf16* dst = reinterpret_cast<bf16*>(out) + (size_t)row * n_out + col;
-    if (ncol == 32 && (n_out % 8) == 0) {
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        uint4 p;
-        __nv_bfloat162 t0 = __floats2bfloat162_rn(f[8 * i], f[8 * i + 1]), t1 = __floats2bfloat162_rn(f[8 * i + 2], f[8 * i + 3]);
-        __nv_bfloat162 t2 = __floats2bfloat162_rn(f[8 * i + 4], f[8 * i + 5]), t3 = __floats2bfloat162_rn(f[8 * i + 6], f[8 * i + 7]);
-        p.x = *reinterpret_cast<uint32_t*>(&t0); p.y = *reinterpret_cast<uint32_t*>(&t1);
-        p.z = *reinterpret_cast<uint32_t*>(&t2); p.w = *reinterpret_cast<uint32_t*>(&t3);
-        reinterpret_cast<uint4*>(dst)[i] = p;
+__device__ __forceinline__ void tc_store4(float (&a)[4], const float (&b)[4], void* __restrict__ out, size_t row, int col, int cols,
+                                          int n_out, const TcEp& ep) {
+  const bool vec = cols >= 4 && (n_out & 3) == 0;
+  float u[4] = {b[0], b[1], b[2], b[3]};
+  if (ep.bias) {
+    if (vec) {
+      const float4 f = __ldg(reinterpret_cast<const float4*>(ep.bias + col));
+      a[0] += f.x; a[1] += f.y; a[2] += f.z; a[3] += f.w;
+      if (EPI == TC_EPI_SILU_MUL) {
+        const float4 g = __ldg(reinterpret_cast<const float4*>(ep.bias + n_out + col));
+        u[0] += g.x; u[1] += g.y; u[2] += g.z; u[3] += g.w;
       }
     } else {
 #pragma unroll
-      for (int i = 0; i < 32; ++i) if (i < ncol) dst[i] = __float2bfloat16_rn(f[i]);
+      for (int j = 0; j < 4; ++j)
+        if (j < cols) {
+          a[j] += __ldg(ep.bias + col + j);
+          if (EPI == TC_EPI_SILU_MUL) u[j] += __ldg(ep.bias + n_out + col + j);
+        }
     }
+  }
+  const size_t at = row * n_out + col;
+  if (EPI == TC_EPI_SILU_MUL) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) a[j] = gate_mul(a[j], u[j], ep.act);
+  }
+  if (EPI == TC_EPI_F32) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) a[j] = soft_limit(a[j], ep.cap);
+    float* dst = reinterpret_cast<float*>(out) + at;
+    if (vec) *reinterpret_cast<float4*>(dst) = make_float4(a[0], a[1], a[2], a[3]);
+    else
+#pragma unroll
+      for (int j = 0; j < 4; ++j) if (j < cols) dst[j] = a[j];
+    return;
+  }
+  if (EPI == TC_EPI_RESID_TANH) {
+    float* h = ep.h + at;
+    if (vec) {
+      const float4 hv = *reinterpret_cast<const float4*>(h);
+      const float4 w = __ldg(reinterpret_cast<const float4*>(ep.gain + col)), s = __ldg(reinterpret_cast<const float4*>(ep.shift + col));
+      a[0] += hv.x; a[1] += hv.y; a[2] += hv.z; a[3] += hv.w;
+      *reinterpret_cast<float4*>(h) = make_float4(a[0], a[1], a[2], a[3]);
+      a[0] = dyn_tanh(a[0], ep.alpha, w.x, s.x); a[1] = dyn_tanh(a[1], ep.alpha, w.y, s.y);
+      a[2] = dyn_tanh(a[2], ep.alpha, w.z, s.z); a[3] = dyn_tanh(a[3], ep.alpha, w.w, s.w);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (j < cols) {
+          const float v = h[j] + a[j];
+          h[j] = v;
+          a[j] = dyn_tanh(v, ep.alpha, __ldg(ep.gain + col + j), __ldg(ep.shift + col + j));
+        }
+    }
+  }
+  bf16* dst = reinterpret_cast<bf16*>(out) + at;
+  if (vec) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(a[0], a[1]), hi = __floats2bfloat162_rn(a[2], a[3]);
+    uint2 pkd;
+    pkd.x = *reinterpret_cast<uint32_t*>(&lo); pkd.y = *reinterpret_cast<uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(dst) = pkd;
+  } else {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) if (j < cols) dst[j] = __float2bfloat16_rn(a[j]);
+  }
+}
+
+// 32 columns of one row out of the accumulator (u: the up half's)
+template <int EPI>
+__device__ __forceinline__ void tc_store_chunk(const uint32_t (&v)[32], const uint32_t (&u)[32], void* __restrict__ out,
+                                               int row, int col, int n_out, const TcEp& ep) {
+  const int ncol = min(32, n_out - col);
+  if (ncol < 32 || (n_out & 7) != 0) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      float a[4], b[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        a[j] = __uint_as_float(v[4 * i + j]);
+        if (EPI == TC_EPI_SILU_MUL) b[j] = __uint_as_float(u[4 * i + j]);
+      }
+      if (4 * i < ncol) tc_store4<EPI>(a, b, out, (size_t)row, col + 4 * i, ncol - 4 * i, n_out, ep);
+    }
+    return;
+  }
+  float f[32];
+#pragma unroll
+  for (int i = 0; i < 32; ++i) f[i] = __uint_as_float(v[i]);
+  const size_t at = (size_t)row * n_out + col;
+  float hv[EPI == TC_EPI_RESID_TANH ? 32 : 1];
+  if (EPI == TC_EPI_RESID_TANH) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float4 h4 = reinterpret_cast<const float4*>(ep.h + at)[i];
+      hv[4 * i] = h4.x; hv[4 * i + 1] = h4.y; hv[4 * i + 2] = h4.z; hv[4 * i + 3] = h4.w;
+    }
+  }
+  if (ep.bias) {
+    const float4* b4 = reinterpret_cast<const float4*>(ep.bias + col);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float4 b = __ldg(b4 + i);
+      f[4 * i] += b.x; f[4 * i + 1] += b.y; f[4 * i + 2] += b.z; f[4 * i + 3] += b.w;
+    }
+  }
+  if (EPI == TC_EPI_SILU_MUL) {
+    const float4* b4 = reinterpret_cast<const float4*>(ep.bias + n_out + col);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (ep.bias) b = __ldg(b4 + i);
+      f[4 * i] = gate_mul(f[4 * i], __uint_as_float(u[4 * i]) + b.x, ep.act);
+      f[4 * i + 1] = gate_mul(f[4 * i + 1], __uint_as_float(u[4 * i + 1]) + b.y, ep.act);
+      f[4 * i + 2] = gate_mul(f[4 * i + 2], __uint_as_float(u[4 * i + 2]) + b.z, ep.act);
+      f[4 * i + 3] = gate_mul(f[4 * i + 3], __uint_as_float(u[4 * i + 3]) + b.w, ep.act);
+    }
+  }
+  if (EPI == TC_EPI_F32) {
+    float* dst = reinterpret_cast<float*>(out) + at;
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      reinterpret_cast<float4*>(dst)[i] = make_float4(soft_limit(f[4 * i], ep.cap), soft_limit(f[4 * i + 1], ep.cap),
+                                                      soft_limit(f[4 * i + 2], ep.cap), soft_limit(f[4 * i + 3], ep.cap));
+    return;
+  }
+  if (EPI == TC_EPI_RESID_TANH) {
+    const float4 *w4 = reinterpret_cast<const float4*>(ep.gain + col), *s4 = reinterpret_cast<const float4*>(ep.shift + col);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float4 w = __ldg(w4 + i), s = __ldg(s4 + i);
+      const float x0 = f[4 * i] + hv[4 * i], x1 = f[4 * i + 1] + hv[4 * i + 1], x2 = f[4 * i + 2] + hv[4 * i + 2],
+                  x3 = f[4 * i + 3] + hv[4 * i + 3];
+      reinterpret_cast<float4*>(ep.h + at)[i] = make_float4(x0, x1, x2, x3);
+      f[4 * i] = dyn_tanh(x0, ep.alpha, w.x, s.x);
+      f[4 * i + 1] = dyn_tanh(x1, ep.alpha, w.y, s.y);
+      f[4 * i + 2] = dyn_tanh(x2, ep.alpha, w.z, s.z);
+      f[4 * i + 3] = dyn_tanh(x3, ep.alpha, w.w, s.w);
+    }
+  }
+  bf16* dst = reinterpret_cast<bf16*>(out) + at;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    uint4 p;
+    __nv_bfloat162 t0 = __floats2bfloat162_rn(f[8 * i], f[8 * i + 1]), t1 = __floats2bfloat162_rn(f[8 * i + 2], f[8 * i + 3]);
+    __nv_bfloat162 t2 = __floats2bfloat162_rn(f[8 * i + 4], f[8 * i + 5]), t3 = __floats2bfloat162_rn(f[8 * i + 6], f[8 * i + 7]);
+    p.x = *reinterpret_cast<uint32_t*>(&t0); p.y = *reinterpret_cast<uint32_t*>(&t1);
+    p.z = *reinterpret_cast<uint32_t*>(&t2); p.w = *reinterpret_cast<uint32_t*>(&t3);
+    reinterpret_cast<uint4*>(dst)[i] = p;
   }
 }
 
@@ -316,7 +446,8 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
                                                                            float* __restrict__ piece_ws,
                                                                            int* __restrict__ piece_count,
                                                                            int* __restrict__ status, const TcQkv qk,
-                                                                           const GateAct act) {
+                                                                           const TcEp ep) {
+  constexpr bool QKV = EPI == TC_EPI_QKV || EPI == TC_EPI_QKV_BIAS;
   constexpr int STAGES = TcShape<BN>::STAGES, B_BYTES = TcShape<BN>::B_BYTES, STAGE_BYTES = TcShape<BN>::STAGE_BYTES;
   extern __shared__ unsigned char tc_smem_raw[];
   unsigned char* tiles = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(tc_smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -453,7 +584,7 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
       // (head preparation: where this thread's token goes is looked up while the tile's MMAs still run)
       const bool live = row < M;
       int pos = 0, page = -1;
-      if (EPI == TC_EPI_QKV && live) {
+      if (QKV && live) {
         pos = qk.positions[row];
         page = qk.block_table[(size_t)qk.seq_of_token[row] * qk.maxp + (pos >> 6)];
       }
@@ -463,15 +594,29 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
       }
       asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
       const uint32_t t_row = tmem_base + buf * BN + ((uint32_t)(quarter * 32) << 16);
-      if (EPI == TC_EPI_QKV) {
+      if (QKV) {
         // head preparation: this thread's token, the tile's two heads one after the other
         const bool page_ok = page >= 0 && page < qk.n_pages;
         {
           const int hh = (warp - 2) >> 2;                 // warps 2-5 take the tile's first head, warps 6-9 its second
           const int head = n0 / 128 + hh;
           float x[128];
+          // (with biases 32 columns at a time, each with its wait: this epilogue is short of registers, and the biases of a
+          //  whole head on the way at once would spill)
 #pragma unroll
-          for (int c = 0; c < 4; ++c) tc_ld32(t_row + hh * 128 + c * 32, *reinterpret_cast<uint32_t(*)[32]>(&x[c * 32]));
+          for (int c = 0; c < 4; ++c) {
+            tc_ld32(t_row + hh * 128 + c * 32, *reinterpret_cast<uint32_t(*)[32]>(&x[c * 32]));
+            if (EPI == TC_EPI_QKV_BIAS) {
+              asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+#pragma unroll
+              for (int i = 0; i < 8; ++i) {
+                float4 b;
+                asm volatile("ld.global.v4.f32 {%0, %1, %2, %3}, [%4];\n" : "=f"(b.x), "=f"(b.y), "=f"(b.z), "=f"(b.w)
+                             : "l"(qk.bias + head * 128 + c * 32 + 4 * i) : "memory");
+                x[c * 32 + 4 * i] += b.x; x[c * 32 + 4 * i + 1] += b.y; x[c * 32 + 4 * i + 2] += b.z; x[c * 32 + 4 * i + 3] += b.w;
+              }
+            }
+          }
           asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
 #pragma unroll
           for (int i = 0; i < 128; ++i) x[i] = __bfloat162float(__float2bfloat16_rn(x[i]));
@@ -547,7 +692,7 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
             __syncwarp();
             if (lane == 0) tc_mbar_arrive(acc_empty0 + 8 * buf);
           }
-          if (row < M && n0 + c0 < n_out) tc_store_chunk<EPI>(v, u, out, row, n0 + c0, n_out, act);
+          if (row < M && n0 + c0 < n_out) tc_store_chunk<EPI>(v, u, out, row, n0 + c0, n_out, ep);
         }
       }
       return true;
@@ -658,31 +803,8 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
             const int r = rb + i * RPI;
             if (r >= r_hi) continue;
             float o[4] = {a[i].x, a[i].y, a[i].z, a[i].w};
-            if (EPI == TC_EPI_SILU_MUL) {
-              const float u[4] = {b[i].x, b[i].y, b[i].z, b[i].w};
-#pragma unroll
-              for (int j = 0; j < 4; ++j) o[j] = gate_mul(o[j], u[j], act);
-            }
-            const size_t at = (size_t)r * n_out + n0 + c4;
-            const bool vec = c4 + 3 < cols && (n_out & 3) == 0;
-            if (EPI == TC_EPI_F32) {
-              float* dst = reinterpret_cast<float*>(out) + at;
-              if (vec) *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
-              else
-#pragma unroll
-                for (int j = 0; j < 4; ++j) if (c4 + j < cols) dst[j] = o[j];
-            } else {
-              bf16* dst = reinterpret_cast<bf16*>(out) + at;
-              if (vec) {
-                __nv_bfloat162 lo = __floats2bfloat162_rn(o[0], o[1]), hi = __floats2bfloat162_rn(o[2], o[3]);
-                uint2 pkd;
-                pkd.x = *reinterpret_cast<uint32_t*>(&lo); pkd.y = *reinterpret_cast<uint32_t*>(&hi);
-                *reinterpret_cast<uint2*>(dst) = pkd;
-              } else {
-#pragma unroll
-                for (int j = 0; j < 4; ++j) if (c4 + j < cols) dst[j] = __float2bfloat16_rn(o[j]);
-              }
-            }
+            const float u[4] = {b[i].x, b[i].y, b[i].z, b[i].w};
+            tc_store4<EPI>(o, u, out, (size_t)r, n0 + c4, cols - c4, n_out, ep);
           }
         }
       }
@@ -749,7 +871,7 @@ static int tc_sm_count() {
 // four columns).  Used when the persistent kernel had no whole tiles to hide its own adding-up behind.
 template <int EPI, int BN>
 __global__ void tc_pieces_reduce_kernel(const float* __restrict__ ws, void* __restrict__ out, int M, int N, int n_whole,
-                                        int R, int nkb, int G, int zmax, int sp, const GateAct act) {
+                                        int R, int nkb, int G, int zmax, int sp, const TcEp ep) {
   pdl_wait();
   pdl_trigger();
   const int n_out = (EPI == TC_EPI_SILU_MUL) ? N / 2 : N;
@@ -781,29 +903,8 @@ __global__ void tc_pieces_reduce_kernel(const float* __restrict__ ws, void* __re
     }
   }
   float o[4] = {a.x, a.y, a.z, a.w};
-  if (EPI == TC_EPI_SILU_MUL) {
-    const float u[4] = {b.x, b.y, b.z, b.w};
-#pragma unroll
-    for (int j = 0; j < 4; ++j) o[j] = gate_mul(o[j], u[j], act);
-  }
-  const size_t at = (size_t)r * n_out + n0 + c4;
-  const bool vec = c4 + 3 < cols && (n_out & 3) == 0;
-  if (EPI == TC_EPI_F32) {
-    float* dst = reinterpret_cast<float*>(out) + at;
-    if (vec) *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
-    else
-      for (int j = 0; j < 4; ++j) if (c4 + j < cols) dst[j] = o[j];
-  } else {
-    bf16* dst = reinterpret_cast<bf16*>(out) + at;
-    if (vec) {
-      __nv_bfloat162 lo = __floats2bfloat162_rn(o[0], o[1]), hi = __floats2bfloat162_rn(o[2], o[3]);
-      uint2 pkd;
-      pkd.x = *reinterpret_cast<uint32_t*>(&lo); pkd.y = *reinterpret_cast<uint32_t*>(&hi);
-      *reinterpret_cast<uint2*>(dst) = pkd;
-    } else {
-      for (int j = 0; j < 4; ++j) if (c4 + j < cols) dst[j] = __float2bfloat16_rn(o[j]);
-    }
-  }
+  const float u[4] = {b.x, b.y, b.z, b.w};
+  tc_store4<EPI>(o, u, out, (size_t)r, n0 + c4, cols - c4, n_out, ep);
 }
 
 // What the persistent kernel does for a product: how many tiles are computed whole, how many are cut, the most
@@ -909,7 +1010,7 @@ extern "C" int sx_gemm_tc_plan(int M, int N, int K, int epi, int* out4) {
 
 template <int EPI, int BN>
 static int tc_launch_persistent(const CUtensorMap& ma, const CUtensorMap& mw, void* out, int M, int N, int K,
-                                const TcHostPlan& h, float* ws, int* counts, cudaStream_t stream, const TcQkv& qk = TcQkv()) {
+                                const TcHostPlan& h, float* ws, int* counts, const TcEp& ep, cudaStream_t stream, const TcQkv& qk = TcQkv()) {
   int* status = tc_status_word();
   if (!status) return (int)cudaErrorMemoryAllocation;
   if (h.n_whole < 0 || h.G <= 0) return SX_ERR_SIZE;
@@ -918,19 +1019,19 @@ static int tc_launch_persistent(const CUtensorMap& ma, const CUtensorMap& mw, vo
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   // with whole tiles after them, the blocks of a cut tile add up inside the kernel; without, a second kernel does
-  int rc = sx_launch(kern, h.G, dim3(TcThreads<EPI>::N), smem, stream, ma, mw, out, M, N, K, h.n_whole, h.zmax, h.sp, ws, counts, status, qk, g_sx_gate);
-  if (rc || h.R == 0 || h.sp > 0 || EPI == TC_EPI_QKV) return rc;
+  int rc = sx_launch(kern, h.G, dim3(TcThreads<EPI>::N), smem, stream, ma, mw, out, M, N, K, h.n_whole, h.zmax, h.sp, ws, counts, status, qk, ep);
+  if (rc || h.R == 0 || h.sp > 0 || EPI == TC_EPI_QKV || EPI == TC_EPI_QKV_BIAS) return rc;
   const int tile_n = (EPI == TC_EPI_SILU_MUL) ? BN / 2 : BN;
   const long long total = (long long)h.R * TC_BM * (tile_n / 4);
   return sx_launch(tc_pieces_reduce_kernel<EPI, BN>, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, (const float*)ws, out,
-                   M, N, h.n_whole, h.R, (K + TC_BK - 1) / TC_BK, h.G, h.zmax, 0, g_sx_gate);
+                   M, N, h.n_whole, h.R, (K + TC_BK - 1) / TC_BK, h.G, h.zmax, 0, ep);
 }
 
 // sum of the split-K partial tiles ws[splits][M][N] in split order, then the epilogue
 template <int EPI>
 // (out has rows of ldo values: a block of a larger matrix when ldo > the block's width)
 __global__ void tc_splitk_reduce_kernel(const float* __restrict__ ws, void* __restrict__ out, int splits, int M, int N,
-                                        long long ldo, const GateAct act) {
+                                        long long ldo, const TcEp ep) {
   pdl_wait();
   pdl_trigger();
   const int n_out = (EPI == TC_EPI_SILU_MUL) ? N / 2 : N;
@@ -944,16 +1045,24 @@ __global__ void tc_splitk_reduce_kernel(const float* __restrict__ ws, void* __re
     a += ws[z * plane + m * N + n];
     if (EPI == TC_EPI_SILU_MUL) b += ws[z * plane + m * N + n_out + n];
   }
+  if (ep.bias) {
+    a += __ldg(ep.bias + n);
+    if (EPI == TC_EPI_SILU_MUL) b += __ldg(ep.bias + n_out + n);
+  }
   const size_t o = m * (size_t)ldo + n;
-  if (EPI == TC_EPI_SILU_MUL) reinterpret_cast<bf16*>(out)[o] = __float2bfloat16_rn(gate_mul(a, b, act));
-  else if (EPI == TC_EPI_F32) reinterpret_cast<float*>(out)[o] = a;
-  else reinterpret_cast<bf16*>(out)[o] = __float2bfloat16_rn(a);
+  if (EPI == TC_EPI_SILU_MUL) reinterpret_cast<bf16*>(out)[o] = __float2bfloat16_rn(gate_mul(a, b, ep.act));
+  else if (EPI == TC_EPI_F32) reinterpret_cast<float*>(out)[o] = soft_limit(a, ep.cap);
+  else if (EPI == TC_EPI_RESID_TANH) {
+    const float v = ep.h[o] + a;
+    ep.h[o] = v;
+    reinterpret_cast<bf16*>(out)[o] = __float2bfloat16_rn(dyn_tanh(v, ep.alpha, __ldg(ep.gain + n), __ldg(ep.shift + n)));
+  } else reinterpret_cast<bf16*>(out)[o] = __float2bfloat16_rn(a);
 }
 
 // K split over `splits` blocks per 128 x 128 tile, float32 partial tiles in `workspace` [splits, M, N], then the sum
 // in split order with the epilogue into out (rows of ldo values)
 static int tc_split_product(const void* A, const void* W, void* out, int M, int N, int K, int epi, int splits,
-                            float* workspace, long long ldo, cudaStream_t stream) {
+                            float* workspace, long long ldo, const TcEp& ep, cudaStream_t stream) {
   CUtensorMap ma, mw;
   int rc = tc_make_map(&ma, A, M, K);
   if (rc) return rc;
@@ -967,9 +1076,12 @@ static int tc_split_product(const void* A, const void* W, void* out, int M, int 
   const size_t n_elems = (size_t)M * (epi == TC_EPI_SILU_MUL ? N / 2 : N);
   const unsigned grid = (unsigned)((n_elems + 255) / 256);
   switch (epi) {
-    case TC_EPI_BF16: return sx_launch(tc_splitk_reduce_kernel<TC_EPI_BF16>, dim3(grid), dim3(256), 0, stream, (const float*)workspace, out, splits, M, N, ldo, g_sx_gate);
-    case TC_EPI_F32: return sx_launch(tc_splitk_reduce_kernel<TC_EPI_F32>, dim3(grid), dim3(256), 0, stream, (const float*)workspace, out, splits, M, N, ldo, g_sx_gate);
-    case TC_EPI_SILU_MUL: return sx_launch(tc_splitk_reduce_kernel<TC_EPI_SILU_MUL>, dim3(grid), dim3(256), 0, stream, (const float*)workspace, out, splits, M, N, ldo, g_sx_gate);
+#define TC_SPLITK_CASE(E) case E: return sx_launch(tc_splitk_reduce_kernel<E>, dim3(grid), dim3(256), 0, stream, (const float*)workspace, out, splits, M, N, ldo, ep)
+    TC_SPLITK_CASE(TC_EPI_BF16);
+    TC_SPLITK_CASE(TC_EPI_F32);
+    TC_SPLITK_CASE(TC_EPI_SILU_MUL);
+    TC_SPLITK_CASE(TC_EPI_RESID_TANH);
+#undef TC_SPLITK_CASE
     default: return SX_ERR_DTYPE;
   }
 }
@@ -983,15 +1095,22 @@ static int tc_split_product(const void* A, const void* W, void* out, int M, int 
 // splits > 1: 128 x 128 tiles, K split over `splits` blocks whose float32 partial tiles go to `workspace`
 //   [splits, M, N] and are added, in split order, by a second kernel that applies the epilogue.  Every split
 //   gets a non-empty range of K.
+// bias [N] (or null) is added to the product ahead of everything an epilogue does with it; epi 1 limits the sum softly at cap
+// (0: not at all).  epi 5: h f32 [M, N] += product in place, out bf16 [M, N] = tanh(alpha h) * gain + shift.
 extern "C" int sx_gemm_tc(const void* A, const void* W, void* out, int M, int N, int K, int epi, int splits,
-                          float* workspace, unsigned long long ws_floats, int* counts, cudaStream_t stream) {
+                          float* workspace, unsigned long long ws_floats, int* counts, const float* bias, float cap, float* h_io,
+                          float alpha, const float* gain, const float* shift, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
+  if (epi == TC_EPI_RESID_TANH && (!h_io || !gain || !shift)) return SX_ERR_SIZE;
+  if (((uintptr_t)bias | (uintptr_t)h_io | (uintptr_t)gain | (uintptr_t)shift) & 15) return SX_ERR_ALIGN;
+  TcEp ep;
+  ep.act = g_sx_gate; ep.bias = bias; ep.cap = cap; ep.h = h_io; ep.alpha = alpha; ep.gain = gain; ep.shift = shift;
   if (K <= 0 || (K & 7) || splits < 1) return SX_ERR_SIZE;
   if (epi == TC_EPI_SILU_MUL && (N & 1)) return SX_ERR_SIZE;
   if (((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return SX_ERR_ALIGN;
   if (splits > 1) {
     if (!workspace || ws_floats < (unsigned long long)splits * M * N) return SX_ERR_SIZE;
-    return tc_split_product(A, W, out, M, N, K, epi, splits, workspace, epi == TC_EPI_SILU_MUL ? N / 2 : N, stream);
+    return tc_split_product(A, W, out, M, N, K, epi, splits, workspace, epi == TC_EPI_SILU_MUL ? N / 2 : N, ep, stream);
   }
   CUtensorMap ma, mw;
   int rc = tc_make_map(&ma, A, M, K);
@@ -1003,24 +1122,26 @@ extern "C" int sx_gemm_tc(const void* A, const void* W, void* out, int M, int N,
   switch (epi) {
     // (128-wide tiles were tried for shapes whose last wave is nearly empty: the MMA then waits on
     //  shared-memory reads of A and the product got slower, 607 against 828 TFLOP/s)
-    case TC_EPI_BF16: return tc_launch_persistent<TC_EPI_BF16, 256>(ma, mw, out, M, N, K, h, workspace, counts, stream);
-    case TC_EPI_F32: return tc_launch_persistent<TC_EPI_F32, 256>(ma, mw, out, M, N, K, h, workspace, counts, stream);
-    case TC_EPI_SILU_MUL: return tc_launch_persistent<TC_EPI_SILU_MUL, 256>(ma, mw, out, M, N, K, h, workspace, counts, stream);
+    case TC_EPI_BF16: return tc_launch_persistent<TC_EPI_BF16, 256>(ma, mw, out, M, N, K, h, workspace, counts, ep, stream);
+    case TC_EPI_F32: return tc_launch_persistent<TC_EPI_F32, 256>(ma, mw, out, M, N, K, h, workspace, counts, ep, stream);
+    case TC_EPI_SILU_MUL: return tc_launch_persistent<TC_EPI_SILU_MUL, 256>(ma, mw, out, M, N, K, h, workspace, counts, ep, stream);
+    case TC_EPI_RESID_TANH: return tc_launch_persistent<TC_EPI_RESID_TANH, 256>(ma, mw, out, M, N, K, h, workspace, counts, ep, stream);
     default: return SX_ERR_DTYPE;
   }
 }
 
 // The fused q/k/v projection of a prompt step with its head preparation as the epilogue (see TcQkv): A [M, K], W [N, K] with
-// N = (nh + 2 nkv) * 128 a multiple of 256; q_out [M, nh * 128]; k_pages / v_pages [n_pages, nkv, 64, 128] (null: nothing is
+// N = (nh + 2 nkv) * 128 (or nh * 128: query heads alone, of a layer that reads another layer's cache) a multiple of 256;
+// bias [N] (null: none); q_out [M, nh * 128]; k_pages / v_pages [n_pages, nkv, 64, 128] (null: nothing is
 // written to the cache); wq / wk [128] (null: no norm); cs / sn [M, 64] (null: no rotation).  All tiles are computed whole.
-extern "C" int sx_gemm_tc_qkv(const void* A, const void* W, int M, int N, int K, void* q_out, void* k_pages, void* v_pages,
+extern "C" int sx_gemm_tc_qkv(const void* A, const void* W, const float* bias, int M, int N, int K, void* q_out, void* k_pages, void* v_pages,
                               const float* wq, const float* wk, const float* cs, const float* sn, const int* positions,
                               const int* seq_of_token, const int* block_table, int maxp, int nh, int nkv, int n_pages,
                               float eps, cudaStream_t stream) {
   if (M <= 0) return 0;
-  if (K <= 0 || (K & 7) || nh <= 0 || nkv <= 0 || N != (nh + 2 * nkv) * 128 || (N & 255) || !q_out || (!cs) != (!sn)) return SX_ERR_SIZE;
+  if (K <= 0 || (K & 7) || nh <= 0 || nkv <= 0 || (N != (nh + 2 * nkv) * 128 && N != nh * 128) || (N & 255) || !q_out || (!cs) != (!sn)) return SX_ERR_SIZE;
   if (((uintptr_t)A & 15) || ((uintptr_t)W & 15) || ((uintptr_t)q_out & 15) || ((uintptr_t)k_pages & 15) || ((uintptr_t)v_pages & 15) ||
-      ((uintptr_t)wq & 15) || ((uintptr_t)wk & 15) || ((uintptr_t)cs & 15) || ((uintptr_t)sn & 15))
+      ((uintptr_t)wq & 15) || ((uintptr_t)wk & 15) || ((uintptr_t)cs & 15) || ((uintptr_t)sn & 15) || ((uintptr_t)bias & 15))
     return SX_ERR_ALIGN;
   CUtensorMap ma, mw;
   int rc = tc_make_map(&ma, A, M, K);
@@ -1028,10 +1149,11 @@ extern "C" int sx_gemm_tc_qkv(const void* A, const void* W, int M, int N, int K,
   if ((rc = tc_make_map(&mw, W, N, K))) return rc;
   const TcHostPlan h = tc_plan_stream(M, N, K, TC_EPI_BF16, false);
   TcQkv qk;
-  qk.q_out = (bf16*)q_out; qk.k_pages = (bf16*)k_pages; qk.v_pages = (bf16*)v_pages; qk.wq = wq; qk.wk = wk; qk.cs = cs; qk.sn = sn;
+  qk.q_out = (bf16*)q_out; qk.k_pages = (bf16*)k_pages; qk.v_pages = (bf16*)v_pages; qk.bias = bias; qk.wq = wq; qk.wk = wk; qk.cs = cs; qk.sn = sn;
   qk.positions = positions; qk.seq_of_token = seq_of_token; qk.block_table = block_table;
   qk.maxp = maxp; qk.nh = nh; qk.nkv = nkv; qk.n_pages = n_pages; qk.eps = eps;
-  return tc_launch_persistent<TC_EPI_QKV, 256>(ma, mw, nullptr, M, N, K, h, nullptr, nullptr, stream, qk);
+  if (bias) return tc_launch_persistent<TC_EPI_QKV_BIAS, 256>(ma, mw, nullptr, M, N, K, h, nullptr, nullptr, TcEp(), stream, qk);
+  return tc_launch_persistent<TC_EPI_QKV, 256>(ma, mw, nullptr, M, N, K, h, nullptr, nullptr, TcEp(), stream, qk);
 }
 
 // 0, or which bounded wait ran out (1 producer, 2 and 4 MMA issuer, 3 epilogue, 5 the blocks of a cut tile waiting for one another)

@@ -20,7 +20,8 @@
 //   all      after a cluster barrier: the sum over the cluster's blocks, the epilogue, the store
 // Epilogues: bfloat16 or float32 store; SiLU(gate) * up; both optionally times a factor per row of C,
 // rsqrt(sum(ssq[row]) / K + eps) (rows of X that lack their RMSNorm factor); or h += C in the float32
-// residual stream with bf16(h * gain) and partial sums of squares of h as outputs (what the next norm needs).
+// residual stream with bf16(h * gain) and partial sums of squares of h as outputs (what the next norm needs), or, where
+// the next norm has no statistics (dyn_tanh), with that norm's finished rows as output.  A bias per column may join.
 // Rows of W beyond N, rows of X beyond M and the tail of K are zero-filled by TMA: every size with K % 8 == 0.
 // Every wait on an mbarrier is bounded; a wait that runs out sets *status and the block still meets the
 // cluster's barriers and frees its tensor memory.
@@ -32,7 +33,7 @@
 #define WS_MAX_ROWS 256
 #define WS_MAX_STAGES 8
 
-enum { WS_EPI_BF16 = 0, WS_EPI_F32 = 1, WS_EPI_SILU_MUL = 2, WS_EPI_RESIDUAL = 3 };
+enum { WS_EPI_BF16 = 0, WS_EPI_F32 = 1, WS_EPI_SILU_MUL = 2, WS_EPI_RESIDUAL = 3, WS_EPI_RESID_TANH = 4 };
 
 struct WsEpilogue {
   const float* ssq_in;   // [M, n_ssq] partial sums of squares behind the row factors, or null
@@ -41,6 +42,10 @@ struct WsEpilogue {
   float* h;              // residual stream [M, N] (WS_EPI_RESIDUAL)
   const float* gain;     // [N]
   float* ssq_out;        // [M, tiles * splits]
+  const float* bias;     // [N] or null: added to the product (a stacked [gate; up] matrix: gate biases, then up biases)
+  float cap;             // WS_EPI_F32: soft_limit of the results (0: none)
+  float alpha;           // WS_EPI_RESID_TANH: out = bf16(tanh(alpha h) * gain + shift)
+  const float* shift;
   GateAct act;              // the gated activation of the SiLU-mul epilogue's place (see common.cuh)
 };
 
@@ -305,21 +310,54 @@ __global__ void __launch_bounds__(WS_THREADS, 2) gemm_ws_kernel(const __grid_con
       }
       float o[4] = {a.x, a.y, a.z, a.w};
       const float rf = (valid && ep.ssq_in != nullptr) ? row_factor[m] : 1.f;
+      float ba[4] = {0.f, 0.f, 0.f, 0.f}, bb[4] = {0.f, 0.f, 0.f, 0.f};
+      if (ep.bias != nullptr && valid) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (n0 + c + j < n_out) {
+            ba[j] = __ldg(ep.bias + n0 + c + j);
+            if (EPI == WS_EPI_SILU_MUL) bb[j] = __ldg(ep.bias + n_out + n0 + c + j);
+          }
+      }
       if (EPI == WS_EPI_SILU_MUL) {
         const float u[4] = {b.x, b.y, b.z, b.w};
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          o[j] = gate_mul(o[j] * rf, u[j] * rf, ep.act);
+          o[j] = gate_mul(fmaf(o[j], rf, ba[j]), fmaf(u[j], rf, bb[j]), ep.act);
         }
       } else {
 #pragma unroll
-        for (int j = 0; j < 4; ++j) o[j] *= rf;
+        for (int j = 0; j < 4; ++j) o[j] = fmaf(o[j], rf, ba[j]);
+        if (EPI == WS_EPI_F32)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) o[j] = soft_limit(o[j], ep.cap);
       }
       const int n = n0 + c;
       const int cols = valid ? min(4, n_out - n) : 0;                      // <= 0: beyond the matrix
       const size_t at = (size_t)m * n_out + n;
       const bool vec = cols == 4 && (n_out & 3) == 0;
-      if (EPI == WS_EPI_RESIDUAL) {
+      if (EPI == WS_EPI_RESID_TANH) {
+        if (cols > 0) {
+          bf16* xo = reinterpret_cast<bf16*>(out) + at;
+          if (vec) {
+            const float4 h4 = *reinterpret_cast<const float4*>(ep.h + at);
+            const float4 g4v = *reinterpret_cast<const float4*>(ep.gain + n), s4v = *reinterpret_cast<const float4*>(ep.shift + n);
+            const float4 v = make_float4(h4.x + o[0], h4.y + o[1], h4.z + o[2], h4.w + o[3]);
+            *reinterpret_cast<float4*>(ep.h + at) = v;
+            __nv_bfloat162 lo = __floats2bfloat162_rn(dyn_tanh(v.x, ep.alpha, g4v.x, s4v.x), dyn_tanh(v.y, ep.alpha, g4v.y, s4v.y));
+            __nv_bfloat162 hi = __floats2bfloat162_rn(dyn_tanh(v.z, ep.alpha, g4v.z, s4v.z), dyn_tanh(v.w, ep.alpha, g4v.w, s4v.w));
+            uint2 pk;
+            pk.x = *reinterpret_cast<uint32_t*>(&lo); pk.y = *reinterpret_cast<uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>(xo) = pk;
+          } else {
+            for (int j = 0; j < cols; ++j) {
+              const float v = ep.h[at + j] + o[j];
+              ep.h[at + j] = v;
+              xo[j] = __float2bfloat16_rn(dyn_tanh(v, ep.alpha, ep.gain[n + j], ep.shift[n + j]));
+            }
+          }
+        }
+      } else if (EPI == WS_EPI_RESIDUAL) {
         float sq = 0.f;
         if (cols > 0) {
           float hv[4] = {0.f, 0.f, 0.f, 0.f}, gv[4] = {0.f, 0.f, 0.f, 0.f};
@@ -486,11 +524,14 @@ static int ws_launch(const void* X, const void* W, void* out, int M, int N, int 
 // 3: h [M, N] float32 += the product in place, out bf16 [M, N] = bf16(h * gain), ssq_out [M, tiles * splits] the sums
 //    of squares of the new h over each block's columns (sx_gemm_ws_plan gives tiles and splits).
 // ssq_in (epi 0-2, may be null): [M, n_ssq] float32; row m of the result is multiplied by rsqrt(sum(ssq_in[m]) / K + eps).
+// 4: h [M, N] float32 += the product in place, out bf16 [M, N] = tanh(alpha h) * gain + shift.
+// bias [N] (or null) is added to the product ahead of everything an epilogue does with it; epi 1 limits the sum softly at
+// cap (0: not at all).
 // splits: blocks of a cluster that share a tile's K (1, 2, 4 or 8); 0 lets the library choose.
 // stages: depth of the ring (2 to 8, as far as shared memory holds them); 0 = what lets two blocks share an SM.
 extern "C" int sx_gemm_ws(const void* X, const void* W, void* out, int M, int N, int K, int epi, int splits, int stages,
                           const float* ssq_in, int n_ssq, float eps, float* h, const float* gain, float* ssq_out,
-                          cudaStream_t stream) {
+                          const float* bias, float cap, float alpha, const float* shift, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > WS_MAX_ROWS || K <= 0 || (K & 7)) return SX_ERR_SIZE;
   if (epi == WS_EPI_SILU_MUL && (N & 1)) return SX_ERR_SIZE;
@@ -503,6 +544,7 @@ extern "C" int sx_gemm_ws(const void* X, const void* W, void* out, int M, int N,
   while (splits > nkb) splits /= 2;
   WsEpilogue ep;
   ep.ssq_in = ssq_in; ep.n_ssq = n_ssq; ep.eps = eps; ep.h = h; ep.gain = gain; ep.ssq_out = ssq_out;
+  ep.bias = bias; ep.cap = cap; ep.alpha = alpha; ep.shift = shift;
   ep.act = g_sx_gate;
   switch (epi) {
     case WS_EPI_BF16: return ws_launch<WS_EPI_BF16>(X, W, out, M, N, K, splits, stages, ep, stream);
@@ -511,6 +553,9 @@ extern "C" int sx_gemm_ws(const void* X, const void* W, void* out, int M, int N,
     case WS_EPI_RESIDUAL:
       if (!h || !gain || !ssq_out || ssq_in) return SX_ERR_SIZE;
       return ws_launch<WS_EPI_RESIDUAL>(X, W, out, M, N, K, splits, stages, ep, stream);
+    case WS_EPI_RESID_TANH:
+      if (!h || !gain || !shift || ssq_in) return SX_ERR_SIZE;
+      return ws_launch<WS_EPI_RESID_TANH>(X, W, out, M, N, K, splits, stages, ep, stream);
     default: return SX_ERR_DTYPE;
   }
 }

@@ -170,13 +170,14 @@ extern "C" int sx_residual_add(float* h, const void* delta, long long n, int dt,
 }
 
 // ---------------------------------------------------------------------------------------
-// C[M,N] = A[M,K] * W[N,K]^T, 32-bit accumulation in k order.  Two kernels:
+// C[M,N] = A[M,K] * W[N,K]^T (+ bias[N]), then soft_limit(., cap), 32-bit accumulation in k order.  Two kernels:
 //   gemm_tile: 64x64x16 tiles, 4x4 outputs per thread (any M);
 //   gemm_rows: one warp per output column, up to 8 rows of A at a time (M <= 16).
 // ---------------------------------------------------------------------------------------
 template <typename TA, typename TW, typename TC>
 __global__ void __launch_bounds__(256) gemm_tile_kernel(const TA* __restrict__ A, const TW* __restrict__ W,
-                                                        TC* __restrict__ C, int M, int N, int K) {
+                                                        TC* __restrict__ C, int M, int N, int K,
+                                                        const float* __restrict__ bias, float cap) {
   constexpr int BM = 64, BN = 64, BK = 16;
   __shared__ float As[BK][BM + 4];
   __shared__ float Ws[BK][BN + 4];
@@ -221,14 +222,15 @@ __global__ void __launch_bounds__(256) gemm_tile_kernel(const TA* __restrict__ A
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < N) C[(size_t)m * N + n] = from_f32<TC>(acc[i][j]);
+      if (n < N) C[(size_t)m * N + n] = from_f32<TC>(soft_limit(bias ? acc[i][j] + bias[n] : acc[i][j], cap));
     }
   }
 }
 
 template <typename TA, typename TW, typename TC>
 __global__ void __launch_bounds__(128) gemm_rows_kernel(const TA* __restrict__ A, const TW* __restrict__ W,
-                                                        TC* __restrict__ C, int M, int N, int K) {
+                                                        TC* __restrict__ C, int M, int N, int K,
+                                                        const float* __restrict__ bias, float cap) {
   const int lane = threadIdx.x & 31;
   const int n = blockIdx.x * 4 + (threadIdx.x >> 5);
   if (n >= N) return;
@@ -246,36 +248,36 @@ __global__ void __launch_bounds__(128) gemm_rows_kernel(const TA* __restrict__ A
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       const float s = warp_sum(acc[i]);
-      if (lane == 0 && m0 + i < M) C[(size_t)(m0 + i) * N + n] = from_f32<TC>(s);
+      if (lane == 0 && m0 + i < M) C[(size_t)(m0 + i) * N + n] = from_f32<TC>(soft_limit(bias ? s + bias[n] : s, cap));
     }
   }
 }
 
 template <typename TA, typename TW, typename TC>
-static int gemm_generic_launch(const void* A, const void* W, void* C, int M, int N, int K,
+static int gemm_generic_launch(const void* A, const void* W, void* C, int M, int N, int K, const float* bias, float cap,
                                cudaStream_t stream) {
   if (M <= 16) {
-    gemm_rows_kernel<TA, TW, TC><<<(N + 3) / 4, 128, 0, stream>>>((const TA*)A, (const TW*)W, (TC*)C, M, N, K);
+    gemm_rows_kernel<TA, TW, TC><<<(N + 3) / 4, 128, 0, stream>>>((const TA*)A, (const TW*)W, (TC*)C, M, N, K, bias, cap);
   } else {
     dim3 grid((N + 63) / 64, (M + 63) / 64);
-    gemm_tile_kernel<TA, TW, TC><<<grid, 256, 0, stream>>>((const TA*)A, (const TW*)W, (TC*)C, M, N, K);
+    gemm_tile_kernel<TA, TW, TC><<<grid, 256, 0, stream>>>((const TA*)A, (const TW*)W, (TC*)C, M, N, K, bias, cap);
   }
   return sx_launch_status();
 }
 
 extern "C" int sx_gemm_generic(const void* A, int a_dt, const void* W, int w_dt, void* C, int c_dt,
-                               int M, int N, int K, cudaStream_t stream) {
+                               int M, int N, int K, const float* bias, float cap, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0) return SX_ERR_SIZE;
   if ((size_t)((M + 63) / 64) > 65535) return SX_ERR_SIZE;
   if (a_dt == SX_F32 && w_dt == SX_F32 && c_dt == SX_F32)
-    return gemm_generic_launch<float, float, float>(A, W, C, M, N, K, stream);
+    return gemm_generic_launch<float, float, float>(A, W, C, M, N, K, bias, cap, stream);
   if (a_dt == SX_BF16 && w_dt == SX_BF16 && c_dt == SX_BF16)
-    return gemm_generic_launch<bf16, bf16, bf16>(A, W, C, M, N, K, stream);
+    return gemm_generic_launch<bf16, bf16, bf16>(A, W, C, M, N, K, bias, cap, stream);
   if (a_dt == SX_BF16 && w_dt == SX_BF16 && c_dt == SX_F32)
-    return gemm_generic_launch<bf16, bf16, float>(A, W, C, M, N, K, stream);
+    return gemm_generic_launch<bf16, bf16, float>(A, W, C, M, N, K, bias, cap, stream);
   if (a_dt == SX_F32 && w_dt == SX_BF16 && c_dt == SX_F32)
-    return gemm_generic_launch<float, bf16, float>(A, W, C, M, N, K, stream);
+    return gemm_generic_launch<float, bf16, float>(A, W, C, M, N, K, bias, cap, stream);
   return SX_ERR_DTYPE;
 }
 

@@ -16,7 +16,9 @@
 //                          over the warp, and the weighted sum of c has a lane own the elements r = lane, lane + 32, ...
 //                          -> float32 [T, H, splits, R] without the division, and each part's maximum and sum
 //   latent_output_kernel   one block a (tile of 8 tokens, head): the parts merged and divided, then
-//                          y[h Dv + j] = sigmoid(gate_h) * sum_r Wuv[h Dv + j, r] o'[h, r]
+//                          y[h Dv + j] = sigmoid(gate) * sum_r Wuv[h Dv + j, r] o'[h, r], the gate one number a head or one
+//                          an output element; a sink per head (a term exp(sink) of the denominator without a key) joins
+//                          once, where the parts are merged
 // Rotation: dims elements, pair i at angle position * inv_freq[i]; pairs = 1: elements (2i, 2i + 1), pairs = 0:
 // elements (i, i + dims / 2); elements from dims on pass unchanged.  `mag` multiplies cos and sin (1 for a plain rotation;
 // a stretched rotation scales both).
@@ -353,7 +355,7 @@ extern "C" int sx_latent_attention(const float* qa, const void* k_pages, const i
 template <typename T>
 __global__ void __launch_bounds__(LT_THREADS) latent_output_kernel(
     const float* __restrict__ ol, const float* __restrict__ ml, int splits, const T* __restrict__ wuv, int H, int Dv, int R,
-    const T* __restrict__ proj, int row, int col_g, T* __restrict__ y, int n_tokens) {
+    const T* __restrict__ proj, int row, int col_g, int g_elem, const float* __restrict__ sinks, T* __restrict__ y, int n_tokens) {
   extern __shared__ float os[];          // LT_TOKENS * R
   __shared__ float wsp[LT_TOKENS][64];   // each split's weight exp(m_s - M) / L
   pdl_wait();
@@ -364,8 +366,9 @@ __global__ void __launch_bounds__(LT_THREADS) latent_output_kernel(
     const int tt = tid;
     if (tt < nt) {
       const float* p = ml + ((size_t)(t0 + tt) * H + h) * splits * 2;
-      float M = -INFINITY, L = 0.f;
+      float M = sinks ? sinks[h] : -INFINITY;
       for (int s = 0; s < splits; ++s) M = fmaxf(M, p[2 * s]);
+      float L = sinks ? expf(sinks[h] - M) : 0.f;
       for (int s = 0; s < splits; ++s) L += p[2 * s + 1] * (p[2 * s] == -INFINITY ? 0.f : expf(p[2 * s] - M));
       for (int s = 0; s < splits; ++s) wsp[tt][s] = (p[2 * s] == -INFINITY ? 0.f : expf(p[2 * s] - M)) / L;
     }
@@ -410,7 +413,7 @@ __global__ void __launch_bounds__(LT_THREADS) latent_output_kernel(
         const float s = warp_sum(acc[a][tt]);
         if (lane == 0 && tt < nt && j0 + a < Dv) {
           float g = 1.f;
-          if (col_g >= 0) g = 1.f / (1.f + expf(-to_f32(proj[(size_t)(t0 + tt) * row + col_g + h])));
+          if (col_g >= 0) g = 1.f / (1.f + expf(-to_f32(proj[(size_t)(t0 + tt) * row + col_g + (g_elem ? h * Dv + j0 + a : h)])));
           y[(size_t)(t0 + tt) * H * Dv + h * Dv + j0 + a] = from_f32<T>(s * g);
         }
       }
@@ -418,7 +421,8 @@ __global__ void __launch_bounds__(LT_THREADS) latent_output_kernel(
 }
 
 extern "C" int sx_latent_output(const float* ol, const float* ml, int splits, const void* wuv, int H, int Dv, int R,
-                                const void* proj, int row, int col_g, void* y, int T, int dt, cudaStream_t stream) {
+                                const void* proj, int row, int col_g, int g_elem, const float* sinks, void* y, int T, int dt,
+                                cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H <= 0 || H > 65535 || Dv <= 0 || R <= 0 || splits < 1 || splits > 64) return SX_ERR_SIZE;
   const size_t smem = (size_t)LT_TOKENS * R * sizeof(float);
@@ -426,10 +430,10 @@ extern "C" int sx_latent_output(const float* ol, const float* ml, int splits, co
   dim3 grid((T + LT_TOKENS - 1) / LT_TOKENS, H, (Dv + (LT_THREADS / 32) * LT_OUTS - 1) / ((LT_THREADS / 32) * LT_OUTS));
   if (dt == SX_F32)
     return sx_launch(latent_output_kernel<float>, grid, dim3(LT_THREADS), smem, stream, ol, ml, splits, (const float*)wuv, H, Dv, R,
-                     (const float*)proj, row, col_g, (float*)y, T);
+                     (const float*)proj, row, col_g, g_elem, sinks, (float*)y, T);
   if (dt == SX_BF16)
     return sx_launch(latent_output_kernel<bf16>, grid, dim3(LT_THREADS), smem, stream, ol, ml, splits, (const bf16*)wuv, H, Dv, R,
-                     (const bf16*)proj, row, col_g, (bf16*)y, T);
+                     (const bf16*)proj, row, col_g, g_elem, sinks, (bf16*)y, T);
   return SX_ERR_DTYPE;
 }
 

@@ -12,6 +12,7 @@ from . import pidutar as _pidutar  # registers the architecture
 from . import ledudra as _ledudra  # registers the architecture
 from . import tamovik as _tamovik  # registers the architecture
 from . import zekalorn as _zekalorn  # registers the architecture
+from . import penopel as _penopel  # registers the architecture
 from .decoder import DecoderModel, Inject, LayerRun, StreamVectors
 
 __all__ = ["DecoderModel", "Inject", "LayerRun", "StreamVectors", "model_skeleton", "load_model", "parse_dtype"]

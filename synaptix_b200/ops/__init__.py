@@ -16,9 +16,9 @@ from ._lib import KernelError, current_gate, gate_activation, late_launch, set_l
 from .attention import (TC_TILE_ROWS, attn_decode, attn_decode_ex, attn_decode_prep, attn_decode_tma, attn_prefill,
                         attn_prefill_ex, attn_prefill_tc,
                         fast_supported, pick_splits, query_tiles, tc_prefill_supported, tma_decode_supported)
-from .decode import MAX_ROWS as SKINNY_MAX_ROWS, skinny_gemm, skinny_gemm_residual, skinny_gemm_scaled, skinny_supported
-from .gemm_tc import gemm_tc, gemm_tc_qkv, qkv_epilogue_supported, tc_supported
-from .gemm_ws import gemm_ws, gemm_ws_residual, ws_supported
+from .decode import MAX_ROWS as SKINNY_MAX_ROWS, skinny_gemm, skinny_gemm_resid_tanh, skinny_gemm_residual, skinny_gemm_scaled, skinny_supported
+from .gemm_tc import gemm_tc, gemm_tc_qkv, gemm_tc_resid_tanh, qkv_epilogue_supported, tc_supported
+from .gemm_ws import gemm_ws, gemm_ws_resid_tanh, gemm_ws_residual, ws_supported
 from .options import OPTIONS, KernelOptions, options, set_options
 from .generic import (add_rmsnorm, attn_generic, decode_advance, decode_begin, embed_gather, gemm_generic, qkv_prepare,
                       residual_add, rope_table, silu_mul)
@@ -26,6 +26,7 @@ from .sequence import add_rmsnorm_conv, capped_glu, mingru, retention, stream_ad
 from .block import add_scaled, add_scaled_rmsnorm, scale_rows, side_gate
 from .delta import DeltaWeights, delta_rule, delta_step_fits
 from .layernorm import add_layernorm
+from .dyntanh import add_dyn_tanh
 from .normed import WeightedRows, add_normed, embed_bigram
 from .convqk import convqk_prepare, sigmoid_gate
 from .scored import attn_scored as attn_scored_all_heads, heads_prepare
@@ -41,7 +42,7 @@ __all__ = ["OPTIONS", "KernelOptions", "options", "set_options", "KernelsUnavail
            "add_rmsnorm_conv", "capped_glu", "mingru", "retention", "stream_add", "gate_activation",
            "add_normed", "WeightedRows", "embed_bigram", "convqk_prepare", "sigmoid_gate", "add_scaled", "add_scaled_rmsnorm", "scale_rows", "add_layernorm", "attn_scored", "heads_prepare", "latent_attention", "latent_output", "latent_prepare",
            "latent_query", "latent_gather", "latent_expand", "latent_rotate_q", "head_gate", "mlstm", "ExpertPlan", "moe_combine", "moe_down", "moe_gate_up", "moe_route", "moe_sort", "moe_up",
-           "late_launch", "side_gate", "DeltaWeights", "delta_rule", "delta_step_fits"]
+           "add_dyn_tanh", "linear_into_dyn_tanh", "late_launch", "side_gate", "DeltaWeights", "delta_rule", "delta_step_fits"]
 
 
 _STATUS_READERS = {"gemm_tc": ("the tcgen05 matrix product (gemm_tc)", "gemm_tc_status"),
@@ -133,8 +134,10 @@ SCALED_MAX_OUT = 65536
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
-           epilogue: Optional[str] = None) -> torch.Tensor:
-    """``x[M, K] @ w[N, K].T`` with 32-bit accumulation; output in ``out_dtype`` (default ``x``'s).
+           epilogue: Optional[str] = None, bias: Optional[torch.Tensor] = None, cap: float = 0.0) -> torch.Tensor:
+    """``x[M, K] @ w[N, K].T`` with 32-bit accumulation; output in ``out_dtype`` (default ``x``'s).  ``bias`` (float32
+    ``[N]``) is added to the product ahead of the epilogue; ``cap > 0`` (float32 output, no other epilogue): the result is
+    ``cap * tanh(. / cap)``.
     ``epilogue="silu_mul"``: ``w`` is ``[gate; up]`` stacked and the result is
     ``silu(x gate^T) * (x up^T)``, ``[M, N/2]``; inside ``gate_activation(alpha, limit)`` it is the capped form
     ``g sigmoid(alpha g) (u + 1)`` with ``g = min(x gate^T, limit)``, ``u = clamp(x up^T, -limit, limit)`` instead."""
@@ -142,6 +145,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = 
     N = w.shape[0]
     if out_dtype is None:
         out_dtype = x.dtype
+    if cap and (out_dtype != torch.float32 or epilogue is not None):
+        raise KernelError("a soft limit is put on float32 results")
     # up to 160 rows: stream W once (mma.sync or tcgen05 with W as the M side, see _weight_stream_kernel); more: the
     # tcgen05 product of prompt steps
     stream_k = _weight_stream_kernel(M, N, K, x.dtype, w.dtype) if out_dtype in (torch.bfloat16, torch.float32) else None
@@ -149,16 +154,16 @@ def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = 
         product = skinny_gemm if stream_k == "skinny" else gemm_ws
         if epilogue == "silu_mul":
             if out_dtype == torch.bfloat16:
-                return product(x, w, epilogue="silu_mul")
+                return product(x, w, epilogue="silu_mul", bias=bias)
         else:
-            return product(x, w, epilogue="f32" if out_dtype == torch.float32 else None)
+            return product(x, w, epilogue="f32" if out_dtype == torch.float32 else None, bias=bias, cap=cap)
     if tc_supported(M, N, K, x.dtype, w.dtype) and out_dtype in (torch.bfloat16, torch.float32):
         if epilogue == "silu_mul":
             if out_dtype == torch.bfloat16:
-                return gemm_tc(x, w, epilogue="silu_mul")
+                return gemm_tc(x, w, epilogue="silu_mul", bias=bias)
         else:
-            return gemm_tc(x, w, epilogue="f32" if out_dtype == torch.float32 else None)
-    y = gemm_generic(x, w, out_dtype=out_dtype if epilogue is None else x.dtype)
+            return gemm_tc(x, w, epilogue="f32" if out_dtype == torch.float32 else None, bias=bias, cap=cap)
+    y = gemm_generic(x, w, out_dtype=out_dtype if epilogue is None else x.dtype, bias=bias, cap=cap)
     if epilogue == "silu_mul":
         alpha, limit, form = current_gate()      # which gated activation the epilogue stands for (see gate_activation)
         y = capped_glu(y, alpha, limit, form) if (limit > 0 or form != 0) else silu_mul(y)
@@ -232,6 +237,25 @@ def linear_scaled(x: torch.Tensor, ssq: torch.Tensor, eps: float, w: torch.Tenso
     return gemm_ws(x, w, epilogue=epi, ssq=ssq, eps=eps)
 
 
+def linear_into_dyn_tanh(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], h: torch.Tensor, alpha: float,
+                         gain: torch.Tensor, shift: torch.Tensor) -> Optional[torch.Tensor]:
+    """``h += x @ w.T + bias`` (float32, in place) and the norm without statistics of that sum, ``tanh(alpha h) * gain +
+    shift`` in bfloat16, all in the product's epilogue, for any number of rows (option ``fused_residual``); ``None`` if no
+    kernel does that for these sizes and dtypes."""
+    M, K = x.shape
+    N = w.shape[0]
+    if not OPTIONS.fused_residual or x.dtype != torch.bfloat16:
+        return None
+    kind = _weight_stream_kernel(M, N, K, x.dtype, w.dtype)
+    if kind is not None:
+        product = skinny_gemm_resid_tanh if kind == "skinny" else gemm_ws_resid_tanh
+    elif tc_supported(M, N, K, x.dtype, w.dtype):
+        product = gemm_tc_resid_tanh
+    else:
+        return None
+    return product(x, w, bias, h, alpha, gain, shift)
+
+
 # Fewer rows than this and the fused projection is one of the weight-streaming products, which have no such epilogue.
 QKV_EPILOGUE_MIN_ROWS = WS_MAX_ROWS + 1
 
@@ -244,7 +268,8 @@ def projection_prepares_heads(M: int, K: int, x_dtype, w_dtype, nh: int, nkv: in
 
 
 def project_and_prepare(x: torch.Tensor, w: torch.Tensor, k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor],
-                        wq, wk, inv_freq, eps: float, ctx, block_table: torch.Tensor, nh: int, nkv: int, hd: int) -> torch.Tensor:
+                        wq, wk, inv_freq, eps: float, ctx, block_table: torch.Tensor, nh: int, nkv: int, hd: int,
+                        bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The prepared queries ``[T, nh * hd]`` of a prompt step straight from the block's input: the fused q/k/v product
     with the head preparation (per-head RMSNorm, rotation, cache write) as its epilogue.  The cosines and sines of the
     step's angles are made once a step and rotation (``ctx.scratch``) and shared by the layers."""
@@ -257,7 +282,7 @@ def project_and_prepare(x: torch.Tensor, w: torch.Tensor, k_pages: Optional[torc
         cos, sin = table
     q = torch.empty((x.shape[0], nh * hd), dtype=x.dtype, device=x.device)
     gemm_tc_qkv(x, w, q, k_pages, v_pages, wq, wk, cos, sin, eps, ctx.positions[:x.shape[0]], ctx.seq_of_token[:x.shape[0]],
-                block_table, nh, nkv)
+                block_table, nh, nkv, bias=bias)
     return q
 
 
@@ -270,15 +295,17 @@ def decode_attention_takes_projection(dtype, nh: int, nkv: int, hd: int, rotary_
 
 def attention_from_projection(qkv: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, ctx,
                               block_table: torch.Tensor, nh: int, nkv: int, hd: int, scale: float,
-                              window: Optional[int], wq, wk, inv_freq, eps: float, write_cache: bool) -> torch.Tensor:
+                              window: Optional[int], wq, wk, inv_freq, eps: float, write_cache: bool,
+                              sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Single-token steps: head preparation and attention in one kernel (see ``attn_decode_prep``)."""
     max_pages = (ctx.max_len + 63) // 64
     if OPTIONS.attn_tma and tma_decode_supported(qkv.dtype, nh, nkv, hd):
         return attn_decode_tma(qkv, k_pages, v_pages, ctx.seq_lens, block_table, nh, nkv, hd, scale, window,
                                pick_splits(ctx.n_seqs, nkv, max_pages, qkv.device), prep=True, wq=wq, wk=wk,
-                               inv_freq=inv_freq, eps=eps, write_cache=write_cache)
+                               inv_freq=inv_freq, eps=eps, write_cache=write_cache, sinks=sinks)
     return attn_decode_prep(qkv, k_pages, v_pages, ctx.seq_lens, block_table, nh, nkv, hd, scale, window,
-                            pick_splits(ctx.n_seqs, nkv, max_pages, qkv.device), wq, wk, inv_freq, eps, write_cache)
+                            pick_splits(ctx.n_seqs, nkv, max_pages, qkv.device), wq, wk, inv_freq, eps, write_cache,
+                            sinks=sinks)
 
 
 def _query_tiles(ctx, rows: int, device):
@@ -323,8 +350,7 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, ctx
     """Causal attention of the step's packed queries over the cache (which already holds
     this step's keys and values).  The options are those of ``attn_generic``: value heads of
     another size, capped scores, a sink per head, chunks of positions, a wider output."""
-    plain = (vd in (None, hd) and softcap is None and sinks is None and chunk is None and out is None
-             and out_scale == 1.0)
+    plain = vd in (None, hd) and softcap is None and chunk is None and out is None and out_scale == 1.0
     if not plain:
         # the mma.sync kernels take the options when keys and values have one of their head sizes; a long window without
         # chunks would want the single-token form's splits, which the options' form does not have
@@ -345,15 +371,15 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, ctx
             max_pages = (ctx.max_len + 63) // 64
             if OPTIONS.attn_tma and tma_decode_supported(q.dtype, nh, nkv, hd):
                 return attn_decode_tma(q, k_pages, v_pages, ctx.seq_lens, block_table, nh, nkv, hd, scale, window,
-                                       pick_splits(ctx.n_seqs, nkv, max_pages, q.device))
+                                       pick_splits(ctx.n_seqs, nkv, max_pages, q.device), sinks=sinks)
             return attn_decode(q, k_pages, v_pages, ctx.seq_lens, block_table, nh, nkv, hd, scale, window,
-                               pick_splits(ctx.n_seqs, nkv, max_pages, q.device))
+                               pick_splits(ctx.n_seqs, nkv, max_pages, q.device), sinks=sinks)
         if ctx.host is not None:
             # prompt steps: tcgen05 kernel (128-row tiles) for head size 128, else the mma.sync kernel (64-row tiles)
             tc = tc_prefill_supported(q.dtype, nh, nkv, hd)
             tiles = _query_tiles(ctx, TC_TILE_ROWS if tc else 64, q.device)
             kernel = attn_prefill_tc if tc else attn_prefill
             return kernel(q, k_pages, v_pages, tiles[0], tiles[1], ctx.cu_seqlens, ctx.seq_past, ctx.seq_lens,
-                          block_table, nh, nkv, hd, scale, window)
+                          block_table, nh, nkv, hd, scale, window, sinks=sinks)
     return attn_generic(q, k_pages, v_pages, ctx.positions, ctx.seq_of_token, block_table, nh, nkv, hd,
-                        scale, window)
+                        scale, window, sinks=sinks)

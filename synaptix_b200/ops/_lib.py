@@ -57,6 +57,21 @@ def stream() -> ctypes.c_void_p:
     return ctypes.c_void_p(torch.cuda.current_stream().cuda_stream)
 
 
+def check_bias(bias: Optional[torch.Tensor], n: int) -> None:
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != n):
+        raise KernelError(f"a product's bias is float32 with one element per output ({n})")
+
+
+def check_resid_tanh(x, w, bias, h, gain, shift) -> None:
+    """What the products that end in the residual stream and its norm without statistics have in common."""
+    (M, K), (N, K2) = x.shape, w.shape
+    if K != K2 or tuple(h.shape) != (M, N) or h.dtype != torch.float32:
+        raise KernelError("the residual stream must be contiguous float32 [M, N]")
+    check_bias(bias, N)
+    if any(t.dtype != torch.float32 or t.numel() != N for t in (gain, shift)):
+        raise KernelError("gain and shift of the norm are float32 [N]")
+
+
 _COUNTER = [None]
 
 

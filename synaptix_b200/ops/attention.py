@@ -30,6 +30,11 @@ def pick_splits(n_seqs: int, nkv: int, max_pages: int, device) -> int:
     return max(1, -(-max_pages // per))
 
 
+def _check_sinks(sinks: Optional[torch.Tensor], nh: int) -> None:
+    if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != nh):
+        raise KernelError("attention: sinks are float32, one per query head")
+
+
 _COUNTERS = {}
 _MAX_COUNTERS = 1 << 16
 
@@ -45,15 +50,18 @@ def _counters(device) -> torch.Tensor:
 def attn_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, seq_lens: torch.Tensor,
                 block_table: torch.Tensor, nh: int, nkv: int, hd: int, scale: float, window: Optional[int],
                 n_splits: int, out: Optional[torch.Tensor] = None,
-                scratch: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, fused_merge: bool = False) -> torch.Tensor:
+                scratch: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, fused_merge: bool = False,
+                sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """One query token per sequence (row ``s`` of ``q`` belongs to sequence ``s``) against the
     sequence's ``seq_lens[s]`` cached keys (its own included).  ``n_splits > 1`` splits the
     pages of every sequence over blocks; partial results go through float32 scratch
     (``scratch = (part_o [S*nh*n_splits*hd], part_ml [S*nh*n_splits*2])``, allocated if absent).
     With ``fused_merge`` the block of a (sequence, kv head) that finishes last merges the splits
     inside the kernel; otherwise (the default: it measured faster, 3.96 against 4.08 ms for a
-    batch-8 step of the 4B shape) a second kernel does."""
-    require_cuda(q, k_pages, v_pages, seq_lens, block_table, out)
+    batch-8 step of the 4B shape) a second kernel does.  ``sinks`` float32 ``[nh]``: ``exp(sink)`` joins the denominator of
+    the head's softmax (not with ``fused_merge``)."""
+    require_cuda(q, k_pages, v_pages, seq_lens, block_table, out, sinks)
+    _check_sinks(sinks, nh)
     S = q.shape[0]
     if not fast_supported(q.dtype, nh, nkv, hd) or k_pages.dtype != q.dtype:
         raise KernelError("attn_decode: bfloat16, head size 32/64/128 and at most 16 query heads per kv head")
@@ -68,7 +76,7 @@ def attn_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, s
             part_o, part_ml = scratch
             if part_o.numel() < S * nh * n_splits * hd or part_ml.numel() < S * nh * n_splits * 2:
                 raise KernelError("attn_decode: scratch is too small")
-    if fused_merge and n_splits > 1 and S * nkv <= _MAX_COUNTERS and n_splits <= 512:
+    if fused_merge and sinks is None and n_splits > 1 and S * nkv <= _MAX_COUNTERS and n_splits <= 512:
         check(fn("attention", "sx_attn_decode_fused")(
             ptr(q), ptr(k_pages), ptr(v_pages), ptr(out), ptr(part_o), ptr(part_ml), ptr(_counters(q.device)),
             ptr(seq_lens), ptr(block_table), c_int(block_table.shape[1]), c_int(S), c_int(nh), c_int(nkv), c_int(hd),
@@ -77,7 +85,7 @@ def attn_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, s
     check(fn("attention", "sx_attn_decode")(
         ptr(q), ptr(k_pages), ptr(v_pages), ptr(out), ptr(part_o), ptr(part_ml), ptr(seq_lens), ptr(block_table),
         c_int(block_table.shape[1]), c_int(S), c_int(nh), c_int(nkv), c_int(hd), c_float(scale),
-        c_int(0 if window is None else int(window)), c_int(n_splits), stream()), "attn_decode",
+        c_int(0 if window is None else int(window)), c_int(n_splits), ptr(sinks), stream()), "attn_decode",
         launches=2 if n_splits > 1 else 1)
     return out
 
@@ -86,13 +94,15 @@ def attn_decode_prep(qkv: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Te
                      block_table: torch.Tensor, nh: int, nkv: int, hd: int, scale: float, window: Optional[int],
                      n_splits: int, wq: Optional[torch.Tensor], wk: Optional[torch.Tensor],
                      inv_freq: Optional[torch.Tensor], eps: float, write_cache: bool,
-                     out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     out: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``attn_decode`` straight from the step's fused projection ``qkv [S, (nh + 2 nkv) hd]``: the kernel
     normalises and rotates the query heads and the new key itself (what ``qkv_prepare`` does), writes the new key
-    and value into the cache (``write_cache``) and attends.  The rotation is of the whole head or none."""
-    require_cuda(qkv, k_pages, v_pages, seq_lens, block_table, out, wq, wk, inv_freq)
+    and value into the cache (``write_cache``) and attends.  The rotation is of the whole head or none.  Without
+    ``write_cache`` the projection may hold the query heads alone, ``[S, nh hd]``.  ``sinks``: see ``attn_decode``."""
+    require_cuda(qkv, k_pages, v_pages, seq_lens, block_table, out, wq, wk, inv_freq, sinks)
+    _check_sinks(sinks, nh)
     S = qkv.shape[0]
-    if not fast_supported(qkv.dtype, nh, nkv, hd) or k_pages.dtype != qkv.dtype or qkv.shape[1] != (nh + 2 * nkv) * hd:
+    if not fast_supported(qkv.dtype, nh, nkv, hd) or k_pages.dtype != qkv.dtype or not _projection_width_ok(qkv, nh, nkv, hd, write_cache):
         raise KernelError("attn_decode_prep: bfloat16 [S, (nh + 2 nkv) hd], head size 32/64/128, at most 16 query heads per kv head")
     if inv_freq is not None and inv_freq.numel() != hd // 2:
         raise KernelError("attn_decode_prep: the rotation must cover the whole head")
@@ -106,9 +116,13 @@ def attn_decode_prep(qkv: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Te
         ptr(qkv), ptr(k_pages), ptr(v_pages), ptr(out), ptr(part_o), ptr(part_ml), ptr(wq), ptr(wk), ptr(inv_freq),
         c_float(eps), c_int(1 if write_cache else 0), c_longlong(k_pages.shape[0]), ptr(seq_lens), ptr(block_table),
         c_int(block_table.shape[1]), c_int(S), c_int(nh), c_int(nkv), c_int(hd), c_float(scale),
-        c_int(0 if window is None else int(window)), c_int(n_splits), stream()), "attn_decode_prep",
+        c_int(0 if window is None else int(window)), c_int(n_splits), ptr(sinks), c_int(qkv.shape[1]), stream()), "attn_decode_prep",
         launches=2 if n_splits > 1 else 1)
     return out
+
+
+def _projection_width_ok(qkv: torch.Tensor, nh: int, nkv: int, hd: int, write_cache: bool) -> bool:
+    return qkv.shape[1] == (nh + 2 * nkv) * hd or (not write_cache and qkv.shape[1] == nh * hd)
 
 
 TMA_HEAD_DIMS = (64, 128)
@@ -135,7 +149,7 @@ def attn_decode_tma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
                     n_splits: int, *, prep: bool = False, wq: Optional[torch.Tensor] = None,
                     wk: Optional[torch.Tensor] = None, inv_freq: Optional[torch.Tensor] = None, eps: float = 0.0,
                     write_cache: bool = True, out: Optional[torch.Tensor] = None,
-                    cluster: Optional[bool] = None) -> torch.Tensor:
+                    cluster: Optional[bool] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Single-token attention with pages brought by TMA and a warp per page (``csrc/attn_decode.cu``).
 
     ``q`` is ``[S, nh * hd]`` prepared queries against a cache that already holds the step's keys and values;
@@ -144,12 +158,14 @@ def attn_decode_tma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
     key itself and, with ``write_cache``, stores the new key and value.  ``n_splits`` blocks share a
     sequence's pages; with 2, 4, 8 or 16 of them and ``cluster`` they merge their partial results among
     themselves as a thread-block cluster, otherwise through scratch memory and a second kernel.  ``cluster=None``
-    decides by ``use_cluster``."""
-    require_cuda(q, k_pages, v_pages, seq_lens, block_table, out, wq, wk, inv_freq)
+    decides by ``use_cluster``.  Without ``write_cache`` the projection may hold the query heads alone, ``[S, nh hd]``.
+    ``sinks`` float32 ``[nh]``: ``exp(sink)`` joins the denominator of the head's softmax."""
+    require_cuda(q, k_pages, v_pages, seq_lens, block_table, out, wq, wk, inv_freq, sinks)
+    _check_sinks(sinks, nh)
     S = q.shape[0]
     if not tma_decode_supported(q.dtype, nh, nkv, hd) or k_pages.dtype != q.dtype:
         raise KernelError("attn_decode_tma: bfloat16, head size 64 or 128 and at most 16 query heads per kv head")
-    if q.shape[1] != ((nh + 2 * nkv) * hd if prep else nh * hd):
+    if not (_projection_width_ok(q, nh, nkv, hd, write_cache) if prep else q.shape[1] == nh * hd):
         raise KernelError("attn_decode_tma: q has the wrong width")
     if inv_freq is not None and inv_freq.numel() != hd // 2:
         raise KernelError("attn_decode_tma: the rotation must cover the whole head")
@@ -165,7 +181,8 @@ def attn_decode_tma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
         ptr(q), ptr(k_pages), ptr(v_pages), ptr(out), ptr(part_o), ptr(part_ml), c_int(1 if prep else 0), ptr(wq),
         ptr(wk), ptr(inv_freq), c_float(eps), c_int(1 if write_cache else 0), c_longlong(k_pages.shape[0]),
         ptr(seq_lens), ptr(block_table), c_int(block_table.shape[1]), c_int(S), c_int(nh), c_int(nkv), c_int(hd),
-        c_float(scale), c_int(0 if window is None else int(window)), c_int(n_splits), stream()), "attn_decode_tma",
+        c_float(scale), c_int(0 if window is None else int(window)), c_int(n_splits), ptr(sinks), c_int(q.shape[1]),
+        stream()), "attn_decode_tma",
         launches=2 if n_splits > 1 and not clustered else 1)
     return out
 
@@ -193,10 +210,12 @@ def query_tiles(cu_seqlens: Sequence[int], rows: int = 64):
 def attn_prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, tile_seq: torch.Tensor,
                  tile_q0: torch.Tensor, cu_seqlens: torch.Tensor, seq_past: torch.Tensor, seq_lens: torch.Tensor,
                  block_table: torch.Tensor, nh: int, nkv: int, hd: int, scale: float, window: Optional[int],
-                 out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 out: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Packed query tokens of sequences with unequal lengths against the cache (which already
-    holds this step's keys); ``tile_seq``/``tile_q0`` list the 64-row query tiles."""
-    require_cuda(q, k_pages, v_pages, tile_seq, tile_q0, cu_seqlens, seq_past, seq_lens, block_table, out)
+    holds this step's keys); ``tile_seq``/``tile_q0`` list the 64-row query tiles.  ``sinks`` float32 ``[nh]``: ``exp(sink)`` joins
+    the denominator of the head's softmax."""
+    require_cuda(q, k_pages, v_pages, tile_seq, tile_q0, cu_seqlens, seq_past, seq_lens, block_table, out, sinks)
+    _check_sinks(sinks, nh)
     T = q.shape[0]
     if not (q.dtype == torch.bfloat16 and hd in FAST_HEAD_DIMS and nh % nkv == 0):
         raise KernelError("attn_prefill: bfloat16 and head size 32/64/128")
@@ -205,7 +224,7 @@ def attn_prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, 
     check(fn("attention", "sx_attn_prefill")(
         ptr(q), ptr(k_pages), ptr(v_pages), ptr(out), ptr(tile_seq), ptr(tile_q0), c_int(tile_seq.numel()),
         ptr(cu_seqlens), ptr(seq_past), ptr(seq_lens), ptr(block_table), c_int(block_table.shape[1]), c_int(nh),
-        c_int(nkv), c_int(hd), c_float(scale), c_int(0 if window is None else int(window)), stream()), "attn_prefill")
+        c_int(nkv), c_int(hd), c_float(scale), c_int(0 if window is None else int(window)), ptr(sinks), stream()), "attn_prefill")
     return out
 
 
@@ -278,10 +297,11 @@ def tc_prefill_supported(dtype, nh: int, nkv: int, hd: int) -> bool:
 def attn_prefill_tc(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, tile_seq: torch.Tensor,
                     tile_q0: torch.Tensor, cu_seqlens: torch.Tensor, seq_past: torch.Tensor, seq_lens: torch.Tensor,
                     block_table: torch.Tensor, nh: int, nkv: int, hd: int, scale: float, window: Optional[int],
-                    out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    out: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``attn_prefill`` on the tcgen05 tensor cores (``csrc/attn_tc.cu``); ``tile_seq``/``tile_q0`` list
     128-row query tiles."""
-    require_cuda(q, k_pages, v_pages, tile_seq, tile_q0, cu_seqlens, seq_past, seq_lens, block_table, out)
+    require_cuda(q, k_pages, v_pages, tile_seq, tile_q0, cu_seqlens, seq_past, seq_lens, block_table, out, sinks)
+    _check_sinks(sinks, nh)
     T = q.shape[0]
     if not tc_prefill_supported(q.dtype, nh, nkv, hd) or k_pages.dtype != q.dtype:
         raise KernelError("attn_prefill_tc: bfloat16 and head size 128")
@@ -291,7 +311,7 @@ def attn_prefill_tc(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
         ptr(q), ptr(k_pages), ptr(v_pages), ptr(out), c_longlong(T), c_longlong(k_pages.shape[0]), ptr(tile_seq),
         ptr(tile_q0), c_int(tile_seq.numel()), ptr(cu_seqlens), ptr(seq_past), ptr(seq_lens), ptr(block_table),
         c_int(block_table.shape[1]), c_int(nh), c_int(nkv), c_int(hd), c_float(scale),
-        c_int(0 if window is None else int(window)), stream()), "attn_prefill_tc")
+        c_int(0 if window is None else int(window)), ptr(sinks), stream()), "attn_prefill_tc")
     return out
 
 

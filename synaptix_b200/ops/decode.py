@@ -5,7 +5,7 @@ from typing import Optional
 
 import torch
 
-from ._lib import KernelError, c_float, c_int, check, fn, ptr, require_cuda, stream, use_gate
+from ._lib import KernelError, c_float, c_int, check, check_bias, check_resid_tanh, fn, ptr, require_cuda, stream, use_gate
 
 _EPI = {None: 0, "f32": 1, "silu_mul": 2}
 MAX_ROWS = 16          # more rows go to the tcgen05 product, which takes every K this kernel takes
@@ -27,8 +27,9 @@ def skinny_gemm(x: Optional[torch.Tensor], w: torch.Tensor, *, epilogue: Optiona
                 ks: Optional[int] = None, out: Optional[torch.Tensor] = None,
                 norm_h: Optional[torch.Tensor] = None, norm_delta: Optional[torch.Tensor] = None,
                 norm_h_out: Optional[torch.Tensor] = None, norm_gain: Optional[torch.Tensor] = None,
-                norm_eps: float = 0.0) -> torch.Tensor:
-    """``x[M, K] @ w[N, K].T`` for ``M <= 16`` rows, reading ``w`` once (``ks``: 8 or 16 warps split K).
+                norm_eps: float = 0.0, bias: Optional[torch.Tensor] = None, cap: float = 0.0) -> torch.Tensor:
+    """``x[M, K] @ w[N, K].T`` for ``M <= 16`` rows, reading ``w`` once (``ks``: 8 or 16 warps split K).  ``bias``
+    (float32 ``[N]``) is added to the product; ``cap`` (with ``"f32"``): ``cap * tanh(. / cap)`` of the result.
 
     ``epilogue``: ``None`` -> bfloat16 ``[M, N]``; ``"f32"`` -> float32 ``[M, N]``;
     ``"silu_mul"`` -> ``w`` is ``[gate; up]`` stacked, result bfloat16 ``[M, N/2]``.
@@ -36,8 +37,9 @@ def skinny_gemm(x: Optional[torch.Tensor], w: torch.Tensor, *, epilogue: Optiona
     ``rmsnorm(norm_h + norm_delta) * norm_gain`` and ``norm_h + norm_delta`` is written to
     ``norm_h_out`` (which must not alias ``norm_h``); then ``M <= 2`` and ``x`` is ``None``.
     """
-    require_cuda(x, w, out, norm_h, norm_delta, norm_h_out, norm_gain)
+    require_cuda(x, w, out, norm_h, norm_delta, norm_h_out, norm_gain, bias)
     N, K = w.shape
+    check_bias(bias, N)
     M = (x if x is not None else norm_h).shape[0]
     if (x if x is not None else norm_h).shape[1] != K:
         raise KernelError("skinny_gemm: inner sizes differ")
@@ -58,7 +60,7 @@ def skinny_gemm(x: Optional[torch.Tensor], w: torch.Tensor, *, epilogue: Optiona
         use_gate("decode")
     check(fn("decode", "sx_skinny_gemm")(ptr(x), ptr(w), ptr(out), c_int(M), c_int(N), c_int(K), c_int(_EPI[epilogue]),
                                          c_int(ks), ptr(norm_h), ptr(norm_delta), ptr(norm_h_out), ptr(norm_gain),
-                                         c_float(norm_eps), stream()), "skinny_gemm")
+                                         c_float(norm_eps), ptr(bias), c_float(cap), stream()), "skinny_gemm")
     return out
 
 
@@ -108,6 +110,20 @@ def skinny_gemm_residual(x: torch.Tensor, w: torch.Tensor, h: torch.Tensor, gain
         ptr(x), ptr(w), ptr(out), c_int(M), c_int(N), c_int(K), c_int(3), c_int(ks), ptr(None), c_int(0),
         c_float(0.0), ptr(h), ptr(gain), ptr(ssq), stream()), "skinny_gemm_residual")
     return out, ssq
+
+
+def skinny_gemm_resid_tanh(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], h: torch.Tensor, alpha: float,
+                           gain: torch.Tensor, shift: torch.Tensor, *, ks: Optional[int] = None) -> torch.Tensor:
+    """``h += x @ w.T + bias`` in place (``h`` float32 ``[M, N]``); returns bfloat16 ``tanh(alpha h) * gain + shift``."""
+    require_cuda(x, w, bias, h, gain, shift)
+    N, K = w.shape
+    M = x.shape[0]
+    check_resid_tanh(x, w, bias, h, gain, shift)
+    out = torch.empty((M, N), dtype=torch.bfloat16, device=w.device)
+    check(fn("decode", "sx_skinny_gemm_resid_tanh")(
+        ptr(x), ptr(w), ptr(out), c_int(M), c_int(N), c_int(K), c_int(ks or pick_ks((N + 15) // 16, K)), ptr(h), ptr(bias),
+        c_float(alpha), ptr(gain), ptr(shift), stream()), "skinny_gemm_resid_tanh")
+    return out
 
 
 _SM_COUNT = {}

@@ -6,11 +6,11 @@ from typing import Optional
 
 import torch
 
-from ._lib import KernelError, c_int, check, fn, ptr, require_cuda, stream, use_gate
+from ._lib import KernelError, c_float, c_int, check, check_bias, check_resid_tanh, fn, ptr, require_cuda, stream, use_gate
 from .decode import sm_count
 from .options import OPTIONS
 
-_EPI = {None: 0, "f32": 1, "silu_mul": 2}
+_EPI = {None: 0, "f32": 1, "silu_mul": 2, "resid_tanh": 5}
 
 
 def tc_supported(M: int, N: int, K: int, x_dtype, w_dtype) -> bool:
@@ -89,7 +89,7 @@ def plan_stream(M: int, N: int, K: int, epilogue: Optional[str] = None):
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, *, epilogue: Optional[str] = None,
             out: Optional[torch.Tensor] = None, splits: Optional[int] = None,
-            cut: Optional[bool] = None) -> torch.Tensor:
+            cut: Optional[bool] = None, bias: Optional[torch.Tensor] = None, cap: float = 0.0) -> torch.Tensor:
     """``x[M, K] @ w[N, K].T`` on the tcgen05 tensor cores, 32-bit accumulation in tensor memory.
 
     Default: the persistent kernel, which cuts tiles over K where whole tiles would leave SMs idle (see
@@ -99,17 +99,33 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, *, epilogue: Optional[str] = None,
     ``splits=1`` for whole tiles (or cut ones) in any case.
 
     ``epilogue``: ``None`` -> bfloat16 ``[M, N]``; ``"f32"`` -> float32 ``[M, N]``; ``"silu_mul"`` ->
-    ``w`` is ``[gate; up]`` stacked and the result is bfloat16 ``[M, N/2]``.  Needs ``K % 8 == 0``.
+    ``w`` is ``[gate; up]`` stacked and the result is bfloat16 ``[M, N/2]``.  Needs ``K % 8 == 0``.  ``bias`` (float32
+    ``[N]``) is added to the product; ``cap`` (with ``"f32"``): ``cap * tanh(. / cap)`` of the result.
     """
-    require_cuda(x, w, out)
+    if epilogue not in (None, "f32", "silu_mul"):
+        raise KernelError(f"gemm_tc: unknown epilogue {epilogue!r}")
+    check_bias(bias, w.shape[0])
+    return _gemm_tc(x, w, epilogue, out, splits, cut, bias, cap)
+
+
+def gemm_tc_resid_tanh(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], h: torch.Tensor, alpha: float,
+                       gain: torch.Tensor, shift: torch.Tensor, *, splits: Optional[int] = None,
+                       cut: Optional[bool] = None) -> torch.Tensor:
+    """``h += x @ w.T + bias`` in place (``h`` float32 ``[M, N]``); returns bfloat16 ``tanh(alpha h) * gain + shift``, in the
+    product's epilogue."""
+    require_cuda(h, gain, shift)
+    check_resid_tanh(x, w, bias, h, gain, shift)
+    return _gemm_tc(x, w, "resid_tanh", None, splits, cut, bias, 0.0, h, alpha, gain, shift)
+
+
+def _gemm_tc(x, w, epilogue, out, splits, cut, bias, cap, h=None, alpha=0.0, gain=None, shift=None) -> torch.Tensor:
+    require_cuda(x, w, out, bias)
     M, K = x.shape
     N, K2 = w.shape
     if K != K2:
         raise KernelError("gemm_tc: inner sizes differ")
     if not tc_supported(M, N, K, x.dtype, w.dtype):
         raise KernelError("gemm_tc: bfloat16 operands and K a multiple of 8")
-    if epilogue not in _EPI:
-        raise KernelError(f"gemm_tc: unknown epilogue {epilogue!r}")
     n_out = N // 2 if epilogue == "silu_mul" else N
     if epilogue == "silu_mul":
         use_gate("gemm_tc")
@@ -138,7 +154,8 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, *, epilogue: Optional[str] = None,
             counts = _counts(x.device)
     check(fn("gemm_tc", "sx_gemm_tc")(ptr(x), ptr(w), ptr(out), c_int(M), c_int(N), c_int(K), c_int(_EPI[epilogue]),
                                       c_int(splits), ptr(ws), ctypes.c_ulonglong(0 if ws is None else ws.numel()),
-                                      ptr(counts), stream()), "gemm_tc", launches=2 if splits > 1 else 1)
+                                      ptr(counts), ptr(bias), c_float(cap), ptr(h), c_float(alpha), ptr(gain), ptr(shift),
+                                      stream()), "gemm_tc", launches=2 if splits > 1 else 1)
     return out
 
 
@@ -155,15 +172,18 @@ def qkv_epilogue_supported(M: int, nh: int, nkv: int, hd: int, K: int, x_dtype, 
 def gemm_tc_qkv(x: torch.Tensor, w: torch.Tensor, q_out: torch.Tensor, k_pages: Optional[torch.Tensor],
                 v_pages: Optional[torch.Tensor], wq: Optional[torch.Tensor], wk: Optional[torch.Tensor],
                 cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], eps: float, positions: torch.Tensor,
-                seq_of_token: torch.Tensor, block_table: torch.Tensor, nh: int, nkv: int) -> None:
+                seq_of_token: torch.Tensor, block_table: torch.Tensor, nh: int, nkv: int,
+                bias: Optional[torch.Tensor] = None) -> None:
     """``x @ w.T`` for the stacked q/k/v matrix with heads of 128, and what ``qkv_prepare`` does to the result, in
     the product's epilogue: per-head RMSNorm of q and k (gains ``wq`` / ``wk``, skipped when ``None``), rotate-half
     rotation by the angles whose cosines and sines are ``cos`` / ``sin [M, 64]`` (skipped when ``None``), q to
-    ``q_out [M, nh * 128]``, k and v into the pages (skipped when ``None``)."""
-    require_cuda(x, w, q_out, k_pages, v_pages, wq, wk, cos, sin, positions, seq_of_token, block_table)
+    ``q_out [M, nh * 128]``, k and v into the pages (skipped when ``None``).  ``w`` may hold the ``nh`` query heads alone;
+    ``bias`` (float32, one element per row of ``w``) is added to the product."""
+    require_cuda(x, w, q_out, k_pages, v_pages, wq, wk, cos, sin, positions, seq_of_token, block_table, bias)
     M, K = x.shape
     N = w.shape[0]
-    if w.shape[1] != K or N != (nh + 2 * nkv) * QKV_HEAD_DIM or not qkv_epilogue_supported(M, nh, nkv, QKV_HEAD_DIM, K, x.dtype, w.dtype):
+    check_bias(bias, N)
+    if w.shape[1] != K or N not in ((nh + 2 * nkv) * QKV_HEAD_DIM, nh * QKV_HEAD_DIM) or not qkv_epilogue_supported(M, nh, nkv if N != nh * QKV_HEAD_DIM else 0, QKV_HEAD_DIM, K, x.dtype, w.dtype):
         raise KernelError("gemm_tc_qkv: bfloat16, heads of 128, an even number of heads, K a multiple of 8")
     if q_out.dtype != torch.bfloat16 or tuple(q_out.shape) != (M, nh * QKV_HEAD_DIM):
         raise KernelError("gemm_tc_qkv: q_out must be bfloat16 [M, nh * 128]")
@@ -183,7 +203,7 @@ def gemm_tc_qkv(x: torch.Tensor, w: torch.Tensor, q_out: torch.Tensor, k_pages: 
         if t.dtype != torch.int32:
             raise KernelError("gemm_tc_qkv: index tensors are int32")
     check(fn("gemm_tc", "sx_gemm_tc_qkv")(
-        ptr(x), ptr(w), c_int(M), c_int(N), c_int(K), ptr(q_out), ptr(k_pages), ptr(v_pages), ptr(wq), ptr(wk), ptr(cos),
+        ptr(x), ptr(w), ptr(bias), c_int(M), c_int(N), c_int(K), ptr(q_out), ptr(k_pages), ptr(v_pages), ptr(wq), ptr(wk), ptr(cos),
         ptr(sin), ptr(positions), ptr(seq_of_token), ptr(block_table), c_int(block_table.shape[1]), c_int(nh), c_int(nkv),
         c_int(n_pages), ctypes.c_float(eps), stream()), "gemm_tc_qkv")
 

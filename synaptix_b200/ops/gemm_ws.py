@@ -6,9 +6,9 @@ from typing import Optional, Tuple
 
 import torch
 
-from ._lib import KernelError, c_float, c_int, check, fn, ptr, require_cuda, stream, use_gate
+from ._lib import KernelError, c_float, c_int, check, check_bias, check_resid_tanh, fn, ptr, require_cuda, stream, use_gate
 
-_EPI = {None: 0, "f32": 1, "silu_mul": 2, "residual": 3}
+_EPI = {None: 0, "f32": 1, "silu_mul": 2, "residual": 3, "resid_tanh": 4}
 MAX_ROWS = 256
 
 
@@ -30,16 +30,18 @@ def plan_ws(M: int, N: int, K: int, epilogue: Optional[str] = None) -> Tuple[int
 
 def gemm_ws(x: torch.Tensor, w: torch.Tensor, *, epilogue: Optional[str] = None, ssq: Optional[torch.Tensor] = None,
             eps: float = 0.0, splits: Optional[int] = None, stages: Optional[int] = None,
-            out: Optional[torch.Tensor] = None) -> torch.Tensor:
+            out: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None, cap: float = 0.0) -> torch.Tensor:
     """``x[M, K] @ w[N, K].T`` for ``M <= 256`` rows with ``w`` as the tensor cores' M side, read once from HBM;
     K is shared by the ``splits`` (1, 2, 4, 8) blocks of a cluster, which add up through their shared memory.
 
     ``epilogue``: ``None`` -> bfloat16 ``[M, N]``; ``"f32"`` -> float32; ``"silu_mul"`` -> ``w`` is ``[gate; up]``
     stacked, result bfloat16 ``[M, N/2]``.  With ``ssq`` (float32 ``[M, n]``) row ``m`` of the product is multiplied
-    by ``rsqrt(sum(ssq[m]) / K + eps)`` before the epilogue: rows of ``x`` that lack their RMSNorm factor."""
-    require_cuda(x, w, ssq, out)
+    by ``rsqrt(sum(ssq[m]) / K + eps)`` before the epilogue: rows of ``x`` that lack their RMSNorm factor.
+    ``bias`` (float32 ``[N]``) is added to the product; ``cap`` (with ``"f32"``): ``cap * tanh(. / cap)`` of the result."""
+    require_cuda(x, w, ssq, out, bias)
     M, K = x.shape
     N = w.shape[0]
+    check_bias(bias, N)
     if w.shape[1] != K:
         raise KernelError("gemm_ws: inner sizes differ")
     if epilogue not in (None, "f32", "silu_mul"):
@@ -55,7 +57,7 @@ def gemm_ws(x: torch.Tensor, w: torch.Tensor, *, epilogue: Optional[str] = None,
         use_gate("gemm_ws")
     check(fn("gemm_ws", "sx_gemm_ws")(ptr(x), ptr(w), ptr(out), c_int(M), c_int(N), c_int(K), c_int(_EPI[epilogue]),
                                       c_int(splits or 0), c_int(stages or 0), ptr(ssq), c_int(0 if ssq is None else ssq.shape[1]),
-                                      c_float(eps), ptr(None), ptr(None), ptr(None), stream()), "gemm_ws")
+                                      c_float(eps), ptr(None), ptr(None), ptr(None), ptr(bias), c_float(cap), c_float(0.0), ptr(None), stream()), "gemm_ws")
     return out
 
 
@@ -83,9 +85,26 @@ def gemm_ws_residual(x: torch.Tensor, w: torch.Tensor, h: torch.Tensor, gain: to
     out = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
     ssq = torch.empty((M, tiles * splits), dtype=torch.float32, device=x.device)
     check(fn("gemm_ws", "sx_gemm_ws")(ptr(x), ptr(w), ptr(out), c_int(M), c_int(N), c_int(K), c_int(3), c_int(splits),
-                                      c_int(stages or 0), ptr(None), c_int(0), c_float(0.0), ptr(h), ptr(gain), ptr(ssq), stream()),
-          "gemm_ws_residual")
+                                      c_int(stages or 0), ptr(None), c_int(0), c_float(0.0), ptr(h), ptr(gain), ptr(ssq), ptr(None), c_float(0.0),
+                                      c_float(0.0), ptr(None), stream()), "gemm_ws_residual")
     return out, ssq
+
+
+def gemm_ws_resid_tanh(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], h: torch.Tensor, alpha: float,
+                       gain: torch.Tensor, shift: torch.Tensor, *, splits: Optional[int] = None,
+                       stages: Optional[int] = None) -> torch.Tensor:
+    """``h += x @ w.T + bias`` in place (``h`` float32 ``[M, N]``); returns bfloat16 ``tanh(alpha h) * gain + shift``."""
+    require_cuda(x, w, bias, h, gain, shift)
+    M, K = x.shape
+    N = w.shape[0]
+    check_resid_tanh(x, w, bias, h, gain, shift)
+    if not ws_supported(M, N, K, x.dtype, w.dtype):
+        raise KernelError("gemm_ws_resid_tanh: bfloat16 operands, at most 256 rows and K a multiple of 8")
+    out = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
+    check(fn("gemm_ws", "sx_gemm_ws")(ptr(x), ptr(w), ptr(out), c_int(M), c_int(N), c_int(K), c_int(_EPI["resid_tanh"]),
+                                      c_int(splits or 0), c_int(stages or 0), ptr(None), c_int(0), c_float(0.0), ptr(h), ptr(gain),
+                                      ptr(None), ptr(bias), c_float(0.0), c_float(alpha), ptr(shift), stream()), "gemm_ws_resid_tanh")
+    return out
 
 
 def gemm_ws_status(reset: bool = False) -> int:

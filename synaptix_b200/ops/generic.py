@@ -5,7 +5,7 @@ from typing import Optional
 
 import torch
 
-from ._lib import (KernelError, c_float, c_int, c_longlong, check, dt_code, fn, ptr, require_cuda,
+from ._lib import (KernelError, c_float, c_int, c_longlong, check, check_bias, dt_code, fn, ptr, require_cuda,
                    stream)
 
 
@@ -67,11 +67,13 @@ def residual_add(h: torch.Tensor, delta: torch.Tensor) -> None:
 
 
 def gemm_generic(a: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
-                 out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """``a[M, K] @ w[N, K].T`` with 32-bit accumulation on CUDA cores (no tensor cores)."""
-    require_cuda(a, w, out)
+                 out: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None, cap: float = 0.0) -> torch.Tensor:
+    """``a[M, K] @ w[N, K].T`` (``+ bias``, float32 ``[N]``; then ``cap * tanh(. / cap)`` if ``cap > 0``) with 32-bit
+    accumulation on CUDA cores (no tensor cores)."""
+    require_cuda(a, w, out, bias)
     M, K = a.shape
     N, K2 = w.shape
+    check_bias(bias, N)
     if K != K2:
         raise KernelError(f"gemm: inner sizes differ ({K} and {K2})")
     if out_dtype is None:
@@ -80,7 +82,7 @@ def gemm_generic(a: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dty
         out = torch.empty((M, N), dtype=out_dtype, device=a.device)
     check(fn("generic", "sx_gemm_generic")(ptr(a), c_int(dt_code(a.dtype)), ptr(w), c_int(dt_code(w.dtype)),
                                            ptr(out), c_int(dt_code(out.dtype)), c_int(M), c_int(N), c_int(K),
-                                           stream()), "gemm_generic")
+                                           ptr(bias), c_float(cap), stream()), "gemm_generic")
     return out
 
 

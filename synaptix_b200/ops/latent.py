@@ -64,11 +64,17 @@ class WeightedLatents:
     def __init__(self, parts, ml, splits):
         self.parts, self.ml, self.splits = parts, ml, splits
 
-    def merged(self) -> torch.Tensor:
+    def merged(self, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
         """float32 ``[T, heads, kv_rank]`` (for tests: torch arithmetic)."""
         m, l = self.ml[..., 0], self.ml[..., 1]
-        w = torch.exp(m - m.max(dim=-1, keepdim=True).values)
-        return (self.parts * w[..., None]).sum(2) / (l * w).sum(-1, keepdim=True)
+        top = m.max(dim=-1, keepdim=True).values
+        if sinks is not None:
+            top = torch.maximum(top, sinks[None, :, None])
+        w = torch.exp(m - top)
+        total = (l * w).sum(-1, keepdim=True)
+        if sinks is not None:
+            total = total + torch.exp(sinks[None, :, None] - top)
+        return (self.parts * w[..., None]).sum(2) / total
 
 
 _SMS = {}
@@ -110,19 +116,25 @@ def latent_attention(qa: torch.Tensor, k_pages: torch.Tensor, ctx, block_table: 
 
 
 def latent_output(ol: WeightedLatents, wuv: torch.Tensor, heads: int, vdim: int, kv_rank: int, proj: torch.Tensor, col_gate: int,
-                  out_dtype: torch.dtype) -> torch.Tensor:
+                  out_dtype: torch.dtype, *, sinks: Optional[torch.Tensor] = None, gate_elements: bool = False) -> torch.Tensor:
     """``y[t, h * vdim + j] = sigmoid(proj[t, col_gate + h]) * sum_r wuv[h * vdim + j, r] * o[t, h, r]`` with ``o`` the
-    merged, divided weighted latents (no gate if ``col_gate < 0``); ``[T, heads * vdim]`` in ``out_dtype``."""
-    require_cuda(ol.parts, ol.ml, wuv, proj)
+    merged, divided weighted latents (no gate if ``col_gate < 0``); ``[T, heads * vdim]`` in ``out_dtype``.
+    ``gate_elements``: a gate per output element, ``proj[t, col_gate + h * vdim + j]``.  ``sinks`` float32 ``[heads]``:
+    ``exp(sink)`` joins each head's denominator where the parts are merged."""
+    require_cuda(ol.parts, ol.ml, wuv, proj, sinks)
+    if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != heads):
+        raise KernelError("latent_output: sinks are float32, one per head")
     T = ol.parts.shape[0]
     if tuple(ol.parts.shape[1:]) != (heads, ol.splits, kv_rank) or tuple(wuv.shape) != (heads * vdim, kv_rank):
         raise KernelError("latent_output: sizes do not fit")
-    if wuv.dtype != out_dtype or proj.dtype != out_dtype or (col_gate >= 0 and col_gate + heads > proj.shape[1]):
+    if wuv.dtype != out_dtype or proj.dtype != out_dtype or (
+            col_gate >= 0 and col_gate + heads * (vdim if gate_elements else 1) > proj.shape[1]):
         raise KernelError("latent_output: dtypes or the gate's columns do not fit")
     y = torch.empty((T, heads * vdim), dtype=out_dtype, device=wuv.device)
     check(fn("latent", "sx_latent_output")(ptr(ol.parts), ptr(ol.ml), c_int(ol.splits), ptr(wuv), c_int(heads), c_int(vdim),
-                                           c_int(kv_rank), ptr(proj), c_int(proj.shape[1]), c_int(col_gate), ptr(y), c_int(T),
-                                           c_int(dt_code(out_dtype)), stream()), "latent_output")
+                                           c_int(kv_rank), ptr(proj), c_int(proj.shape[1]), c_int(col_gate),
+                                           c_int(1 if gate_elements else 0), ptr(sinks), ptr(y), c_int(T), c_int(dt_code(out_dtype)),
+                                           stream()), "latent_output")
     return y
 
 

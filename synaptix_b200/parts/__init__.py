@@ -8,10 +8,10 @@ from .embedding import BigramEmbedding, Embedding, OutputHead
 from .linear import JoinedLinear, Linear
 from .latent import LatentAttention
 from .mlp import CappedGLU, GeluGLU, MixtureOfExperts, SwiGLU
-from .norm import LayerNorm, RMSNorm
+from .norm import DynamicTanh, LayerNorm, RMSNorm
 from .parallel import NormedParallelMixers, ParallelMixers
 from .recurrent import MLSTM, MinGRU, Retention
-from .rope import FrequencyRamp, NoPosition, RotaryHalf, RotaryPairs, rotary_inv_freq
+from .rope import FrequencyBands, FrequencyRamp, NoPosition, RotaryHalf, RotaryPairs, rotary_inv_freq
 from .scored import ScoredAttention
 from .side import TokenSide
 
@@ -19,4 +19,5 @@ __all__ = ["Attention", "FeedForward", "Mixer", "Norm", "Part", "PendingLinear",
            "StepContext", "PreNormBlock", "ConvPreNormBlock", "TokenConv", "Embedding", "OutputHead", "Linear", "JoinedLinear",
            "SwiGLU", "CappedGLU", "RMSNorm", "ParallelMixers", "MinGRU", "Retention", "NoPosition", "RotaryHalf",
            "rotary_inv_freq", "ParallelBlock", "LatentAttention", "MixtureOfExperts", "MLSTM", "RotaryPairs", "FrequencyRamp", "ScoredAttention", "LayerNorm", "SandwichBlock", "TokenShift",
-           "PostNormBlock", "BigramEmbedding", "GeluGLU", "NormedParallelMixers", "ConvNormAttention", "ChannelDelta", "TokenSide"]
+           "PostNormBlock", "BigramEmbedding", "GeluGLU", "NormedParallelMixers", "ConvNormAttention", "ChannelDelta", "TokenSide",
+           "DynamicTanh", "FrequencyBands"]

@@ -121,17 +121,17 @@ class PendingNorm:
 
 
 class PendingLinear:
-    """A branch's last matrix product that has not run yet: ``x @ weight.T``.
+    """A branch's last matrix product that has not run yet: ``x @ weight.T`` (``+ bias``, float32, if there is one).
 
     A mixer or feed-forward that is asked to (``forward(..., defer_output=True)``; only parts with
     ``can_defer_output`` are asked) may return this instead of the product.  A norm that says
     ``takes_pending_product`` may then run the product so that it adds itself into the residual stream and
     prepares the norm (``ScaledRows``); anybody else calls ``materialize()`` and gets the plain tensor.
     """
-    __slots__ = ("x", "weight", "_y")
+    __slots__ = ("x", "weight", "bias", "_y")
 
-    def __init__(self, x, weight):
-        self.x, self.weight = x, weight
+    def __init__(self, x, weight, bias=None):
+        self.x, self.weight, self.bias = x, weight, bias
         self._y = None
 
     @property
@@ -141,7 +141,7 @@ class PendingLinear:
     def materialize(self) -> torch.Tensor:
         if self._y is None:
             from .. import ops
-            self._y = ops.linear(self.x, self.weight)
+            self._y = ops.linear(self.x, self.weight, bias=self.bias)
         return self._y
 
 

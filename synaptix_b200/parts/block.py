@@ -40,13 +40,16 @@ from .base import (FeedForward, Mixer, Norm, NormedDelta, NormedSum, Part, Pendi
 
 
 class PreNormBlock(Part):
+    """``norm2`` and ``ffn`` may both be ``None`` (a layer without a feed-forward)."""
     takes_pending_product = True   # forward's ``pending`` may be a PendingLinear
 
-    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Norm, ffn: FeedForward):
+    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Optional[Norm], ffn: Optional[FeedForward]):
+        if (norm2 is None) != (ffn is None):
+            raise ValueError("norm2 and ffn come together or not at all")
         self.norm1, self.mixer, self.norm2, self.ffn = norm1, mixer, norm2, ffn
 
     def children(self) -> List[Part]:
-        return [self.norm1, self.mixer, self.norm2, self.ffn]
+        return [p for p in (self.norm1, self.mixer, self.norm2, self.ffn) if p is not None]
 
     def cache_request(self):
         return self.mixer.cache_request()
@@ -58,12 +61,14 @@ class PreNormBlock(Part):
         if isinstance(pending, PendingLinear) and not self.norm1.takes_pending_product:
             pending = pending.materialize()
         x = self.norm1.add_forward(h, pending, lazy=self.mixer.accepts_lazy_input)
-        if self.mixer.can_defer_output and self.norm2.takes_pending_product:
+        if self.mixer.can_defer_output and (self.norm2 is None or self.norm2.takes_pending_product):
             a = self.mixer.forward(x, ctx, cache_view, write_cache, defer_output=True)
         else:
             a = self.mixer.forward(x, ctx, cache_view, write_cache)
         if isinstance(x, (PendingNorm, ScaledRows)):
             h = x.h_after()
+        if self.ffn is None:
+            return h, a
         y = self.norm2.add_forward(h, a, lazy=self.ffn.accepts_lazy_input)
         m = self.ffn.forward(y, ctx, defer_output=True) if self.ffn.can_defer_output else self.ffn.forward(y, ctx)
         if isinstance(y, (PendingNorm, ScaledRows)):

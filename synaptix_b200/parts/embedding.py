@@ -92,12 +92,16 @@ class BigramEmbedding(Embedding):
 
 class OutputHead(Part):
     """``tied`` is True, False, or None (= tied iff the weights hold no matrix of that name).  ``scale``: the logits
-    are multiplied by it (in 32-bit)."""
+    are multiplied by it (in 32-bit).  ``softcap``: they become ``softcap * tanh(logits / softcap)``, in 32-bit in the
+    product's epilogue (not together with a scale)."""
 
     def __init__(self, weight_name: str, vocab: int, width: int, tied: Optional[bool], embedding: Embedding,
-                 scale: float = 1.0):
+                 scale: float = 1.0, softcap: Optional[float] = None):
         self.weight_name, self.vocab, self.width = weight_name, vocab, width
         self.scale = float(scale)
+        self.softcap = float(softcap) if softcap else 0.0
+        if self.softcap and self.scale != 1.0:
+            raise ValueError("logits are either scaled or capped")
         self.tied = tied
         self.embedding = embedding
         self.linear = Linear(weight_name, width, vocab)
@@ -116,7 +120,7 @@ class OutputHead(Part):
 
     def forward(self, x) -> torch.Tensor:
         """``x``: the normalised rows, or a ``PendingNorm`` of them."""
-        logits = self.linear.forward(x, out_dtype=torch.float32)
+        logits = self.linear.forward(x, out_dtype=torch.float32, cap=self.softcap)
         if self.scale != 1.0:
             ops.scale_rows(logits, self.scale)
         return logits

@@ -35,11 +35,13 @@ class SwiGLU(FeedForward):
 
     NAMES = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}
 
-    def __init__(self, prefix: str, width: int, intermediate: int, names: Optional[Mapping[str, str]] = None):
+    def __init__(self, prefix: str, width: int, intermediate: int, names: Optional[Mapping[str, str]] = None,
+                 bias_suffix: Optional[str] = None):
+        """``bias_suffix``: all three projections have biases, named like them with the suffix added."""
         self.width, self.intermediate = width, intermediate
         n = dict(self.NAMES, **(names or {}))
-        self.gate_up = Linear([prefix + n["gate"], prefix + n["up"]], width, [intermediate, intermediate])
-        self.down = Linear(prefix + n["down"], intermediate, width)
+        self.gate_up = Linear([prefix + n["gate"], prefix + n["up"]], width, [intermediate, intermediate], bias_suffix=bias_suffix)
+        self.down = Linear(prefix + n["down"], intermediate, width, bias_suffix=bias_suffix)
 
     def children(self) -> List[Part]:
         return [self.gate_up, self.down]

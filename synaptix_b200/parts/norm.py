@@ -57,7 +57,7 @@ class RMSNorm(Norm):
             return ops.add_scaled_rmsnorm(h, delta.terms, [self.weight], self.eps, self._dtype, rows=rows)[0]
         if isinstance(delta, PendingLinear):
             N, K = delta.weight.shape
-            if (lazy and rows is None and N == self.width and h.dtype == torch.float32 and h.is_contiguous()
+            if (lazy and delta.bias is None and rows is None and N == self.width and h.dtype == torch.float32 and h.is_contiguous()
                     and delta.weight.dtype == self._dtype and delta.x.dtype == self._dtype
                     and ops.residual_product_fusable(h.shape[0], N, K, self._dtype)):
                 # the product adds itself into h and leaves the rows of this norm without their factor
@@ -109,3 +109,48 @@ class LayerNorm(Norm):
         y, h_after = ops.add_layernorm(h, delta, self.weight, self.bias, self.eps, self._dtype, rows=rows, shift=shift,
                                        state=state, ctx=ctx, in_place=in_place, **kw)
         return (y, h_after) if shift is not None else y
+
+
+class DynamicTanh(Norm):
+    """A norm without statistics of the row: ``tanh(alpha x) * w + b`` with a learned number ``alpha`` and vectors ``w`` and
+    ``b`` over the width, all in 32-bit (the layer of "Transformers without Normalization", Zhu, Chen, He, LeCun, Liu).
+    Tensors: ``weight_name``, and with ``.alpha`` and ``.b`` added the other two.
+
+    Every element stands on its own, so a branch's last product can add itself into the residual stream AND finish this norm
+    in its epilogue, whatever the number of rows: no norm kernel, no second pass, nothing left for the consumer."""
+    takes_pending_product = True
+
+    def __init__(self, weight_name: str, width: int, *, alpha_suffix: str = ".alpha", bias_suffix: str = ".b"):
+        self.weight_name, self.width = weight_name, width
+        self.alpha_name, self.bias_name = weight_name + alpha_suffix, weight_name + bias_suffix
+        self.alpha: float = 0.0
+        self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+        self._dtype = None
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        return {self.weight_name: TensorSpec((self.width,), "gain"), self.bias_name: TensorSpec((self.width,), "bias"),
+                self.alpha_name: TensorSpec((), "gain")}
+
+    def bind(self, tensors: Mapping[str, torch.Tensor], rt: Runtime) -> None:
+        self.weight = to_device_f32(tensors[self.weight_name], rt)
+        self.bias = to_device_f32(tensors[self.bias_name], rt)
+        self.alpha = float(tensors[self.alpha_name])        # handed to the kernels by value
+        self._dtype = rt.dtype
+
+    def forward(self, h: torch.Tensor) -> torch.Tensor:
+        return ops.add_dyn_tanh(h, None, self.alpha, self.weight, self.bias, self._dtype)
+
+    def add_forward(self, h, delta, rows=None, lazy=False):
+        delta_bias = None
+        if isinstance(delta, PendingLinear):
+            if rows is None and delta._y is None and delta.weight.shape[0] == self.width:
+                y = ops.linear_into_dyn_tanh(delta.x, delta.weight, delta.bias, h, self.alpha, self.weight, self.bias)
+                if y is not None:
+                    return y
+            if delta._y is None and self._dtype != torch.float32:
+                # unfused: the product's own bias joins in 32-bit on its way into the stream
+                delta_bias, delta = delta.bias, ops.linear(delta.x, delta.weight)
+            else:
+                delta = delta.materialize()
+        return ops.add_dyn_tanh(h, plain(delta), self.alpha, self.weight, self.bias, self._dtype, delta_bias=delta_bias, rows=rows)

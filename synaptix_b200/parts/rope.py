@@ -110,5 +110,25 @@ class FrequencyRamp(NamedTuple):
         return f / self.factor * ramp + f * (1.0 - ramp)
 
 
+class FrequencyBands(NamedTuple):
+    """Context extension by bands of wavelengths (the scheme of Llama 3.1): a pair that turns more than ``high`` times over
+    ``original`` positions keeps its frequency ``f``, one that turns less than ``low`` times gets ``f / factor``, and
+    between the two, with ``s = (turns - low) / (high - low)``, it is ``(1 - s) f / factor + s f``.  cos and sin keep
+    their size."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+    def magnitude(self) -> float:
+        return 1.0
+
+    def apply(self, f: np.ndarray, base: float, dims: int) -> np.ndarray:
+        wave = 2.0 * math.pi / f
+        s = (self.original / wave - self.low) / max(self.high - self.low, 1e-30)
+        blend = (1.0 - s) * f / self.factor + s * f
+        return np.where(wave < self.original / self.high, f, np.where(wave > self.original / self.low, f / self.factor, blend))
+
+
 class NoPosition(PositionEncoding):
     """Queries and keys are used as they are."""
