@@ -313,9 +313,29 @@ def zekalorn_config(width, ff, nh, nkv, hd, rh, runs, vocab):
                 max_positions=8192, token_side=dict(dim=256), loop=dict(start=0, stop=2, times=2), layers=layers)
 
 
+def penopel_config(width, ff, nh, nkv, hd, rh, runs, vocab):
+    """``runs`` layers (attention, latent attention, latent attention, an attention that reads the first one's keys) repeated.
+    Attention: grouped heads of ``hd``, half of a head rotated with frequencies scaled by bands, every earlier key visible;
+    latent attention: heads of ``hd/2`` unrotated and ``hd/2`` rotated elements with values of ``hd``, latents of ``width/8``
+    (queries ``width/2``), windows of 1,000; gated feed-forwards of ``ff`` everywhere."""
+    att = dict(heads=nh, kv_heads=nkv, dim=hd, vdim=hd, scale=hd ** -0.5,
+               rot=dict(dims=hd // 2, base=5.0e5, scaling=dict(factor=4.0, low=1.0, high=4.0, original=2048)))
+    lat = dict(heads=nh, dim=hd // 2, rot_dim=hd // 2, vdim=hd, q_rank=width // 2, kv_rank=width // 8, scale=hd ** -0.5,
+               mask=dict(size=1000), rot=dict(dims=hd // 2, base=1.0e6))
+    mlp = dict(kind="dense", ff=ff)
+    layers = []
+    for i in range(runs):
+        if i % 4 in (1, 2):
+            layers.append(dict(type="latent_attention", mixer=lat, mlp=mlp))
+        else:
+            layers.append(dict(type="attention", mixer=dict(att, kv_from=i - 3) if i % 4 == 3 else att, mlp=mlp))
+    return dict(architecture="Penopel", vocab=vocab, width=width, norm=dict(eps=1e-5), embedding=dict(scale=1.0),
+                logit_softcap=30.0, layers=layers)
+
+
 def arch_points(torch, a):
     from synaptix_b200.api import LLM
-    from synaptix_b200.config import LedudraConfig, PidutarConfig, Qwen3Config, TamovikConfig, VemedraConfig, ZekalornConfig
+    from synaptix_b200.config import LedudraConfig, PenopelConfig, PidutarConfig, Qwen3Config, TamovikConfig, VemedraConfig, ZekalornConfig
     from synaptix_b200.engine import DecodeRow, Entry
     from synaptix_b200.models import model_skeleton
     from synaptix_b200.parts import Runtime
@@ -378,11 +398,13 @@ def arch_points(torch, a):
             measure(TamovikConfig.from_dict(tamovik_config(width, ff, nh, nkv, hd, rh, RUNS, VOCAB)), f"tamovik_{name}")
         if a.arch == "zekalorn":
             measure(ZekalornConfig.from_dict(zekalorn_config(width, ff, nh, nkv, hd, rh, RUNS, VOCAB)), f"zekalorn_{name}")
+        if a.arch == "penopel":
+            measure(PenopelConfig.from_dict(penopel_config(width, ff, nh, nkv, hd, rh, RUNS, VOCAB)), f"penopel_{name}")
         if a.only:
             continue
-        if a.arch in ("pidutar", "tamovik", "zekalorn"):
+        if a.arch in ("pidutar", "tamovik", "zekalorn", "penopel"):
             measure(PidutarConfig.from_dict(pidutar_config(width, ff, nh, nkv, hd, rh, RUNS, VOCAB)), f"pidutar_{name}")
-        if a.arch in ("tamovik", "zekalorn"):
+        if a.arch in ("tamovik", "zekalorn", "penopel"):
             pass
         elif a.arch == "ledudra":
             measure(LedudraConfig.from_dict(ledudra_config(width, ff, nh, nkv, hd, rh, RUNS, VOCAB)), f"ledudra_{name}")
@@ -392,7 +414,8 @@ def arch_points(torch, a):
                                            num_key_value_heads=nkv, head_dim=hd, intermediate_size=ff, vocab_size=VOCAB,
                                            tie_word_embeddings=False)), f"qwen3_{name}")
     beside = {"pidutar": "Pidutar beside Vemedra and", "vemedra": "Vemedra beside", "ledudra": "Ledudra beside",
-              "tamovik": "Tamovik beside Pidutar and", "zekalorn": "Zekalorn beside Pidutar and"}[a.arch]
+              "tamovik": "Tamovik beside Pidutar and", "zekalorn": "Zekalorn beside Pidutar and",
+              "penopel": "Penopel beside Pidutar and"}[a.arch]
     return {"metric": f"prompt step and decode step, {beside} Qwen3 at equal sizes (bf16, random weights)", "impl": "ours",
             "layer_runs": RUNS, "vocab": VOCAB, "context": CONTEXT, "steps": K, "warmup": a.warmup, "sizes": VEMEDRA_SIZES,
             "data": "synthetic", "dtype": "bf16", "points": out}
@@ -419,12 +442,12 @@ def main():
     ap.add_argument("--short", action="store_true",
                     help="decode only 5 x --steps + --warmup tokens instead of at least 255 (small cases for profilers: "
                          "every launch under a profiler costs a good part of a second)")
-    ap.add_argument("--arch", default="qwen3", choices=["qwen3", "vemedra", "pidutar", "ledudra", "tamovik", "zekalorn"],
+    ap.add_argument("--arch", default="qwen3", choices=["qwen3", "vemedra", "pidutar", "ledudra", "tamovik", "zekalorn", "penopel"],
                     help="vemedra: the Vemedra decoder beside Qwen3 at equal sizes (prompt step, decode at batch 1 and 8) instead of "
                          "the default run; pidutar: the Pidutar decoder beside both; ledudra: the Ledudra decoder beside Qwen3; "
-                         "tamovik / zekalorn: that decoder beside Pidutar and Qwen3")
+                         "tamovik / zekalorn / penopel: that decoder beside Pidutar and Qwen3")
     ap.add_argument("--arch-sizes", default="", help="with another --arch than qwen3: which of 1k,2.5k,4k (default: all)")
-    ap.add_argument("--only", action="store_true", help="with --arch tamovik or zekalorn: that decoder alone (for profilers)")
+    ap.add_argument("--only", action="store_true", help="with --arch tamovik, zekalorn or penopel: that decoder alone (for profilers)")
     a = ap.parse_args()
 
     if a.impl == "reference":

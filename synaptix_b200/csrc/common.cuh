@@ -188,22 +188,30 @@ __device__ __forceinline__ float unary_act(float z, const GateAct a) {
 __device__ __forceinline__ float gelu_tanh_f32(float z) {
   // 1 + tanh(y) = 2 / (1 + exp(-2 y)): one exponential, no cancellation for large |y|
   const float y = 0.7978845608028654f * (z + 0.044715f * z * z * z);
-  return z / (1.f + __expf(-2.f * y));
+  return __fdividef(z, 1.f + __expf(-2.f * y));
 }
+// (The quotients are the fast ones, within 2 ulp: an exact division is a branch per value, and a product's epilogue, where a
+// warp has its scheduler to itself, then walks its values one after the other instead of side by side.)
 __device__ __forceinline__ float gate_mul(float g, float u, const GateAct a) {
   if (a.form == SX_GATE_GELU_TANH) return gelu_tanh_f32(g) * u;
   if (a.limit > 0.f) {
     g = fminf(g, a.limit);
     u = fminf(fmaxf(u, -a.limit), a.limit);
-    return g / (1.f + __expf(-a.alpha * g)) * (u + 1.f);
+    return __fdividef(g, 1.f + __expf(-a.alpha * g)) * (u + 1.f);
   }
-  return g / (1.f + __expf(-g)) * u;
+  return __fdividef(g, 1.f + __expf(-g)) * u;
 }
+// tanh(x) = 1 - 2 / (e^(2x) + 1) without a branch, absolute error of a few 1e-7: for the epilogues of 16-bit products (see
+// gate_mul about branches there); the 32-bit kernels call tanhf
+__device__ __forceinline__ float tanh_flat(float x) { return 1.f - __fdividef(2.f, __expf(2.f * x) + 1.f); }
 // cap * tanh(z / cap); cap <= 0: z as it is
 __device__ __forceinline__ float soft_limit(float z, float cap) { return cap > 0.f ? cap * tanhf(z / cap) : z; }
+__device__ __forceinline__ float soft_limit_flat(float z, float cap) { return cap > 0.f ? cap * tanh_flat(__fdividef(z, cap)) : z; }
 // The norm without statistics of a row: tanh(alpha v) * w + b, every element on its own.  Because it needs nothing of the
-// row's other elements, a product that adds itself into the residual stream finishes this norm in its epilogue.
+// row's other elements, a product that adds itself into the residual stream finishes this norm in its epilogue
+// (dyn_tanh_flat).
 __device__ __forceinline__ float dyn_tanh(float v, float alpha, float w, float b) { return fmaf(tanhf(alpha * v), w, b); }
+__device__ __forceinline__ float dyn_tanh_flat(float v, float alpha, float w, float b) { return fmaf(tanh_flat(alpha * v), w, b); }
 static GateAct g_sx_gate = {0.f, 0.f, SX_GATE_SIGMOID};
 extern "C" void sx_set_gate_act(float alpha, float limit, int form) { g_sx_gate.alpha = alpha; g_sx_gate.limit = limit; g_sx_gate.form = form; }
 

@@ -364,12 +364,12 @@ __global__ void __launch_bounds__(KS > SK_WARPS ? KS * 32 : SK_THREADS) skinny_g
         if (n0 < N) {
           const float v = hv[nt][j] + acc[nt][j];
           nrm.h_io[(size_t)b * N + n0] = v;
-          reinterpret_cast<bf16*>(out)[(size_t)b * N + n0] = __float2bfloat16_rn(dyn_tanh(v, nrm.alpha, gnext[0], shift[0]));
+          reinterpret_cast<bf16*>(out)[(size_t)b * N + n0] = __float2bfloat16_rn(dyn_tanh_flat(v, nrm.alpha, gnext[0], shift[0]));
         }
         if (n1 < N) {
           const float v = hv[nt][2 + j] + acc[nt][2 + j];
           nrm.h_io[(size_t)b * N + n1] = v;
-          reinterpret_cast<bf16*>(out)[(size_t)b * N + n1] = __float2bfloat16_rn(dyn_tanh(v, nrm.alpha, gnext[1], shift[1]));
+          reinterpret_cast<bf16*>(out)[(size_t)b * N + n1] = __float2bfloat16_rn(dyn_tanh_flat(v, nrm.alpha, gnext[1], shift[1]));
         }
       }
   } else if (EPI == EPI_RESID) {
@@ -418,8 +418,8 @@ __global__ void __launch_bounds__(KS > SK_WARPS ? KS * 32 : SK_THREADS) skinny_g
       } else {
         const int n0 = tile * 16 + g, n1 = n0 + 8;
         if (EPI == EPI_F32) {
-          if (n0 < N) reinterpret_cast<float*>(out)[(size_t)b * N + n0] = soft_limit(acc[nt][j], nrm.cap);
-          if (n1 < N) reinterpret_cast<float*>(out)[(size_t)b * N + n1] = soft_limit(acc[nt][2 + j], nrm.cap);
+          if (n0 < N) reinterpret_cast<float*>(out)[(size_t)b * N + n0] = soft_limit_flat(acc[nt][j], nrm.cap);
+          if (n1 < N) reinterpret_cast<float*>(out)[(size_t)b * N + n1] = soft_limit_flat(acc[nt][2 + j], nrm.cap);
         } else {
           if (n0 < N) reinterpret_cast<bf16*>(out)[(size_t)b * N + n0] = __float2bfloat16_rn(acc[nt][j]);
           if (n1 < N) reinterpret_cast<bf16*>(out)[(size_t)b * N + n1] = __float2bfloat16_rn(acc[nt][2 + j]);

@@ -26,8 +26,9 @@
 #define TC_BK 64
 #define TC_A_BYTES (TC_BM * TC_BK * 2)            // 16 KB
 #define TC_THREADS 192
-// (the epilogue that prepares heads has eight epilogue warps, one group of four per head of the tile)
-template <int EPI> struct TcThreads { static constexpr int N = (EPI == 4 || EPI == 6) ? 320 : TC_THREADS; };
+// (Two groups of four epilogue warps, each with half of the tile's columns, where the epilogue has much to do: the ones that
+// prepare heads (a head a group) and the one that ends in the residual stream and its norm, which moves 10 bytes an element.)
+template <int EPI> struct TcThreads { static constexpr int N = (EPI == 4 || EPI == 5 || EPI == 6) ? 320 : TC_THREADS; };
 #define TC_RED_ROWS 6
 
 enum { TC_EPI_BF16 = 0, TC_EPI_F32 = 1, TC_EPI_SILU_MUL = 2, TC_EPI_PARTIAL = 3, TC_EPI_QKV = 4, TC_EPI_RESID_TANH = 5, TC_EPI_QKV_BIAS = 6 };
@@ -259,7 +260,7 @@ __device__ __forceinline__ void tc_store4(float (&a)[4], const float (&b)[4], vo
   }
   if (EPI == TC_EPI_F32) {
 #pragma unroll
-    for (int j = 0; j < 4; ++j) a[j] = soft_limit(a[j], ep.cap);
+    for (int j = 0; j < 4; ++j) a[j] = soft_limit_flat(a[j], ep.cap);
     float* dst = reinterpret_cast<float*>(out) + at;
     if (vec) *reinterpret_cast<float4*>(dst) = make_float4(a[0], a[1], a[2], a[3]);
     else
@@ -274,15 +275,15 @@ __device__ __forceinline__ void tc_store4(float (&a)[4], const float (&b)[4], vo
       const float4 w = __ldg(reinterpret_cast<const float4*>(ep.gain + col)), s = __ldg(reinterpret_cast<const float4*>(ep.shift + col));
       a[0] += hv.x; a[1] += hv.y; a[2] += hv.z; a[3] += hv.w;
       *reinterpret_cast<float4*>(h) = make_float4(a[0], a[1], a[2], a[3]);
-      a[0] = dyn_tanh(a[0], ep.alpha, w.x, s.x); a[1] = dyn_tanh(a[1], ep.alpha, w.y, s.y);
-      a[2] = dyn_tanh(a[2], ep.alpha, w.z, s.z); a[3] = dyn_tanh(a[3], ep.alpha, w.w, s.w);
+      a[0] = dyn_tanh_flat(a[0], ep.alpha, w.x, s.x); a[1] = dyn_tanh_flat(a[1], ep.alpha, w.y, s.y);
+      a[2] = dyn_tanh_flat(a[2], ep.alpha, w.z, s.z); a[3] = dyn_tanh_flat(a[3], ep.alpha, w.w, s.w);
     } else {
 #pragma unroll
       for (int j = 0; j < 4; ++j)
         if (j < cols) {
           const float v = h[j] + a[j];
           h[j] = v;
-          a[j] = dyn_tanh(v, ep.alpha, __ldg(ep.gain + col + j), __ldg(ep.shift + col + j));
+          a[j] = dyn_tanh_flat(v, ep.alpha, __ldg(ep.gain + col + j), __ldg(ep.shift + col + j));
         }
     }
   }
@@ -352,8 +353,8 @@ __device__ __forceinline__ void tc_store_chunk(const uint32_t (&v)[32], const ui
     float* dst = reinterpret_cast<float*>(out) + at;
 #pragma unroll
     for (int i = 0; i < 8; ++i)
-      reinterpret_cast<float4*>(dst)[i] = make_float4(soft_limit(f[4 * i], ep.cap), soft_limit(f[4 * i + 1], ep.cap),
-                                                      soft_limit(f[4 * i + 2], ep.cap), soft_limit(f[4 * i + 3], ep.cap));
+      reinterpret_cast<float4*>(dst)[i] = make_float4(soft_limit_flat(f[4 * i], ep.cap), soft_limit_flat(f[4 * i + 1], ep.cap),
+                                                      soft_limit_flat(f[4 * i + 2], ep.cap), soft_limit_flat(f[4 * i + 3], ep.cap));
     return;
   }
   if (EPI == TC_EPI_RESID_TANH) {
@@ -364,10 +365,10 @@ __device__ __forceinline__ void tc_store_chunk(const uint32_t (&v)[32], const ui
       const float x0 = f[4 * i] + hv[4 * i], x1 = f[4 * i + 1] + hv[4 * i + 1], x2 = f[4 * i + 2] + hv[4 * i + 2],
                   x3 = f[4 * i + 3] + hv[4 * i + 3];
       reinterpret_cast<float4*>(ep.h + at)[i] = make_float4(x0, x1, x2, x3);
-      f[4 * i] = dyn_tanh(x0, ep.alpha, w.x, s.x);
-      f[4 * i + 1] = dyn_tanh(x1, ep.alpha, w.y, s.y);
-      f[4 * i + 2] = dyn_tanh(x2, ep.alpha, w.z, s.z);
-      f[4 * i + 3] = dyn_tanh(x3, ep.alpha, w.w, s.w);
+      f[4 * i] = dyn_tanh_flat(x0, ep.alpha, w.x, s.x);
+      f[4 * i + 1] = dyn_tanh_flat(x1, ep.alpha, w.y, s.y);
+      f[4 * i + 2] = dyn_tanh_flat(x2, ep.alpha, w.z, s.z);
+      f[4 * i + 3] = dyn_tanh_flat(x3, ep.alpha, w.w, s.w);
     }
   }
   bf16* dst = reinterpret_cast<bf16*>(out) + at;
@@ -573,7 +574,9 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
     }
   } else {
     const int quarter = warp & 3;
-    const int et = threadIdx.x - 64;                                    // 0..127 among the epilogue threads
+    constexpr int ET = TcThreads<EPI>::N - 64, GROUPS = ET / 128;        // epilogue threads; groups of four warps
+    const int group = (warp - 2) >> 2;                                  // which half of the tile's columns (one group: all)
+    const int et = threadIdx.x - 64;                                    // among the epilogue threads
     // a partial tile in the workspace: [tile among the cut ones][piece][128 rows][BN columns] float32
     auto ws_of = [&](int tile, int z) { return piece_ws + ((size_t)(tile - n_whole) * zmax + z) * (TC_BM * BN); };
     // a finished accumulator -> out, with the epilogue
@@ -681,12 +684,12 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
         }
       } else {
 #pragma unroll 1
-        for (int c0 = 0; c0 < tile_n; c0 += 32) {
+        for (int c0 = group * (tile_n / GROUPS); c0 < (group + 1) * (tile_n / GROUPS); c0 += 32) {
           uint32_t v[32], u[32];
           tc_ld32(t_row + c0, v);
           if (EPI == TC_EPI_SILU_MUL) tc_ld32(t_row + BN / 2 + c0, u);
           asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
-          if (c0 + 32 >= tile_n) {
+          if (c0 + 32 >= (group + 1) * (tile_n / GROUPS)) {
             // everything of this accumulator is in registers: hand it back before the last stores
             asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
             __syncwarp();
@@ -717,12 +720,12 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
       float* dst = ws_of(tile, pc[w].z) + (size_t)(quarter * 32 + lane) * BN;
       // (four tcgen05.ld on the way per wait)
 #pragma unroll 1
-      for (int c0 = 0; c0 < BN; c0 += 128) {
+      for (int c0 = group * (BN / GROUPS); c0 < (group + 1) * (BN / GROUPS); c0 += 128) {
         uint32_t v[4][32];
 #pragma unroll
         for (int j = 0; j < 4; ++j) tc_ld32(t_row + c0 + 32 * j, v[j]);
         asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
-        if (c0 + 128 >= BN) {
+        if (c0 + 128 >= (group + 1) * (BN / GROUPS)) {
           asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
           __syncwarp();
           if (lane == 0) tc_mbar_arrive(acc_empty0 + 8 * buf);
@@ -738,7 +741,7 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
       }
       if (coop) {
         __threadfence();
-        asm volatile("bar.sync 1, 128;\n" ::: "memory");                 // the four epilogue warps
+        asm volatile("bar.sync 1, %0;\n" ::"n"(ET) : "memory");                 // the epilogue warps
         if (threadIdx.x == 64) atomicAdd(piece_count + 2 * (tile - n_whole), 1);
       }
     }
@@ -762,7 +765,7 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
         if (!all) sx_set_status(status, 5);
         *piece_ok = all;
       }
-      asm volatile("bar.sync 1, 128;\n" ::: "memory");
+      asm volatile("bar.sync 1, %0;\n" ::"n"(ET) : "memory");
       if (*piece_ok) {
         __threadfence();
         const int m0 = (tile % tiles_m) * TC_BM, n0 = (tile / tiles_m) * tile_n;
@@ -771,7 +774,7 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
         const int r_lo = m0 + z * per, r_hi = min(m0 + rows_here, r_lo + per);
         const int cols = min(tile_n, n_out - n0);                        // output columns of this tile
         constexpr int TPR = EPI == TC_EPI_SILU_MUL ? 32 : 64;            // threads a row (four columns a thread)
-        constexpr int RPI = 128 / TPR;                                   // rows at a time
+        constexpr int RPI = ET / TPR;                                   // rows at a time
         const int c4 = (et % TPR) * 4;
         const float* base = ws_of(tile, 0);
         const size_t plane = (size_t)TC_BM * BN;
@@ -808,11 +811,11 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
           }
         }
       }
-      asm volatile("bar.sync 1, 128;\n" ::: "memory");                   // everyone has read; piece_ok is free again
+      asm volatile("bar.sync 1, %0;\n" ::"n"(ET) : "memory");                   // everyone has read; piece_ok is free again
       if (threadIdx.x == 64 && *piece_ok) {
         if (atomicAdd(cnt + 1, 1) == nz - 1) { cnt[1] = 0; __threadfence(); cnt[0] = 0; }
       }
-      asm volatile("bar.sync 1, 128;\n" ::: "memory");
+      asm volatile("bar.sync 1, %0;\n" ::"n"(ET) : "memory");
     }
     // 3: the whole tiles
     for (int w = n_pc; w < n_work && alive; ++w) {
@@ -1051,11 +1054,11 @@ __global__ void tc_splitk_reduce_kernel(const float* __restrict__ ws, void* __re
   }
   const size_t o = m * (size_t)ldo + n;
   if (EPI == TC_EPI_SILU_MUL) reinterpret_cast<bf16*>(out)[o] = __float2bfloat16_rn(gate_mul(a, b, ep.act));
-  else if (EPI == TC_EPI_F32) reinterpret_cast<float*>(out)[o] = soft_limit(a, ep.cap);
+  else if (EPI == TC_EPI_F32) reinterpret_cast<float*>(out)[o] = soft_limit_flat(a, ep.cap);
   else if (EPI == TC_EPI_RESID_TANH) {
     const float v = ep.h[o] + a;
     ep.h[o] = v;
-    reinterpret_cast<bf16*>(out)[o] = __float2bfloat16_rn(dyn_tanh(v, ep.alpha, __ldg(ep.gain + n), __ldg(ep.shift + n)));
+    reinterpret_cast<bf16*>(out)[o] = __float2bfloat16_rn(dyn_tanh_flat(v, ep.alpha, __ldg(ep.gain + n), __ldg(ep.shift + n)));
   } else reinterpret_cast<bf16*>(out)[o] = __float2bfloat16_rn(a);
 }
 

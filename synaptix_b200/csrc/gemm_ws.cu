@@ -330,7 +330,7 @@ __global__ void __launch_bounds__(WS_THREADS, 2) gemm_ws_kernel(const __grid_con
         for (int j = 0; j < 4; ++j) o[j] = fmaf(o[j], rf, ba[j]);
         if (EPI == WS_EPI_F32)
 #pragma unroll
-          for (int j = 0; j < 4; ++j) o[j] = soft_limit(o[j], ep.cap);
+          for (int j = 0; j < 4; ++j) o[j] = soft_limit_flat(o[j], ep.cap);
       }
       const int n = n0 + c;
       const int cols = valid ? min(4, n_out - n) : 0;                      // <= 0: beyond the matrix
@@ -344,8 +344,8 @@ __global__ void __launch_bounds__(WS_THREADS, 2) gemm_ws_kernel(const __grid_con
             const float4 g4v = *reinterpret_cast<const float4*>(ep.gain + n), s4v = *reinterpret_cast<const float4*>(ep.shift + n);
             const float4 v = make_float4(h4.x + o[0], h4.y + o[1], h4.z + o[2], h4.w + o[3]);
             *reinterpret_cast<float4*>(ep.h + at) = v;
-            __nv_bfloat162 lo = __floats2bfloat162_rn(dyn_tanh(v.x, ep.alpha, g4v.x, s4v.x), dyn_tanh(v.y, ep.alpha, g4v.y, s4v.y));
-            __nv_bfloat162 hi = __floats2bfloat162_rn(dyn_tanh(v.z, ep.alpha, g4v.z, s4v.z), dyn_tanh(v.w, ep.alpha, g4v.w, s4v.w));
+            __nv_bfloat162 lo = __floats2bfloat162_rn(dyn_tanh_flat(v.x, ep.alpha, g4v.x, s4v.x), dyn_tanh_flat(v.y, ep.alpha, g4v.y, s4v.y));
+            __nv_bfloat162 hi = __floats2bfloat162_rn(dyn_tanh_flat(v.z, ep.alpha, g4v.z, s4v.z), dyn_tanh_flat(v.w, ep.alpha, g4v.w, s4v.w));
             uint2 pk;
             pk.x = *reinterpret_cast<uint32_t*>(&lo); pk.y = *reinterpret_cast<uint32_t*>(&hi);
             *reinterpret_cast<uint2*>(xo) = pk;
@@ -353,7 +353,7 @@ __global__ void __launch_bounds__(WS_THREADS, 2) gemm_ws_kernel(const __grid_con
             for (int j = 0; j < cols; ++j) {
               const float v = ep.h[at + j] + o[j];
               ep.h[at + j] = v;
-              xo[j] = __float2bfloat16_rn(dyn_tanh(v, ep.alpha, ep.gain[n + j], ep.shift[n + j]));
+              xo[j] = __float2bfloat16_rn(dyn_tanh_flat(v, ep.alpha, ep.gain[n + j], ep.shift[n + j]));
             }
           }
         }
