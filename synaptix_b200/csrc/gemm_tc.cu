@@ -67,6 +67,10 @@ struct TcEp {
   const float* shift;
 };
 
+// floats a warp of the persistent kernel's epilogue stages of a tile's vectors (see tc_store_chunk)
+template <int EPI> struct TcVec { static constexpr int N = EPI == 4 ? 0 : (EPI == 6 ? 128 : (EPI == 5 ? 384 : 256)); };
+template <int EPI> constexpr int tc_vec_floats() { return TcVec<EPI>::N * ((TcThreads<EPI>::N - 64) / 32); }
+
 // BN: columns of W per block (256, or 128 for the split-K form); stages fill the shared memory
 template <int BN> struct TcShape {
   static constexpr int B_BYTES = BN * TC_BK * 2;
@@ -299,12 +303,28 @@ __device__ __forceinline__ void tc_store4(float (&a)[4], const float (&b)[4], vo
   }
 }
 
-// 32 columns of one row out of the accumulator (u: the up half's)
+// eight 32-bit words to or from 32-byte aligned global memory, one instruction
+__device__ __forceinline__ void tc_ldg8(const float* p, float* v) {
+  asm volatile("ld.global.v8.f32 {%0,%1,%2,%3,%4,%5,%6,%7}, [%8];\n"
+               : "=f"(v[0]), "=f"(v[1]), "=f"(v[2]), "=f"(v[3]), "=f"(v[4]), "=f"(v[5]), "=f"(v[6]), "=f"(v[7]) : "l"(p) : "memory");
+}
+__device__ __forceinline__ void tc_stg8(float* p, const float* v) {
+  asm volatile("st.global.v8.f32 [%8], {%0,%1,%2,%3,%4,%5,%6,%7};\n"
+               ::"f"(v[0]), "f"(v[1]), "f"(v[2]), "f"(v[3]), "f"(v[4]), "f"(v[5]), "f"(v[6]), "f"(v[7]), "l"(p) : "memory");
+}
+__device__ __forceinline__ float tc_pack_bf16(float a, float b) {
+  __nv_bfloat162 t = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<float*>(&t);
+}
+
+// 32 columns of one row out of the accumulator (u: the up half's).  `sv` is what the warp has staged of the tile's vectors, at
+// this chunk: its biases (SILU_MUL: 128 further the up half's; RESID_TANH: 128 further the gains, 256 further the shifts); hv the
+// stream's values.  Both are for whole chunks of rows of a multiple of 16 elements (`whole`), the rest reads memory.
 template <int EPI>
 __device__ __forceinline__ void tc_store_chunk(const uint32_t (&v)[32], const uint32_t (&u)[32], void* __restrict__ out,
-                                               int row, int col, int n_out, const TcEp& ep) {
-  const int ncol = min(32, n_out - col);
-  if (ncol < 32 || (n_out & 7) != 0) {
+                                               int row, int col, int n_out, bool whole, const float* sv, const float* hv, const TcEp& ep) {
+  if (!whole) {
+    const int ncol = min(32, n_out - col);
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       float a[4], b[4] = {0.f, 0.f, 0.f, 0.f};
@@ -321,28 +341,18 @@ __device__ __forceinline__ void tc_store_chunk(const uint32_t (&v)[32], const ui
 #pragma unroll
   for (int i = 0; i < 32; ++i) f[i] = __uint_as_float(v[i]);
   const size_t at = (size_t)row * n_out + col;
-  float hv[EPI == TC_EPI_RESID_TANH ? 32 : 1];
-  if (EPI == TC_EPI_RESID_TANH) {
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const float4 h4 = reinterpret_cast<const float4*>(ep.h + at)[i];
-      hv[4 * i] = h4.x; hv[4 * i + 1] = h4.y; hv[4 * i + 2] = h4.z; hv[4 * i + 3] = h4.w;
-    }
-  }
   if (ep.bias) {
-    const float4* b4 = reinterpret_cast<const float4*>(ep.bias + col);
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      const float4 b = __ldg(b4 + i);
+      const float4 b = *reinterpret_cast<const float4*>(sv + 4 * i);
       f[4 * i] += b.x; f[4 * i + 1] += b.y; f[4 * i + 2] += b.z; f[4 * i + 3] += b.w;
     }
   }
   if (EPI == TC_EPI_SILU_MUL) {
-    const float4* b4 = reinterpret_cast<const float4*>(ep.bias + n_out + col);
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (ep.bias) b = __ldg(b4 + i);
+      if (ep.bias) b = *reinterpret_cast<const float4*>(sv + 128 + 4 * i);
       f[4 * i] = gate_mul(f[4 * i], __uint_as_float(u[4 * i]) + b.x, ep.act);
       f[4 * i + 1] = gate_mul(f[4 * i + 1], __uint_as_float(u[4 * i + 1]) + b.y, ep.act);
       f[4 * i + 2] = gate_mul(f[4 * i + 2], __uint_as_float(u[4 * i + 2]) + b.z, ep.act);
@@ -352,34 +362,32 @@ __device__ __forceinline__ void tc_store_chunk(const uint32_t (&v)[32], const ui
   if (EPI == TC_EPI_F32) {
     float* dst = reinterpret_cast<float*>(out) + at;
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
-      reinterpret_cast<float4*>(dst)[i] = make_float4(soft_limit_flat(f[4 * i], ep.cap), soft_limit_flat(f[4 * i + 1], ep.cap),
-                                                      soft_limit_flat(f[4 * i + 2], ep.cap), soft_limit_flat(f[4 * i + 3], ep.cap));
+    for (int i = 0; i < 32; ++i) f[i] = soft_limit_flat(f[i], ep.cap);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) tc_stg8(dst + 8 * i, f + 8 * i);
     return;
   }
   if (EPI == TC_EPI_RESID_TANH) {
-    const float4 *w4 = reinterpret_cast<const float4*>(ep.gain + col), *s4 = reinterpret_cast<const float4*>(ep.shift + col);
+#pragma unroll
+    for (int i = 0; i < 32; ++i) f[i] += hv[i];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) tc_stg8(ep.h + at + 8 * i, f + 8 * i);
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      const float4 w = __ldg(w4 + i), s = __ldg(s4 + i);
-      const float x0 = f[4 * i] + hv[4 * i], x1 = f[4 * i + 1] + hv[4 * i + 1], x2 = f[4 * i + 2] + hv[4 * i + 2],
-                  x3 = f[4 * i + 3] + hv[4 * i + 3];
-      reinterpret_cast<float4*>(ep.h + at)[i] = make_float4(x0, x1, x2, x3);
-      f[4 * i] = dyn_tanh_flat(x0, ep.alpha, w.x, s.x);
-      f[4 * i + 1] = dyn_tanh_flat(x1, ep.alpha, w.y, s.y);
-      f[4 * i + 2] = dyn_tanh_flat(x2, ep.alpha, w.z, s.z);
-      f[4 * i + 3] = dyn_tanh_flat(x3, ep.alpha, w.w, s.w);
+      const float4 w = *reinterpret_cast<const float4*>(sv + 128 + 4 * i), s = *reinterpret_cast<const float4*>(sv + 256 + 4 * i);
+      f[4 * i] = dyn_tanh_flat(f[4 * i], ep.alpha, w.x, s.x);
+      f[4 * i + 1] = dyn_tanh_flat(f[4 * i + 1], ep.alpha, w.y, s.y);
+      f[4 * i + 2] = dyn_tanh_flat(f[4 * i + 2], ep.alpha, w.z, s.z);
+      f[4 * i + 3] = dyn_tanh_flat(f[4 * i + 3], ep.alpha, w.w, s.w);
     }
   }
   bf16* dst = reinterpret_cast<bf16*>(out) + at;
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    uint4 p;
-    __nv_bfloat162 t0 = __floats2bfloat162_rn(f[8 * i], f[8 * i + 1]), t1 = __floats2bfloat162_rn(f[8 * i + 2], f[8 * i + 3]);
-    __nv_bfloat162 t2 = __floats2bfloat162_rn(f[8 * i + 4], f[8 * i + 5]), t3 = __floats2bfloat162_rn(f[8 * i + 6], f[8 * i + 7]);
-    p.x = *reinterpret_cast<uint32_t*>(&t0); p.y = *reinterpret_cast<uint32_t*>(&t1);
-    p.z = *reinterpret_cast<uint32_t*>(&t2); p.w = *reinterpret_cast<uint32_t*>(&t3);
-    reinterpret_cast<uint4*>(dst)[i] = p;
+  for (int i = 0; i < 2; ++i) {
+    float p[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) p[j] = tc_pack_bf16(f[16 * i + 2 * j], f[16 * i + 2 * j + 1]);
+    tc_stg8(reinterpret_cast<float*>(dst + 16 * i), p);
   }
 }
 
@@ -455,6 +463,7 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
   uint64_t* bars = reinterpret_cast<uint64_t*>(tiles + STAGES * STAGE_BYTES);   // full[S], empty[S], acc_full[2], acc_empty[2]
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 2 * STAGES + 4);
   volatile int* piece_ok = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  float* vecs = reinterpret_cast<float*>((reinterpret_cast<uintptr_t>(tmem_slot + 2) + 15) & ~(uintptr_t)15);   // [epilogue warps][TcVec]
   const uint32_t full0 = tc_smem(bars), empty0 = tc_smem(bars + STAGES);
   const uint32_t acc_full0 = tc_smem(bars + 2 * STAGES), acc_empty0 = tc_smem(bars + 2 * STAGES + 2);
 
@@ -591,6 +600,43 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
         pos = qk.positions[row];
         page = qk.block_table[(size_t)qk.seq_of_token[row] * qk.maxp + (pos >> 6)];
       }
+      // Vectors over the columns, and the stream's first values, are asked for while the tile's MMAs still run.  A warp keeps
+      // its own copy (a barrier among warps is not needed); threads own rows, so every thread reads all of them.
+      constexpr bool RESID = EPI == TC_EPI_RESID_TANH;
+      constexpr int CW = (EPI == TC_EPI_SILU_MUL ? BN / 2 : BN) / GROUPS;     // columns of C this warp finishes
+      const int cb = group * CW;
+      float* sv = vecs + (warp - 2) * TcVec<EPI>::N;
+      const bool wide = (n_out & 15) == 0 && ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(ep.h)) & 31) == 0;
+      auto whole_at = [&](int c0) { return wide && n0 + c0 + 32 <= n_out; };
+      float hv[RESID ? 32 : 1];
+      auto load_h = [&](int c0, float* dst) {
+        if (row < M && whole_at(c0)) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) tc_ldg8(ep.h + (size_t)row * n_out + n0 + c0 + 8 * i, dst + 8 * i);
+        }
+      };
+      if (!QKV && wide && (RESID || ep.bias)) {
+        __syncwarp();                                  // (the tile before has been read)
+        for (int i = lane * 4; i < CW; i += 128) {
+          const int col = n0 + cb + i;
+          if (col + 4 <= n_out) {
+            if (ep.bias) *reinterpret_cast<float4*>(sv + i) = __ldg(reinterpret_cast<const float4*>(ep.bias + col));
+            if (EPI == TC_EPI_SILU_MUL && ep.bias)
+              *reinterpret_cast<float4*>(sv + 128 + i) = __ldg(reinterpret_cast<const float4*>(ep.bias + n_out + col));
+            if (RESID) {
+              *reinterpret_cast<float4*>(sv + 128 + i) = __ldg(reinterpret_cast<const float4*>(ep.gain + col));
+              *reinterpret_cast<float4*>(sv + 256 + i) = __ldg(reinterpret_cast<const float4*>(ep.shift + col));
+            }
+          }
+        }
+        __syncwarp();
+      }
+      if (EPI == TC_EPI_QKV_BIAS) {                    // (a warp's columns are one head's)
+        __syncwarp();
+        *reinterpret_cast<float4*>(sv + lane * 4) = __ldg(reinterpret_cast<const float4*>(qk.bias + n0 + cb) + lane);
+        __syncwarp();
+      }
+      if (RESID) load_h(cb, hv);
       if (!tc_mbar_wait(acc_full0 + 8 * buf, use & 1)) {
         if (lane == 0) sx_set_status(status, 3);
         return false;
@@ -604,25 +650,18 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
           const int hh = (warp - 2) >> 2;                 // warps 2-5 take the tile's first head, warps 6-9 its second
           const int head = n0 / 128 + hh;
           float x[128];
-          // (with biases 32 columns at a time, each with its wait: this epilogue is short of registers, and the biases of a
-          //  whole head on the way at once would spill)
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            tc_ld32(t_row + hh * 128 + c * 32, *reinterpret_cast<uint32_t(*)[32]>(&x[c * 32]));
-            if (EPI == TC_EPI_QKV_BIAS) {
-              asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
-#pragma unroll
-              for (int i = 0; i < 8; ++i) {
-                float4 b;
-                asm volatile("ld.global.v4.f32 {%0, %1, %2, %3}, [%4];\n" : "=f"(b.x), "=f"(b.y), "=f"(b.z), "=f"(b.w)
-                             : "l"(qk.bias + head * 128 + c * 32 + 4 * i) : "memory");
-                x[c * 32 + 4 * i] += b.x; x[c * 32 + 4 * i + 1] += b.y; x[c * 32 + 4 * i + 2] += b.z; x[c * 32 + 4 * i + 3] += b.w;
-              }
-            }
-          }
+          for (int c = 0; c < 4; ++c) tc_ld32(t_row + hh * 128 + c * 32, *reinterpret_cast<uint32_t(*)[32]>(&x[c * 32]));
           asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
 #pragma unroll
-          for (int i = 0; i < 128; ++i) x[i] = __bfloat162float(__float2bfloat16_rn(x[i]));
+          for (int i = 0; i < 32; ++i) {
+            if (EPI == TC_EPI_QKV_BIAS) {
+              const float4 b = *reinterpret_cast<const float4*>(sv + 4 * i);
+              x[4 * i] += b.x; x[4 * i + 1] += b.y; x[4 * i + 2] += b.z; x[4 * i + 3] += b.w;
+            }
+#pragma unroll
+            for (int jj = 0; jj < 4; ++jj) x[4 * i + jj] = __bfloat162float(__float2bfloat16_rn(x[4 * i + jj]));
+          }
           // this warp's part of the accumulator is in registers: hand it back
           asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
           __syncwarp();
@@ -684,18 +723,24 @@ __global__ void __launch_bounds__(TcThreads<EPI>::N, 1) gemm_tc_persistent_kerne
         }
       } else {
 #pragma unroll 1
-        for (int c0 = group * (tile_n / GROUPS); c0 < (group + 1) * (tile_n / GROUPS); c0 += 32) {
+        for (int c0 = cb; c0 < cb + CW; c0 += 32) {
           uint32_t v[32], u[32];
+          float hn[RESID ? 32 : 1];
           tc_ld32(t_row + c0, v);
           if (EPI == TC_EPI_SILU_MUL) tc_ld32(t_row + BN / 2 + c0, u);
+          if (RESID && c0 + 32 < cb + CW) load_h(c0 + 32, hn);       // (the next chunk's values, behind this chunk's work)
           asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
-          if (c0 + 32 >= (group + 1) * (tile_n / GROUPS)) {
+          if (c0 + 32 >= cb + CW) {
             // everything of this accumulator is in registers: hand it back before the last stores
             asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
             __syncwarp();
             if (lane == 0) tc_mbar_arrive(acc_empty0 + 8 * buf);
           }
-          if (row < M && n0 + c0 < n_out) tc_store_chunk<EPI>(v, u, out, row, n0 + c0, n_out, ep);
+          if (row < M && n0 + c0 < n_out) tc_store_chunk<EPI>(v, u, out, row, n0 + c0, n_out, whole_at(c0), sv + (c0 - cb), hv, ep);
+          if (RESID) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) hv[i] = hn[i];
+          }
         }
       }
       return true;
@@ -1017,7 +1062,7 @@ static int tc_launch_persistent(const CUtensorMap& ma, const CUtensorMap& mw, vo
   int* status = tc_status_word();
   if (!status) return (int)cudaErrorMemoryAllocation;
   if (h.n_whole < 0 || h.G <= 0) return SX_ERR_SIZE;
-  const size_t smem = 1024 + TcShape<BN>::STAGES * TcShape<BN>::STAGE_BYTES + (2 * TcShape<BN>::STAGES + 4) * sizeof(uint64_t) + 32;
+  const size_t smem = 1024 + TcShape<BN>::STAGES * TcShape<BN>::STAGE_BYTES + (2 * TcShape<BN>::STAGES + 4) * sizeof(uint64_t) + 32 + tc_vec_floats<EPI>() * sizeof(float);
   auto kern = gemm_tc_persistent_kernel<EPI, BN>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
