@@ -20,7 +20,8 @@ switches in its runtime options (crates/synaptix-config/src/runtime.rs, ``AttnBa
 ``qkv_epilogue``    prompt steps at head size 128: the q/k/v product prepares the heads in its epilogue (norm,
                     rotation, cache write; else a head-preparation launch)
 ``fused_residual``  2 to 160 rows: the o / down product adds itself into the residual stream and
-                    prepares the next norm
+                    prepares the next norm; any number of rows where that norm needs no statistics of the row
+                    (the product then finishes it)
 ``attn_options_fast``  attention with capped scores, sinks or chunks of positions at head size 32 / 64 / 128 in
                     bfloat16 on the ``mma.sync`` kernels (else the plain kernel)
 ``attn_scored_tc``  prompt portions of the attention with sigmoid weights of scores mixed over the heads, in bfloat16
