@@ -319,7 +319,7 @@ def penopel_config(width, ff, nh, nkv, hd, rh, runs, vocab):
     latent attention: heads of ``hd/2`` unrotated and ``hd/2`` rotated elements with values of ``hd``, latents of ``width/8``
     (queries ``width/2``), windows of 1,000; gated feed-forwards of ``ff`` everywhere."""
     att = dict(heads=nh, kv_heads=nkv, dim=hd, vdim=hd, scale=hd ** -0.5,
-               rot=dict(dims=hd // 2, base=5.0e5, scaling=dict(factor=4.0, low=1.0, high=4.0, original=2048)))
+               rot=dict(dims=hd // 2, base=2.0e5, scaling=dict(factor=4.0, low=1.0, high=3.0, original=2048)))
     lat = dict(heads=nh, dim=hd // 2, rot_dim=hd // 2, vdim=hd, q_rank=width // 2, kv_rank=width // 8, scale=hd ** -0.5,
                mask=dict(size=1000), rot=dict(dims=hd // 2, base=1.0e6))
     mlp = dict(kind="dense", ff=ff)

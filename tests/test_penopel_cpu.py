@@ -112,7 +112,7 @@ def test_a_partial_rotation_bound_as_a_whole_one():
 
 def test_frequencies_by_bands_of_wavelengths():
     from synaptix_b200.parts import FrequencyBands, RotaryHalf, RotaryPairs, Runtime
-    for dims, base, bands in ((16, 3.0e4, (5.0, 1.0, 3.0, 400.0)), (6, 9000.0, (3.0, 0.5, 6.0, 60.0)), (32, 1.0e6, (8.0, 1.0, 4.0, 90.0)),
+    for dims, base, bands in ((16, 3.0e4, (5.0, 1.0, 3.0, 400.0)), (6, 9000.0, (3.0, 0.5, 6.0, 60.0)), (32, 4.0e6, (6.0, 1.2, 4.5, 90.0)),
                               (8, 10.0, (2.0, 1.5, 1.5, 30.0))):
         rot = dict(dims=dims, base=base, scaling=dict(zip(("factor", "low", "high", "original"), bands)))
         want = PN.frequencies(rot)
